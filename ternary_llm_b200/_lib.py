@@ -61,7 +61,19 @@ SIGNATURES = {
     "tllm_b200_decoder_reset": (_int, [_vp, _vp]),
     "tllm_b200_decoder_forward": (_int, [_vp, _vp, _int, _int, _vp, _vp]),
     "tllm_b200_decoder_generate": (_int, [_vp, _int, _int, _int, _vp, _vp]),
+    # include/tllm_b200_mixed.h
+    "tllm_b200_mixed_decoder_create": (_int, [_vp, _int, _int, _vp]),
+    "tllm_b200_mixed_decoder_runs": (_int, [_vp]),
+    "tllm_b200_decoder_forward_logits": (_int, [_vp, _int, _vp, _int, _int, _vp, _int, _vp, _vp, _vp]),
+    "tllm_b200_dense_linear": (_int, [_int] + [_vp] * 4 + [_int] * 5 + [_vp]),
+    "tllm_b200_causal_conv": (_int, [_int] + [_vp] * 5 + [_int] * 6 + [_vp]),
+    "tllm_b200_selective_scan": (_int, [_int] + [_vp] * 8 + [_int] * 5 + [_vp]),
+    "tllm_b200_gated_scan": (_int, [_int] + [_vp] * 6 + [_int, _int, ctypes.c_float] + [_int] * 4 + [_vp]),
+    "tllm_b200_latent_attention": (_int, [_int] + [_vp] * 4 + [_int] * 3 + [ctypes.c_float] + [_int] * 4 + [_vp]),
+    "tllm_b200_latent_attention_expanded": (_int, [_vp] * 7 + [_int] * 5 + [ctypes.c_float] + [_int] * 3 + [_vp]),
 }
+
+TENSORS_PER_LAYER = 31      # TLLM_T_COUNT
 
 
 class TernaryWeightDesc(ctypes.Structure):
@@ -84,6 +96,22 @@ class ModelDesc(ctypes.Structure):
                [("rope_theta", ctypes.c_float), ("rms_norm_eps", ctypes.c_float),
                 ("embedding_table", _vp), ("final_norm_weight", _vp), ("lm_head_weight", _vp),
                 ("lm_head_ternary", TernaryWeightDesc), ("layers", ctypes.POINTER(LayerWeightsDesc))]
+
+
+class MixedLayerDesc(ctypes.Structure):
+    """tllm_b200_mixed_layer (include/tllm_b200_mixed.h)."""
+    _fields_ = [(n, _int) for n in ("type", "heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank")] + \
+               [("scale", ctypes.c_float), ("rot_base", ctypes.c_double)] + \
+               [(n, _int) for n in ("channels", "taps", "state", "dt_rank", "blocks")] + \
+               [("decay", ctypes.c_float)] + [(n, _int) for n in ("gate_act", "ff", "ff_act")] + \
+               [("t", _vp * TENSORS_PER_LAYER)]
+
+
+class MixedDesc(ctypes.Structure):
+    """tllm_b200_mixed_desc."""
+    _fields_ = [(n, _int) for n in ("vocab_size", "width", "n_layers", "max_seq_len")] + [("norm_eps", ctypes.c_float)] + \
+               [(n, _int) for n in ("loop_start", "loop_stop", "loop_times", "loop_inject")] + \
+               [("embedding", _vp), ("final_norm", _vp), ("layers", ctypes.POINTER(MixedLayerDesc))]
 
 
 class TllmError(RuntimeError):

@@ -13,11 +13,17 @@
 // every GEMV, src/transformer.cpp:132-136), the position and the token live in device
 // memory too, and greedy sampling runs on the device, so that one decode step can be
 // captured as a CUDA graph and replayed.
+//
+// What does not depend on the kind of model -- the handle, the greedy loop replayed as a CUDA
+// graph, the checks of slots and positions -- is the base class Decoder (decoder.cuh); the C
+// entry points at the end of this file work on any model built on it.
 #include <utility>
 #include <vector>
 
+#include "decoder.cuh"
 #include "layer.cuh"
 #include "tllm_b200_layer.h"
+#include "tllm_b200_mixed.h"
 
 namespace tllm {
 
@@ -37,9 +43,8 @@ struct LayerW {
     const half* ffn_norm = nullptr;
 };
 
-struct Decoder {
+struct LlamaDecoder : Decoder {
     tllm_b200_model_desc d = {};
-    int flags = 0;
     std::vector<LayerW> layers;
     PackedW lm_head;
     // activations (max_seq_len rows where a prefill needs them)
@@ -49,38 +54,16 @@ struct Decoder {
     half *qkv1 = nullptr, *gu1 = nullptr;      // single-token outputs of the concatenated matrices
     half* residual2 = nullptr;                 // second residual vector of the fused single-token step
     bool fused_ok = false;                     // every layer has concatenated q|k|v and gate|up
-    int max_batch = 1;                         // sequences with their own KV cache
     int8_t* xq = nullptr;
     float* xscale = nullptr;
     float* attn_ws = nullptr;
     float* attn_ws2 = nullptr;     // split records of the fused single-token attention
     unsigned* attn_counters = nullptr;
-    // device-side state of the graph-replayed decode loop
-    int* state = nullptr;          // [0] token, [1] position, [2] step
-    int* history = nullptr;        // generated tokens
-    int history_cap = 0;
-    float* am_val = nullptr;
-    int* am_idx = nullptr;
-    unsigned* am_counter = nullptr;
-    cudaStream_t stream = nullptr; // owned, for generate()
-    cudaGraphExec_t step_graph = nullptr;
-    std::vector<void*> owned;
-};
 
-template <typename T>
-int dev_alloc(Decoder* D, T** out, size_t n, bool zero)
-{
-    void* p = nullptr;
-    const cudaError_t e = cudaMalloc(&p, n * sizeof(T));
-    if (e != cudaSuccess) {
-        cudaGetLastError();
-        return fail(TLLM_ERR_LAUNCH, "decoder: cudaMalloc(%zu bytes): %s", n * sizeof(T), cudaGetErrorString(e));
-    }
-    if (zero) cudaMemset(p, 0, n * sizeof(T));
-    D->owned.push_back(p);
-    *out = static_cast<T*>(p);
-    return TLLM_OK;
-}
+    int forward(const int* tokens, int n, int start_pos, const int* pos_dev, int seq, int batch, cudaStream_t s) override;
+    int reset(cudaStream_t s) override;
+    void* logits_row(int seq) override { return logits + (size_t)seq * d.vocab_size; }
+};
 
 int check_weight(const tllm_b200_ternary_weight& w)
 {
@@ -92,20 +75,20 @@ int check_weight(const tllm_b200_ternary_weight& w)
 }
 
 // dst == nullptr: allocate; else repack into dst (part of a concatenated buffer)
-int pack(Decoder* D, const tllm_b200_ternary_weight& w, PackedW* out, cudaStream_t stream, uint8_t* dst = nullptr)
+int pack(LlamaDecoder* D, const tllm_b200_ternary_weight& w, PackedW* out, cudaStream_t stream, uint8_t* dst = nullptr)
 {
     int st = check_weight(w);
     if (st) return st;
     out->rows = w.out_features;
     out->cols = w.in_features;
     if (dst) out->p = dst;
-    else if ((st = dev_alloc(D, &out->p, packed_bytes(w.out_features, w.in_features), false))) return st;
+    else if ((st = D->dev_alloc(&out->p, packed_bytes(w.out_features, w.in_features), false))) return st;
     return weight_prepare(static_cast<const uint32_t*>(w.nonzero_masks), static_cast<const uint32_t*>(w.sign_masks),
                           static_cast<const half*>(w.scales), w.out_features, w.in_features, out->p, stream);
 }
 
 // Packs `count` matrices with the same input width back to back; `all` views them as one.
-int pack_group(Decoder* D, int count, const tllm_b200_ternary_weight* const* w, PackedW* const* out, PackedW* all,
+int pack_group(LlamaDecoder* D, int count, const tllm_b200_ternary_weight* const* w, PackedW* const* out, PackedW* all,
                cudaStream_t stream)
 {
     int st;
@@ -125,7 +108,7 @@ int pack_group(Decoder* D, int count, const tllm_b200_ternary_weight* const* w, 
         return TLLM_OK;
     }
     uint8_t* base = nullptr;
-    if ((st = dev_alloc(D, &base, total, false))) return st;
+    if ((st = D->dev_alloc(&base, total, false))) return st;
     size_t off = 0;
     for (int i = 0; i < count; i++) {
         if ((st = pack(D, *w[i], out[i], stream, base + off))) return st;
@@ -146,7 +129,7 @@ int linear_f16(const PackedW& w, const half* x, half* y, int n_tokens, cudaStrea
     return launch_gemv_packed(w.p, x, y, n_tokens, w.rows, w.cols, stream);
 }
 
-int linear_multi(Decoder* D, int count, const PackedW* const* w, half* const* y, const half* x, bool int8,
+int linear_multi(LlamaDecoder* D, int count, const PackedW* const* w, half* const* y, const half* x, bool int8,
                  int n_tokens, cudaStream_t stream)
 {
     const uint8_t* p[TLLM_MAX_FUSED];
@@ -171,8 +154,9 @@ int linear_multi(Decoder* D, int count, const PackedW* const* w, half* const* y,
 //               token whose position is read from device memory, start_pos ignored);
 //   batch  > 0: one token of each of the sequences 0..batch-1 (n == batch), all at position
 //               start_pos, each against its own KV cache; logits for every sequence.
-int forward(Decoder* D, const int* tokens, int n, int start_pos, const int* pos_dev, int seq, int batch, cudaStream_t s)
+int LlamaDecoder::forward(const int* tokens, int n, int start_pos, const int* pos_dev, int seq, int batch, cudaStream_t s)
 {
+    LlamaDecoder* D = this;
     const tllm_b200_model_desc& c = D->d;
     const int hidden = c.hidden_dim, inter = c.intermediate_dim, qdim = c.n_heads * c.head_dim;
     const bool i8 = (n == 1) && (D->flags & TLLM_DECODER_INT8_DECODE);
@@ -298,7 +282,52 @@ int forward(Decoder* D, const int* tokens, int n, int start_pos, const int* pos_
     return TLLM_OK;
 }
 
+int LlamaDecoder::reset(cudaStream_t s)
+{
+    const size_t bytes = (size_t)d.n_layers * max_batch * d.max_seq_len * d.n_kv_heads * d.head_dim * sizeof(half);
+    cudaMemsetAsync(k_cache, 0, bytes, s);
+    cudaMemsetAsync(v_cache, 0, bytes, s);
+    return check_launch("decoder_reset");
+}
+
 }  // namespace
+
+Decoder::~Decoder()
+{
+    if (step_graph) cudaGraphExecDestroy(step_graph);
+    if (stream) cudaStreamDestroy(stream);
+    for (void* p : owned) cudaFree(p);
+}
+
+int Decoder::dev_alloc_bytes(void** out, size_t bytes, bool zero)
+{
+    void* p = nullptr;
+    const cudaError_t e = cudaMalloc(&p, bytes);
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        return fail(TLLM_ERR_LAUNCH, "decoder: cudaMalloc(%zu bytes): %s", bytes, cudaGetErrorString(e));
+    }
+    if (zero) cudaMemset(p, 0, bytes);
+    owned.push_back(p);
+    *out = p;
+    return TLLM_OK;
+}
+
+int Decoder::init_common(int flags_, int max_batch_, int max_seq_, int vocab_)
+{
+    flags = flags_;
+    max_batch = max_batch_;
+    max_seq = max_seq_;
+    vocab = vocab_;
+    history_cap = max_seq_;
+    if (cudaStreamCreateWithFlags(&stream, cudaStreamNonBlocking) != cudaSuccess)
+        return fail(TLLM_ERR_LAUNCH, "decoder_create: cudaStreamCreate failed");
+    int st;
+    if ((st = dev_alloc(&state, 4, true)) || (st = dev_alloc(&history, (size_t)history_cap, true)) || (st = dev_alloc(&am_val, 64, true)) ||
+        (st = dev_alloc(&am_idx, 64, true)) || (st = dev_alloc(&am_counter, 1, true)))
+        return st;
+    return TLLM_OK;
+}
 
 }  // namespace tllm
 
@@ -306,15 +335,7 @@ using namespace tllm;
 
 extern "C" {
 
-void tllm_b200_decoder_destroy(void* decoder)
-{
-    Decoder* D = static_cast<Decoder*>(decoder);
-    if (!D) return;
-    if (D->step_graph) cudaGraphExecDestroy(D->step_graph);
-    if (D->stream) cudaStreamDestroy(D->stream);
-    for (void* p : D->owned) cudaFree(p);
-    delete D;
-}
+void tllm_b200_decoder_destroy(void* decoder) { delete static_cast<Decoder*>(decoder); }
 
 int tllm_b200_decoder_create(const tllm_b200_model_desc* desc, int flags, void** out)
 {
@@ -338,17 +359,14 @@ int tllm_b200_decoder_create_batched(const tllm_b200_model_desc* desc, int flags
         if (!(hd == 16 || hd == 32 || hd == 64 || hd == 128) || group > 16 || group * (hd / 8) > 256)
             return fail(TLLM_ERR_SHAPE, "decoder_create: head_dim=%d with %d query heads per KV head is not supported", hd, group);
     }
-    Decoder* D = new Decoder();
+    LlamaDecoder* D = new LlamaDecoder();
     D->d = c;
-    D->flags = flags;
-    D->max_batch = max_batch;
     int st = TLLM_OK;
     auto bail = [&](int code) {
-        tllm_b200_decoder_destroy(D);
+        delete D;
         return code;
     };
-    if (cudaStreamCreateWithFlags(&D->stream, cudaStreamNonBlocking) != cudaSuccess)
-        return bail(fail(TLLM_ERR_LAUNCH, "decoder_create: cudaStreamCreate failed"));
+    if ((st = D->init_common(flags, max_batch, c.max_seq_len, c.vocab_size))) return bail(st);
     D->layers.resize(c.n_layers);
     for (int l = 0; l < c.n_layers; l++) {
         const tllm_b200_layer_weights& w = c.layers[l];
@@ -379,37 +397,31 @@ int tllm_b200_decoder_create_batched(const tllm_b200_model_desc* desc, int flags
     if (qdim > maxdim) maxdim = qdim;
     const size_t kv_elems = (size_t)c.n_layers * max_batch * c.max_seq_len * kvdim;
 #define ALLOC(x) do { if ((st = (x)) != TLLM_OK) return bail(st); } while (0)
-    ALLOC(dev_alloc(D, &D->residual, mt * c.hidden_dim, true));
-    ALLOC(dev_alloc(D, &D->hidden, mt * c.hidden_dim, true));
-    ALLOC(dev_alloc(D, &D->hidden2, mt * c.hidden_dim, true));
-    ALLOC(dev_alloc(D, &D->q, mt * qdim, true));
-    ALLOC(dev_alloc(D, &D->k, mt * kvdim, true));
-    ALLOC(dev_alloc(D, &D->v, mt * kvdim, true));
-    ALLOC(dev_alloc(D, &D->attn_out, mt * qdim, true));
-    ALLOC(dev_alloc(D, &D->gate, mt * c.intermediate_dim, true));
-    ALLOC(dev_alloc(D, &D->up, mt * c.intermediate_dim, true));
-    ALLOC(dev_alloc(D, &D->ffn_out, mt * c.hidden_dim, true));
-    ALLOC(dev_alloc(D, &D->logits, (size_t)max_batch * c.vocab_size, true));
-    ALLOC(dev_alloc(D, &D->k_cache, kv_elems, true));
-    ALLOC(dev_alloc(D, &D->v_cache, kv_elems, true));
-    ALLOC(dev_alloc(D, &D->residual2, (size_t)c.hidden_dim, true));
-    ALLOC(dev_alloc(D, &D->qkv1, qdim + 2 * kvdim, true));
-    ALLOC(dev_alloc(D, &D->gu1, (size_t)2 * c.intermediate_dim, true));
-    ALLOC(dev_alloc(D, &D->xq, maxdim, true));
-    ALLOC(dev_alloc(D, &D->xscale, 4, true));
-    ALLOC(dev_alloc(D, &D->attn_ws, attention_workspace_bytes(max_batch, c.n_heads, c.n_kv_heads, c.head_dim, c.max_seq_len) / sizeof(float), true));
-    ALLOC(dev_alloc(D, &D->attn_ws2, attention_decode_workspace_bytes(c.n_heads, c.n_kv_heads, c.head_dim, c.max_seq_len) / sizeof(float), true));
-    ALLOC(dev_alloc(D, &D->attn_counters, (size_t)max_batch * c.n_kv_heads, true));
-    ALLOC(dev_alloc(D, &D->state, 4, true));
-    D->history_cap = c.max_seq_len;
-    ALLOC(dev_alloc(D, &D->history, (size_t)D->history_cap, true));
-    ALLOC(dev_alloc(D, &D->am_val, 64, true));
-    ALLOC(dev_alloc(D, &D->am_idx, 64, true));
-    ALLOC(dev_alloc(D, &D->am_counter, 1, true));
+    ALLOC(D->dev_alloc(&D->residual, mt * c.hidden_dim, true));
+    ALLOC(D->dev_alloc(&D->hidden, mt * c.hidden_dim, true));
+    ALLOC(D->dev_alloc(&D->hidden2, mt * c.hidden_dim, true));
+    ALLOC(D->dev_alloc(&D->q, mt * qdim, true));
+    ALLOC(D->dev_alloc(&D->k, mt * kvdim, true));
+    ALLOC(D->dev_alloc(&D->v, mt * kvdim, true));
+    ALLOC(D->dev_alloc(&D->attn_out, mt * qdim, true));
+    ALLOC(D->dev_alloc(&D->gate, mt * c.intermediate_dim, true));
+    ALLOC(D->dev_alloc(&D->up, mt * c.intermediate_dim, true));
+    ALLOC(D->dev_alloc(&D->ffn_out, mt * c.hidden_dim, true));
+    ALLOC(D->dev_alloc(&D->logits, (size_t)max_batch * c.vocab_size, true));
+    ALLOC(D->dev_alloc(&D->k_cache, kv_elems, true));
+    ALLOC(D->dev_alloc(&D->v_cache, kv_elems, true));
+    ALLOC(D->dev_alloc(&D->residual2, (size_t)c.hidden_dim, true));
+    ALLOC(D->dev_alloc(&D->qkv1, qdim + 2 * kvdim, true));
+    ALLOC(D->dev_alloc(&D->gu1, (size_t)2 * c.intermediate_dim, true));
+    ALLOC(D->dev_alloc(&D->xq, maxdim, true));
+    ALLOC(D->dev_alloc(&D->xscale, 4, true));
+    ALLOC(D->dev_alloc(&D->attn_ws, attention_workspace_bytes(max_batch, c.n_heads, c.n_kv_heads, c.head_dim, c.max_seq_len) / sizeof(float), true));
+    ALLOC(D->dev_alloc(&D->attn_ws2, attention_decode_workspace_bytes(c.n_heads, c.n_kv_heads, c.head_dim, c.max_seq_len) / sizeof(float), true));
+    ALLOC(D->dev_alloc(&D->attn_counters, (size_t)max_batch * c.n_kv_heads, true));
 #undef ALLOC
     if (cudaStreamSynchronize(D->stream) != cudaSuccess)
         return bail(fail(TLLM_ERR_LAUNCH, "decoder_create: %s", cudaGetErrorString(cudaGetLastError())));
-    *out = D;
+    *out = static_cast<Decoder*>(D);
     return TLLM_OK;
 }
 
@@ -417,10 +429,7 @@ int tllm_b200_decoder_reset(void* decoder, void* stream)
 {
     Decoder* D = static_cast<Decoder*>(decoder);
     if (!D) return fail(TLLM_ERR_NULL, "decoder_reset: null decoder");
-    const size_t bytes = (size_t)D->d.n_layers * D->max_batch * D->d.max_seq_len * D->d.n_kv_heads * D->d.head_dim * sizeof(half);
-    cudaMemsetAsync(D->k_cache, 0, bytes, static_cast<cudaStream_t>(stream));
-    cudaMemsetAsync(D->v_cache, 0, bytes, static_cast<cudaStream_t>(stream));
-    return check_launch("decoder_reset");
+    return D->reset(static_cast<cudaStream_t>(stream));
 }
 
 int tllm_b200_decoder_forward(void* decoder, const int* token_ids, int n_tokens, int start_pos, void** logits,
@@ -435,12 +444,13 @@ int tllm_b200_decoder_forward_seq(void* decoder, int seq, const int* token_ids, 
     Decoder* D = static_cast<Decoder*>(decoder);
     if (!D || !token_ids || !logits) return fail(TLLM_ERR_NULL, "decoder_forward: null argument");
     if (seq < 0 || seq >= D->max_batch) return fail(TLLM_ERR_BATCH, "decoder_forward: sequence %d outside 0..%d", seq, D->max_batch - 1);
-    if (n_tokens < 1 || start_pos < 0 || start_pos + n_tokens > D->d.max_seq_len)
-        return fail(TLLM_ERR_SHAPE, "decoder_forward: n_tokens=%d start_pos=%d max_seq_len=%d", n_tokens, start_pos,
-                    D->d.max_seq_len);
-    const int st = forward(D, token_ids, n_tokens, start_pos, nullptr, seq, 0, static_cast<cudaStream_t>(stream));
+    if (n_tokens < 1 || start_pos < 0 || start_pos + n_tokens > D->max_seq)
+        return fail(TLLM_ERR_SHAPE, "decoder_forward: n_tokens=%d start_pos=%d max_seq_len=%d", n_tokens, start_pos, D->max_seq);
+    int st = D->advance(seq, 1, start_pos, n_tokens);
     if (st) return st;
-    *logits = D->logits + (size_t)seq * D->d.vocab_size;
+    st = D->forward(token_ids, n_tokens, start_pos, nullptr, seq, 0, static_cast<cudaStream_t>(stream));
+    if (st) return st;
+    *logits = D->logits_row(seq);
     return TLLM_OK;
 }
 
@@ -449,11 +459,30 @@ int tllm_b200_decoder_forward_batch(void* decoder, const int* token_ids, int bat
     Decoder* D = static_cast<Decoder*>(decoder);
     if (!D || !token_ids || !logits) return fail(TLLM_ERR_NULL, "decoder_forward_batch: null argument");
     if (batch < 1 || batch > D->max_batch) return fail(TLLM_ERR_BATCH, "decoder_forward_batch: batch=%d outside 1..%d", batch, D->max_batch);
-    if (pos < 0 || pos >= D->d.max_seq_len) return fail(TLLM_ERR_SHAPE, "decoder_forward_batch: pos=%d max_seq_len=%d", pos, D->d.max_seq_len);
-    const int st = forward(D, token_ids, batch, pos, nullptr, 0, batch, static_cast<cudaStream_t>(stream));
+    if (pos < 0 || pos >= D->max_seq) return fail(TLLM_ERR_SHAPE, "decoder_forward_batch: pos=%d max_seq_len=%d", pos, D->max_seq);
+    int st = D->advance(0, batch, pos, 1);
     if (st) return st;
-    *logits = D->logits;
+    st = D->forward(token_ids, batch, pos, nullptr, 0, batch, static_cast<cudaStream_t>(stream));
+    if (st) return st;
+    *logits = D->logits_row(0);
     return TLLM_OK;
+}
+
+int tllm_b200_decoder_forward_logits(void* decoder, int seq, const int* token_ids, int n_tokens, int start_pos,
+                                     const int* want_host, int n_want, float* logits, float* taps, void* stream)
+{
+    Decoder* D = static_cast<Decoder*>(decoder);
+    if (!D || !token_ids || (n_want > 0 && (!want_host || !logits))) return fail(TLLM_ERR_NULL, "decoder_forward_logits: null argument");
+    if (seq < 0 || seq >= D->max_batch) return fail(TLLM_ERR_BATCH, "decoder_forward_logits: sequence %d outside 0..%d", seq, D->max_batch - 1);
+    if (n_tokens < 1 || start_pos < 0 || start_pos + n_tokens > D->max_seq || n_want < 0)
+        return fail(TLLM_ERR_SHAPE, "decoder_forward_logits: n_tokens=%d start_pos=%d max_seq_len=%d n_want=%d", n_tokens, start_pos, D->max_seq,
+                    n_want);
+    for (int i = 0; i < n_want; i++)
+        if (want_host[i] < 0 || want_host[i] >= n_tokens)
+            return fail(TLLM_ERR_SHAPE, "decoder_forward_logits: place %d outside 0..%d", want_host[i], n_tokens - 1);
+    const int st = D->advance(seq, 1, start_pos, n_tokens);
+    if (st) return st;
+    return D->forward_logits(token_ids, n_tokens, start_pos, seq, want_host, n_want, logits, taps, static_cast<cudaStream_t>(stream));
 }
 
 int tllm_b200_decoder_generate(void* decoder, int first_token, int start_pos, int n_steps, int* tokens_host,
@@ -461,26 +490,30 @@ int tllm_b200_decoder_generate(void* decoder, int first_token, int start_pos, in
 {
     Decoder* D = static_cast<Decoder*>(decoder);
     if (!D || !tokens_host) return fail(TLLM_ERR_NULL, "decoder_generate: null argument");
-    if (n_steps < 1 || n_steps > D->history_cap || start_pos < 0 || start_pos + n_steps > D->d.max_seq_len)
-        return fail(TLLM_ERR_SHAPE, "decoder_generate: n_steps=%d start_pos=%d max_seq_len=%d", n_steps, start_pos,
-                    D->d.max_seq_len);
+    if (n_steps < 1 || n_steps > D->history_cap || start_pos < 0 || start_pos + n_steps > D->max_seq)
+        return fail(TLLM_ERR_SHAPE, "decoder_generate: n_steps=%d start_pos=%d max_seq_len=%d", n_steps, start_pos, D->max_seq);
     cudaStream_t s = D->stream;
-    int st;
+    int st = D->advance(0, 1, start_pos, n_steps);
+    if (st) return st;
     // work queued by the caller on other streams (a prefill) must be complete
     if (cudaDeviceSynchronize() != cudaSuccess) return fail(TLLM_ERR_LAUNCH, "decoder_generate: %s", cudaGetErrorString(cudaGetLastError()));
     const int init[3] = {first_token, start_pos, 0};
     cudaMemcpyAsync(D->state, init, sizeof(init), cudaMemcpyHostToDevice, s);
     auto step = [&]() -> int {
-        int e = forward(D, D->state, 1, 0, D->state + 1, 0, 0, s);
+        int e = D->forward(D->state, 1, 0, D->state + 1, 0, 0, s);
         if (e) return e;
-        return launch_argmax(D->logits, D->d.vocab_size, D->state, D->history, D->state + 2, D->am_val, D->am_idx,
-                             D->am_counter, D->state + 1, s);
+        if (D->logits_f32)
+            return launch_argmax(static_cast<const float*>(D->logits_row(0)), D->vocab, D->state, D->history, D->state + 2, D->am_val,
+                                 D->am_idx, D->am_counter, D->state + 1, s);
+        return launch_argmax(static_cast<const half*>(D->logits_row(0)), D->vocab, D->state, D->history, D->state + 2, D->am_val,
+                             D->am_idx, D->am_counter, D->state + 1, s);
     };
     if (!D->step_graph) {
         // One eager step first: it performs every lazy set-up (scratch allocation, kernel
         // attributes) outside the capture.  A step rewrites the same cache slot and
-        // buffers when repeated, so the state is put back and the step captured.
-        if ((st = step())) return st;
+        // buffers when repeated, so the state is put back (a model whose sequences carry more
+        // than a cache keeps a copy of it over the step) and the step captured.
+        if ((st = D->save_sequence(0, s)) || (st = step()) || (st = D->restore_sequence(0, s))) return st;
         if (cudaStreamSynchronize(s) != cudaSuccess) return fail(TLLM_ERR_LAUNCH, "decoder_generate: %s", cudaGetErrorString(cudaGetLastError()));
         cudaMemcpyAsync(D->state, init, sizeof(init), cudaMemcpyHostToDevice, s);
         cudaGraph_t g = nullptr;

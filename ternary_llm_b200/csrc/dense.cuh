@@ -1,0 +1,109 @@
+// Dense (not ternary) linear operators of the mixed-layer decoder: BF16 or FP32 weights and
+// activations, FP32 accumulation.  Every matrix is packed at load time so that rows start on
+// 16-byte boundaries: `ld` elements per row, a multiple of 8, padding columns zero.
+#pragma once
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace tllm {
+
+using bf16 = __nv_bfloat16;
+
+// element-wise function applied to (product + bias)
+enum Act { kActNone = 0, kActGeluTanh = 1, kActSilu = 2, kActSoftplus = 3, kActSigmoid = 4 };
+
+// y[m, z, n] = post(sum_k W[z, n, k] x[m, z, k]),  z = 0..batch-1
+template <typename T>
+struct LinearArgs {
+    const T* w = nullptr;        // [batch * w_rows, ldw]
+    int ldw = 0, w_rows = 0;     // rows of one batch entry in w
+    const T* x = nullptr;        // row stride ldx, entry z starts at column z * x_batch
+    int ldx = 0, x_batch = 0;
+    void* y = nullptr;           // T or float, row stride ldy, entry z starts at column z * y_batch
+    int ldy = 0, y_batch = 0;
+    bool y_f32 = false;
+    int M = 0, N = 0, K = 0, batch = 1;   // K: a multiple of 8 (padded)
+    const float* bias = nullptr; // [batch * N], null = none
+    int act = kActNone;
+    // glu: w holds N gate rows followed by N up rows; y = act(gate) * up
+    bool glu = false;
+    const T* gate = nullptr;     // y *= sigmoid(gate[m * gate_ld + z])
+    int gate_ld = 0;
+};
+
+// vectors one after the other against streamed weights; at most 8 vectors per pass
+template <typename T>
+int launch_dense_gemv(const LinearArgs<T>& a, cudaStream_t stream);
+int launch_dense_gemm_tcgen05(const LinearArgs<bf16>& a, cudaStream_t stream);
+int launch_dense_gemm_f32(const LinearArgs<float>& a, cudaStream_t stream);
+// dispatch by the number of rows
+int linear(const LinearArgs<bf16>& a, cudaStream_t stream);
+int linear(const LinearArgs<float>& a, cudaStream_t stream);
+
+// ---- load-time packing ---------------------------------------------------------------
+// How a BF16 matrix is laid out with padding: row groups of `r` rows, `rs` source rows apart,
+// become groups `rp` rows apart; column groups of `c` columns become `cp` wide.  dst row
+// (i * rp + a), column (j * cp + b) = fn(src row (i * rs + a), column (j * c + b)); everything
+// else of dst stays as it is (zero).  transpose: each row group is transposed (gc must be 1):
+// dst row (i * rp + b), column a.
+enum PackFn { kPackCopy = 0, kPackNegExpLog2e = 1, kPackSoftplus = 2 };   // applied once at load, in double
+struct PackSpec {
+    int gr = 1, r = 1, rs = 1, rp = 1;
+    int gc = 1, c = 1, cp = 1;
+    bool transpose = false;
+    int fn = kPackCopy;
+};
+template <typename D>
+int launch_pack(const void* src, const PackSpec& p, D* dst, int ld, cudaStream_t stream);
+
+// ---- small device helpers --------------------------------------------------------------
+template <typename T> __device__ __forceinline__ float to_f(T v);
+template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f<bf16>(bf16 v) { return __bfloat162float(v); }
+template <> __device__ __forceinline__ float to_f<half>(half v) { return __half2float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+__device__ __forceinline__ float apply_act(int act, float z)
+{
+    switch (act) {
+        case kActGeluTanh: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+        case kActSilu: return z * sigmoid_f(z);
+        case kActSoftplus: return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+        case kActSigmoid: return sigmoid_f(z);
+        default: return z;
+    }
+}
+
+// 16 bytes of T as floats
+template <typename T> struct Vec16;
+template <> struct Vec16<bf16> {
+    static constexpr int n = 8;
+    static __device__ __forceinline__ void unpack(const uint4& v, float* f)
+    {
+        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            f[2 * i] = __uint_as_float(w[i] << 16);
+            f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+        }
+    }
+};
+template <> struct Vec16<float> {
+    static constexpr int n = 4;
+    static __device__ __forceinline__ void unpack(const uint4& v, float* f)
+    {
+        f[0] = __uint_as_float(v.x);
+        f[1] = __uint_as_float(v.y);
+        f[2] = __uint_as_float(v.z);
+        f[3] = __uint_as_float(v.w);
+    }
+};
+
+inline int pad8(int n) { return (n + 7) / 8 * 8; }
+
+}  // namespace tllm

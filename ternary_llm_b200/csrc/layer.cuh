@@ -28,6 +28,8 @@ int launch_fp16_gemm(const half* A, const half* B, half* C, int M, int N, int K,
 // null, *pos is advanced by one together with the token (the decode loop's cache position).
 int launch_argmax(const half* logits, int n, int* out, int* history, int* step, float* part_val, int* part_idx,
                   unsigned* counter, int* pos, cudaStream_t stream);
+int launch_argmax(const float* logits, int n, int* out, int* history, int* step, float* part_val, int* part_idx,
+                  unsigned* counter, int* pos, cudaStream_t stream);
 
 size_t attention_workspace_bytes(int batch, int n_heads, int n_kv_heads, int head_dim, int kv_len_max);
 // kv_len_dev: decode only, kv_len = kv_len + *kv_len_dev.  ws / counters: decode split scratch or null.

@@ -636,8 +636,12 @@ int launch_fp16_gemm(const half* A, const half* B, half* C, int M, int N, int K,
 constexpr int kArgmaxCtas = 64;
 constexpr int kArgmaxThreads = 256;
 
+__device__ __forceinline__ float logit_f(half v) { return __half2float(v); }
+__device__ __forceinline__ float logit_f(float v) { return v; }
+
+template <typename T>
 __global__ void __launch_bounds__(kArgmaxThreads)
-argmax_kernel(const half* __restrict__ logits, int n, int* __restrict__ out, int* __restrict__ history,
+argmax_kernel(const T* __restrict__ logits, int n, int* __restrict__ out, int* __restrict__ history,
               int* __restrict__ step, float* __restrict__ part_val, int* __restrict__ part_idx,
               unsigned* __restrict__ counter, int* __restrict__ pos)
 {
@@ -649,7 +653,7 @@ argmax_kernel(const half* __restrict__ logits, int n, int* __restrict__ out, int
     float best = -FLT_MAX;
     int bi = 0x7fffffff;
     for (int i = blockIdx.x * kArgmaxThreads + threadIdx.x; i < n; i += kArgmaxCtas * kArgmaxThreads) {
-        const float v = __half2float(logits[i]);
+        const float v = logit_f(logits[i]);
         if (v > best || (v == best && i < bi)) {
             best = v;
             bi = i;
@@ -712,9 +716,15 @@ argmax_kernel(const half* __restrict__ logits, int n, int* __restrict__ out, int
 int launch_argmax(const half* logits, int n, int* out, int* history, int* step, float* part_val, int* part_idx,
                   unsigned* counter, int* pos, cudaStream_t stream)
 {
-    return launch_pdl("argmax", argmax_kernel, dim3(kArgmaxCtas), dim3(kArgmaxThreads), 0, stream, logits, n, out,
+    return launch_pdl("argmax", argmax_kernel<half>, dim3(kArgmaxCtas), dim3(kArgmaxThreads), 0, stream, logits, n, out,
+                      history, step, part_val, part_idx, counter, pos);
+}
+
+int launch_argmax(const float* logits, int n, int* out, int* history, int* step, float* part_val, int* part_idx,
+                  unsigned* counter, int* pos, cudaStream_t stream)
+{
+    return launch_pdl("argmax", argmax_kernel<float>, dim3(kArgmaxCtas), dim3(kArgmaxThreads), 0, stream, logits, n, out,
                       history, step, part_val, part_idx, counter, pos);
 }
 
 }  // namespace tllm
-

@@ -3,6 +3,9 @@ library's decoder (include/tllm_b200_layer.h): construct from a model, forward(t
 start_pos) -> logits of the last token, reset(), and generate() for the greedy decode loop
 replayed as a CUDA graph.  The model's tensors are uploaded with torch; every operator runs
 in libtllm_b200.so.
+
+The same class serves every design of the registry (models.py): the LLaMA design on ternary
+weights (.tllm) and models made of mixer layers (mixed.py).
 """
 from __future__ import annotations
 
@@ -11,8 +14,9 @@ import ctypes
 import numpy as np
 import torch
 
-from . import _lib
-from .tllm_format import PROJ_NAMES, TernaryTensor, TllmFile, read_tllm
+from . import _lib, models
+from .mixed import MixedModel
+from .tllm_format import PROJ_NAMES, TernaryTensor, TllmFile
 
 
 class _DevArray:
@@ -23,15 +27,58 @@ class _DevArray:
 
 
 class Decoder:
-    def __init__(self, model, device=None, int8_decode: bool = True, max_batch: int = 1):
-        """max_batch > 1: room for that many independent sequences, each with its own KV cache
-        (forward_seq for one of them, forward_batch for a lock-step decode of several)."""
+    def __init__(self, model, device=None, int8_decode: bool = True, max_batch: int = 1, max_seq_len: int | None = None,
+                 dtype: str = "bfloat16"):
+        """model: a model object (tllm_format.TllmFile, mixed.MixedModel) or the path of one.
+        max_batch > 1: room for that many independent sequences, each with its own cache and
+        state (forward_seq for one of them, forward_batch for a lock-step decode of several).
+        int8_decode: ternary models only.  max_seq_len, dtype ("bfloat16" or "float32"): mixer
+        models only (a .tllm file states its own length; its activations are FP16)."""
         if isinstance(model, str):
-            model = read_tllm(model)
-        assert isinstance(model, TllmFile)
-        self.config = cfg = model.config
+            model = models.load(model)
         self.device = torch.device("cuda", torch.cuda.current_device()) if device is None else torch.device(device)
+        self.max_batch = max_batch
+        self._h = None
         self._keep = []          # tensors the decoder keeps pointers to (embedding, norms, FP16 lm_head)
+        if isinstance(model, TllmFile):
+            self._create_llama(model, int8_decode)
+        elif isinstance(model, MixedModel):
+            self._create_mixed(model, 4096 if max_seq_len is None else max_seq_len, dtype)
+        else:
+            raise TypeError(f"Decoder takes a TllmFile, a MixedModel or a path, not {type(model).__name__}")
+
+    def _create_mixed(self, model: MixedModel, max_seq_len: int, dtype: str) -> None:
+        if dtype not in ("bfloat16", "float32"):
+            raise ValueError(f"dtype {dtype!r}: bfloat16 or float32")
+        staging = []             # source tensors, needed only until create() has packed them
+
+        def up(a):
+            if isinstance(a, torch.Tensor):
+                t = a.to(self.device).contiguous()
+                if t.dtype != torch.bfloat16:
+                    raise TypeError(f"weights must be bfloat16, got {t.dtype}")
+            else:
+                a = np.array(a)
+                if a.dtype != np.uint16:
+                    raise TypeError(f"weights must be BF16 bit patterns (uint16), got {a.dtype}")
+                t = torch.from_numpy(a.view(np.int16)).to(self.device)
+            staging.append(t)
+            return t.data_ptr()
+
+        handle = ctypes.c_void_p()
+        with torch.cuda.device(self.device):
+            d = model.fill_desc(up, max_seq_len)
+            torch.cuda.synchronize()
+            _lib.check(_lib.lib().tllm_b200_mixed_decoder_create(ctypes.byref(d), 2 if dtype == "float32" else 0, self.max_batch,
+                                                                 ctypes.byref(handle)))
+        self._h = handle
+        self.config = model
+        self.vocab_size, self.max_seq_len, self.width = model.vocab_size, max_seq_len, model.width
+        self._logits = ("<f4", torch.float32)
+        del staging
+
+    def _create_llama(self, model: TllmFile, int8_decode: bool) -> None:
+        self.config = cfg = model.config
         staging = []             # ternary source arrays, needed only until create() has repacked them
 
         def up(a, keep=True):
@@ -73,9 +120,10 @@ class Decoder:
         with torch.cuda.device(self.device):
             torch.cuda.synchronize()
             _lib.check(_lib.lib().tllm_b200_decoder_create_batched(ctypes.byref(d), 1 if int8_decode else 0,
-                                                                   max_batch, ctypes.byref(handle)))
+                                                                   self.max_batch, ctypes.byref(handle)))
         self._h = handle
-        self.max_batch = max_batch
+        self.vocab_size, self.max_seq_len, self.width = cfg.vocab_size, cfg.max_seq_len, cfg.hidden_dim
+        self._logits = ("<f2", torch.float16)
         del staging
 
     def reset(self) -> None:
@@ -87,8 +135,9 @@ class Decoder:
             raise TypeError("token_ids must be a contiguous int32 CUDA tensor")
 
     def forward(self, token_ids, start_pos: int) -> torch.Tensor:
-        """token_ids: int32 CUDA tensor [n]; returns the FP16 logits of the last token
-        (a view of the decoder's buffer, overwritten by the next call)."""
+        """token_ids: int32 CUDA tensor [n]; returns the logits of the last token, FP16 for a
+        ternary model, FP32 for a mixer model (a view of the decoder's buffer, overwritten by the
+        next call)."""
         return self.forward_seq(0, token_ids, start_pos)
 
     def forward_seq(self, seq: int, token_ids, start_pos: int) -> torch.Tensor:
@@ -98,18 +147,33 @@ class Decoder:
         _lib.check(_lib.lib().tllm_b200_decoder_forward_seq(self._h, seq, token_ids.data_ptr(), token_ids.numel(),
                                                             start_pos, ctypes.byref(out),
                                                             torch.cuda.current_stream().cuda_stream))
-        return torch.as_tensor(_DevArray(out.value, self.config.vocab_size, "<f2"), device=self.device)
+        return torch.as_tensor(_DevArray(out.value, self.vocab_size, self._logits[0]), device=self.device)
 
     def forward_batch(self, token_ids, pos: int) -> torch.Tensor:
         """One lock-step decode step: token_ids[b] is the next token of sequence b, all at cache
-        position pos.  Returns FP16 logits [batch, vocab] (a view of the decoder's buffer)."""
+        position pos.  Returns logits [batch, vocab] (a view of the decoder's buffer)."""
         self._check_tokens(token_ids)
         b = token_ids.numel()
         out = ctypes.c_void_p()
         _lib.check(_lib.lib().tllm_b200_decoder_forward_batch(self._h, token_ids.data_ptr(), b, pos, ctypes.byref(out),
                                                               torch.cuda.current_stream().cuda_stream))
-        flat = torch.as_tensor(_DevArray(out.value, b * self.config.vocab_size, "<f2"), device=self.device)
-        return flat.view(b, self.config.vocab_size)
+        flat = torch.as_tensor(_DevArray(out.value, b * self.vocab_size, self._logits[0]), device=self.device)
+        return flat.view(b, self.vocab_size)
+
+    def forward_logits(self, seq: int, token_ids, start_pos: int, want, taps: bool = False):
+        """Runs token_ids of sequence `seq` from start_pos on and returns FP32 logits
+        [len(want), vocab] of the tokens at the places `want`; with taps also the residual stream
+        after every layer run, [runs, tokens, width].  Mixer models only."""
+        self._check_tokens(token_ids)
+        n = token_ids.numel()
+        places = (ctypes.c_int * max(1, len(want)))(*want)
+        out = torch.empty(len(want), self.vocab_size, dtype=torch.float32, device=self.device)
+        runs = _lib.lib().tllm_b200_mixed_decoder_runs(self._h)
+        res = torch.empty(runs, n, self.width, dtype=torch.float32, device=self.device) if taps else None
+        _lib.check(_lib.lib().tllm_b200_decoder_forward_logits(
+            self._h, seq, token_ids.data_ptr(), n, start_pos, places, len(want), out.data_ptr() if len(want) else None,
+            res.data_ptr() if taps else None, torch.cuda.current_stream().cuda_stream))
+        return (out, res) if taps else out
 
     def generate(self, first_token: int, start_pos: int, n_steps: int):
         """Greedy continuation: returns (tokens [n_steps], ms per step measured on the device)."""
