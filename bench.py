@@ -1016,9 +1016,77 @@ def decode_sample(torch, tl, dev, n_prompt=512, n_steps=128):
     return out
 
 
+# Models of mixer layers (Petulix) at the sizes of the ternary models they are put beside: the
+# same width, feed-forward width, layer count and vocabulary; every layer has a feed-forward.
+MIXED_SIZES = {
+    "1b": dict(width=2048, ff=8192, n_layers=16, vocab=128256, heads=16, inner=4096, dt_rank=128, lru=2048, lru_blocks=16),
+    "8b": dict(width=4096, ff=14336, n_layers=32, vocab=128256, heads=32, inner=8192, dt_rank=256, lru=4096, lru_blocks=16),
+}
+MIXED_SIZES["1b-3l"] = dict(MIXED_SIZES["1b"], n_layers=3, vocab=32000)      # one layer of each kind, for profilers
+
+
+def mixed_config(size):
+    z = MIXED_SIZES[size]
+    kinds = [
+        {"type": "latent_attention", "mixer": {"heads": z["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512,
+                                               "rot": {"base": 10000.0, "dims": 64}, "scale": 192 ** -0.5}},
+        {"type": "mamba1", "mixer": {"inner": z["inner"], "state": 16, "dt_rank": z["dt_rank"], "conv": 4}},
+        {"type": "rglru", "mixer": {"width": z["lru"], "blocks": z["lru_blocks"], "conv": 4}},
+    ]
+    layers = [dict(kinds[i % 3], mlp={"kind": "dense", "ff": z["ff"]}) for i in range(z["n_layers"])]
+    return {"architecture": "Petulix", "vocab": z["vocab"], "width": z["width"], "layers": layers, "norm": {"eps": 1e-5},
+            "loop": {"start": 0, "stop": 0, "times": 1}}
+
+
+def mixed_case(torch, tl, dev, size, n_prompt, n_steps, eager):
+    """mixed:SIZE[:prompt[:steps[:eager]]] -- prefill and greedy decode of a model of mixer layers
+    with seeded random BF16 weights (1b, 8b; 1b-3l with `eager` for profilers)."""
+    from ternary_llm_b200 import mixed
+    cfg = mixed_config(size)
+    shapes = mixed.Petulix.tensor_shapes(cfg)
+    tensors = mixed.random_tensors(shapes, 2026, dev)
+    # every matrix is read once per token (the embedding table as output head)
+    weight_bytes = 2 * sum(int(np.prod(s)) for s in shapes.values())
+    dec = tl.Decoder(mixed.Petulix.from_config(cfg, tensors), max_seq_len=n_prompt + n_steps + 8)
+    del tensors
+    prompt = torch.from_numpy(np.random.default_rng(0).integers(0, cfg["vocab"], n_prompt).astype(np.int32)).to(dev)
+    first = int(dec.forward(prompt, 0).argmax().item())
+    info = {"weight_bytes_per_token": weight_bytes, "prompt": n_prompt}
+    if eager:
+        tok = first
+        for i in range(n_steps):
+            tok = int(dec.forward(torch.tensor([tok], dtype=torch.int32, device=dev), n_prompt + i).argmax().item())
+    else:
+        ms = []
+        for _ in range(5):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            dec.forward(prompt, 0)
+            e1.record()
+            torch.cuda.synchronize()
+            ms.append(e0.elapsed_time(e1))
+        dec.generate(first, n_prompt, 4)
+        dec.forward(prompt, 0)
+        torch.cuda.synchronize()
+        with ClockSampler(0) as clk:
+            _, step_ms = dec.generate(first, n_prompt, n_steps)
+        peak, src = measured_peak_hbm()
+        gbs = weight_bytes / (step_ms * 1e-3) / 1e9
+        pre = statistics.median(ms)
+        # two operations per weight and token (the head runs for the last token only)
+        flops = 2.0 * n_prompt * (weight_bytes / 2 - cfg["vocab"] * cfg["width"])
+        info.update({"prefill_ms": pre, "prefill_tok_per_s": n_prompt / pre * 1e3, "prefill_tflops_of_weights": flops / pre / 1e9,
+                     "decode_ms_per_token": step_ms, "tok_per_s": 1e3 / step_ms, "hbm_gbs": gbs, f"hbm_fraction_of_{src}": gbs / peak,
+                     "clocks": clk.summary()})
+    tl.check_device_errors()
+    dec.close()
+    return info
+
+
 def run_case(args):
     """A small single-kernel case for profilers: `gemv:NxK[:copies]`, `gemv_int8:NxK[:copies]`
-    `gemm:MxNxK`, or `decode:ARCH[:prompt[:steps[:eager]]]` (the decoder on a random model).
+    `gemm:MxNxK`, or `decode:ARCH[:prompt[:steps[:eager]]]` (the decoder on a random model), or
+    `mixed:SIZE[:prompt[:steps[:eager]]]` (mixed_case).
     Distinct matrices are cycled so that the weights come from HBM."""
     import torch
 
@@ -1068,6 +1136,11 @@ def run_case(args):
         c = torch.zeros(m, n, device=dev, dtype=torch.float16)
         for _ in range(4):
             tl.ternary_gemm_packed(a, w, c, m)
+    elif kind == "mixed":
+        info = mixed_case(torch, tl, dev, dims, int(rest[0]) if rest else 2048, int(rest[1]) if len(rest) > 1 else 64,
+                          len(rest) > 2 and rest[2] == "eager")
+        print(json.dumps({"case": args.case, "status": "ok", **info}))
+        return
     elif kind == "decode_batch":
         # decode_batch:1b|1b-4l:B[:prompt[:steps]] -- B sequences decoded in lock step (graph-replayed step)
         from ternary_llm_b200 import tllm_format as tf
@@ -1112,6 +1185,8 @@ def run_case(args):
         # the benchmark's 1B architecture (`1b`, 16 layers) or a 4-layer cut of it (`1b-4l`)
         from ternary_llm_b200 import tllm_format as tf
         arch = dict(DECODE_ARCH_1B)
+        if len(rest) > 0:       # a longer prompt needs a longer cache
+            arch["max_seq_len"] = max(arch["max_seq_len"], int(rest[0]) + (int(rest[1]) if len(rest) > 1 else 128) + 8)
         if dims == "1b-4l":
             arch.update(n_layers=4, vocab_size=32000)
         elif dims == "8b":      # LLaMA-3-8B architecture (the benchmark's GEMV shapes), weights drawn on the device

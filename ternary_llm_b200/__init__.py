@@ -14,10 +14,10 @@ from .ops import (GROUP_SIZE, MAX_BATCH, FusedAllReduce, PreparedWeight, ternary
                   ternary_gemv_int8_packed, ternary_gemv_packed, ternary_gemv_packed_multi,
                   ternary_gemv_packed_multi_norm, prepare_group)
 
-from . import layer_ops  # noqa: F401,E402
+from . import layer_ops, mixed_ops  # noqa: F401,E402
 from . import models  # noqa: F401,E402
 from .decoder import Decoder  # noqa: F401,E402
 
-__all__ = ["layer_ops", "models", "Decoder", "prepare_group", "pack", "lib", "TllmError", "LIB_PATH", "GROUP_SIZE", "MAX_BATCH", "ternary_gemv",
+__all__ = ["layer_ops", "mixed_ops", "models", "Decoder", "prepare_group", "pack", "lib", "TllmError", "LIB_PATH", "GROUP_SIZE", "MAX_BATCH", "ternary_gemv",
            "ternary_gemv_batched", "ternary_gemv_int8", "quantize_absmax_int8", "ternary_gemm",
            "PreparedWeight", "FusedAllReduce", "ternary_gemv_packed_allreduce", "ternary_gemm_packed", "check_device_errors", "packed_bytes", "ternary_gemv_packed", "ternary_gemv_int8_packed", "ternary_gemv_packed_multi", "ternary_gemv_packed_multi_norm"]

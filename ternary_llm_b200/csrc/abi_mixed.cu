@@ -63,6 +63,18 @@ int conv(const void* x, const float* w, const float* bias, void* state, void* y,
     return launch_causal_conv<T>(a, s);
 }
 
+// Scratch of a stand-alone call: allocated in stream order for its size and freed behind it.
+template <typename F>
+int with_records(size_t floats, float** rec, cudaStream_t s, F&& launch)
+{
+    if (!floats) return launch();
+    if (cudaMallocAsync(reinterpret_cast<void**>(rec), floats * sizeof(float), s) != cudaSuccess)
+        return fail(TLLM_ERR_LAUNCH, "operator scratch: %s", cudaGetErrorString(cudaGetLastError()));
+    const int st = launch();
+    cudaFreeAsync(*rec, s);
+    return st;
+}
+
 template <typename T>
 int sel_scan(const void* x, const float* dt, const void* bc, const void* z, const float* a2, const float* d, float* state, void* y,
              int channels, int states, StepGeo g, cudaStream_t s)
@@ -83,7 +95,7 @@ int sel_scan(const void* x, const float* dt, const void* bc, const void* z, cons
     a.channels = channels;
     a.states = states;
     a.g = g;
-    return launch_selective_scan<T>(a, s);
+    return with_records(scan_record_floats(g.n_seq, g.seq_len, channels, states), &a.rec, s, [&] { return launch_selective_scan<T>(a, s); });
 }
 
 template <typename T>
@@ -104,7 +116,7 @@ int gate_scan(const void* u, const float* gates, const float* soft_lam, const vo
     a.channels = channels;
     a.block = channels / blocks;
     a.g = g;
-    return launch_gated_scan<T>(a, s);
+    return with_records(scan_record_floats(g.n_seq, g.seq_len, channels, 1), &a.rec, s, [&] { return launch_gated_scan<T>(a, s); });
 }
 
 template <typename T>
@@ -125,16 +137,12 @@ LatentArgs<T> latent(const void* cache, const float* sink, int heads, int dim, i
     return a;
 }
 
-// Scratch of the stand-alone absorbed attention: allocated for the call's size, freed with it.
 int latent_op(const LatentArgs<bf16>& a, const void* q, void* o, cudaStream_t s)
 {
     float* ws = nullptr;
-    const size_t n = latent_workspace_floats(a.g.rows(), a.heads, a.rank);
-    if (cudaMallocAsync(reinterpret_cast<void**>(&ws), n * sizeof(float), s) != cudaSuccess)
-        return fail(TLLM_ERR_LAUNCH, "latent_attention: %s", cudaGetErrorString(cudaGetLastError()));
-    const int st = launch_latent_absorbed<bf16>(a, static_cast<const bf16*>(q), static_cast<bf16*>(o), ws, s);
-    cudaFreeAsync(ws, s);
-    return st;
+    return with_records(latent_workspace_floats(a.g.rows(), a.heads, a.rank), &ws, s, [&] {
+        return launch_latent_absorbed<bf16>(a, static_cast<const bf16*>(q), static_cast<bf16*>(o), ws, s);
+    });
 }
 }  // namespace
 

@@ -32,9 +32,57 @@ struct LinearArgs {
     int gate_ld = 0;
 };
 
+// ---- what a GEMV of a decode step takes over from its neighbours --------------------------
+// Staging: x = norm(x_in + post-normed y (+ extra)) computed by every CTA instead of a launch of
+// its own (the step of the residual chain in mixers.cuh); the sum goes to x_out, a different
+// buffer than x_in, because every CTA reads the old one while the first writes.
+struct GemvNorm {
+    const float* y = nullptr;       // [M, K]; null: no norm staging, the vectors come from x
+    const float* w_post = nullptr;  // null: plain add
+    const float* x_in = nullptr;
+    float* x_out = nullptr;
+    const float* extra = nullptr;
+    const float* w_next = nullptr;
+    int width = 0;                  // true width (K is padded)
+    float eps = 0.f;
+};
+// Tails, for one new token per sequence (vector m belongs to slot first_slot + m):
+//   kTailConv: output rows [lo, hi) are the inputs of a causal convolution with carried inputs;
+//     act(convolution) goes to out, the carried inputs move on, y is not written for these rows;
+//   kTailGate: rows n and N + n of entry z are the two gates of channel z * N + n of a
+//     real-gated recurrence whose input is x itself: state update and out = S act(y).
+enum Tail { kTailNone = 0, kTailConv = 1, kTailGate = 2 };
+template <typename T>
+struct GemvTail {
+    int kind = kTailNone;
+    int lo = 0, hi = 0, taps = 0, act = kActNone;
+    const float* w = nullptr;         // convolution [hi - lo, taps]
+    const float* bias = nullptr;      // convolution bias or null
+    T* carried = nullptr;             // [slot][taps - 1][hi - lo]
+    const float* soft_lam = nullptr;  // recurrence
+    float decay = 0.f;
+    const T* y = nullptr;
+    int ld_y = 0;
+    float* state = nullptr;           // [slot][channels]
+    size_t slot_stride = 0;
+    int first_slot = 0, start_pos = 0;
+    const int* pos_dev = nullptr;
+    T* out = nullptr;                 // [M, ld_out]
+    int ld_out = 0;
+};
+
 // vectors one after the other against streamed weights; at most 8 vectors per pass
 template <typename T>
 int launch_dense_gemv(const LinearArgs<T>& a, cudaStream_t stream);
+// at most 8 vectors
+template <typename T>
+int launch_dense_gemv_fused(const LinearArgs<T>& a, const GemvNorm& norm, const GemvTail<T>& tail, cudaStream_t stream);
+// the tails need this many lanes per row
+template <typename T>
+bool gemv_tail_fits(int k, int taps);
+// norm staging of up to 8 rows of this width
+template <typename T>
+bool gemv_norm_fits(int k);
 int launch_dense_gemm_tcgen05(const LinearArgs<bf16>& a, cudaStream_t stream);
 int launch_dense_gemm_f32(const LinearArgs<float>& a, cudaStream_t stream);
 // dispatch by the number of rows
@@ -66,17 +114,57 @@ template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 
-__device__ __forceinline__ float apply_act(int act, float z)
+// z * sigmoid(2u) with u = sqrt(2/pi) (z + 0.044715 z^3): the same number as 0.5 z (1 + tanh(u))
+__device__ __forceinline__ float gelu_tanh_f(float z) { return z * sigmoid_f(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+// 2^x for x <= 0, flushed to zero below the normal range
+__device__ __forceinline__ float exp2_neg(float x)
+{
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+
+// 1 - e^t for t <= 0: the power series near zero (no cancellation when the decay is close to
+// one), the plain difference elsewhere
+__device__ __forceinline__ float one_minus_exp(float t, float e)
+{
+    const float p = -t * (1.f + t * (1.f / 2) * (1.f + t * (1.f / 3) * (1.f + t * (1.f / 4) * (1.f + t * (1.f / 5) * (1.f + t * (1.f / 6))))));
+    return t > -0.25f ? p : 1.f - e;
+}
+
+// the switch stays outside the loop over the elements
+template <int N>
+__device__ __forceinline__ void apply_act_n(int act, float (&v)[N])
 {
     switch (act) {
-        case kActGeluTanh: return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-        case kActSilu: return z * sigmoid_f(z);
-        case kActSoftplus: return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-        case kActSigmoid: return sigmoid_f(z);
-        default: return z;
+        case kActGeluTanh:
+#pragma unroll
+            for (int i = 0; i < N; i++) v[i] = gelu_tanh_f(v[i]);
+            break;
+        case kActSilu:
+#pragma unroll
+            for (int i = 0; i < N; i++) v[i] = v[i] * sigmoid_f(v[i]);
+            break;
+        case kActSoftplus:
+#pragma unroll
+            for (int i = 0; i < N; i++) v[i] = softplus_f(v[i]);
+            break;
+        case kActSigmoid:
+#pragma unroll
+            for (int i = 0; i < N; i++) v[i] = sigmoid_f(v[i]);
+            break;
+        default: break;
     }
+}
+__device__ __forceinline__ float apply_act(int act, float z)
+{
+    float v[1] = {z};
+    apply_act_n<1>(act, v);
+    return v[0];
 }
 
 // 16 bytes of T as floats

@@ -2,15 +2,17 @@
 // with FP32 accumulation in tensor memory and the element-wise tail of the operator (bias,
 // activation, gated product, per-head gate) in the epilogue.
 //
-// One CTA computes 128 tokens x TN features.  Both operands are K-major tiles of 64 columns
-// brought by TMA with the 128-byte swizzle (out-of-range rows and columns read as zero, so no
-// size needs to divide a tile); one thread issues tcgen05.mma kind::f16 (M = 128, N = TN,
-// K = 16); a TMEM lane is a token, so an epilogue thread owns a token and writes runs of
-// adjacent features.  A gated feed-forward loads TN/2 gate rows and the TN/2 up rows with the
-// same numbers into one tile, so both factors of a product meet in the same thread.
-// blockIdx.z walks the entries of a block-diagonal or per-head product (column offset in X and
-// Y, row offset in W).  All mbarrier waits are bounded; a wait that gives up sets the device
-// error flag, the roles wait for their own copies and MMAs (bounded again), and TMEM is freed.
+// A tile is 128 tokens x TN features.  One persistent CTA per SM walks tiles with three roles
+// that run ahead of one another: a TMA producer (K-major tiles of 64 columns, 128-byte swizzle;
+// out-of-range rows and columns read as zero, so no size needs to divide a tile), one thread
+// that issues tcgen05.mma kind::f16 (M = 128, N = TN, K = 16) into one of two accumulators in
+// tensor memory, and eight epilogue warps that empty the other one: a TMEM lane is a token, the
+// rows pass through a small shared-memory tile per warp so that global stores are whole lines.
+// A gated feed-forward loads TN/2 gate rows and the TN/2 up rows with the same numbers into one
+// tile, so both factors of a product meet in the same thread.  Tiles also run over the entries
+// of a block-diagonal or per-head product (column offset in X and Y, row offset in W).  All
+// mbarrier waits are bounded; a wait that gives up sets the device error flag, the roles wait
+// for their own copies and MMAs (bounded again), and TMEM is freed.
 #include <mutex>
 
 #include "dense.cuh"
@@ -25,16 +27,19 @@ using namespace gemm;
 
 constexpr int kTok = 128;            // tokens per CTA (MMA M, TMEM lanes)
 constexpr int kBlkK = 64;            // K per stage: one 128-byte swizzled row
-constexpr int kThr = 256;
+constexpr int kEpiWarps = 8;         // two per quarter of the TMEM lanes, taking turns at 32 columns
+constexpr int kThr = 128 + 32 * kEpiWarps;
+
+constexpr int kStageLd = 20;         // words per row of an epilogue warp's tile: 16 of data (16 FP32 or 32 BF16 columns)
 
 template <int TN>
 struct DCfg {
     static constexpr int kXBytes = kTok * kBlkK * 2;
     static constexpr int kWBytes = TN * kBlkK * 2;
     static constexpr int kStage = kXBytes + kWBytes;
-    static constexpr int kStages = (TN == 256) ? 4 : (TN == 128) ? 3 : 4;
-    static constexpr int kPerSm = (TN == 256) ? 1 : 2;
-    static constexpr size_t kSmem = (size_t)kStages * kStage + 1024;
+    static constexpr int kStages = (TN == 256) ? 4 : (TN == 128) ? 6 : 8;
+    static constexpr int kEpiBytes = kEpiWarps * 32 * kStageLd * 4;
+    static constexpr size_t kSmem = (size_t)kStages * kStage + kEpiBytes + 1024;
 };
 
 struct DenseEpi {
@@ -43,7 +48,8 @@ struct DenseEpi {
     const bf16* gate;
     int ldy, y_batch, gate_ld;
     int M, N, K, x_batch, w_rows;
-    int act, glu, y_f32, vec;
+    int mt, nt, tiles;             // tiles along the tokens, along the features, in all
+    int act, glu, y_f32, vec, bias_vec;
     int* err;
 };
 
@@ -62,39 +68,48 @@ __device__ __forceinline__ void mma_ss(uint32_t d, uint64_t a, uint64_t b, uint3
 }
 
 template <int TN>
-__global__ void __launch_bounds__(kThr, DCfg<TN>::kPerSm)
+__global__ void __launch_bounds__(kThr, 1)
 dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w, const DenseEpi a)
 {
     constexpr int kStages = DCfg<TN>::kStages, kStage = DCfg<TN>::kStage, kXBytes = DCfg<TN>::kXBytes;
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-    __shared__ __align__(8) uint64_t bars[2 * kStages + 1];
+    __shared__ __align__(8) uint64_t bars[2 * kStages + 4];
     __shared__ uint32_t tmem_slot;
     __shared__ int abort_flag;
     pdl_launch_dependents();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int m0 = blockIdx.x * kTok, z = blockIdx.z;
-    const int outs = a.glu ? TN / 2 : TN;              // output features of this tile
-    const int n0 = blockIdx.y * outs;
+    const int outs = a.glu ? TN / 2 : TN;              // output features of a tile
     const int nk = (a.K + kBlkK - 1) / kBlkK;
     const uint32_t bar0 = smem_u32(bars);
     auto full = [&](int s) { return bar0 + 8u * s; };
     auto empty = [&](int s) { return bar0 + 8u * (kStages + s); };
-    const uint32_t done = bar0 + 8u * (2 * kStages);
+    auto acc_full = [&](int i) { return bar0 + 8u * (2 * kStages + i); };
+    auto acc_empty = [&](int i) { return bar0 + 8u * (2 * kStages + 2 + i); };
+    // tile -> first token, first feature, batch entry; tokens vary fastest (neighbours share W)
+    auto where = [&](int tile, int& m0, int& n0, int& z) {
+        m0 = (tile % a.mt) * kTok;
+        tile /= a.mt;
+        n0 = (tile % a.nt) * outs;
+        z = tile / a.nt;
+    };
 
     if (tid == 0) {
         for (int s = 0; s < kStages; s++) {
             mbar_init(full(s), 1);
             mbar_init(empty(s), 1);
         }
-        mbar_init(done, 1);
+        for (int i = 0; i < 2; i++) {
+            mbar_init(acc_full(i), 1);
+            mbar_init(acc_empty(i), 32 * kEpiWarps);
+        }
         abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
     if (warp == 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;"
-                     ::"r"(smem_u32(&tmem_slot)), "r"(TN) : "memory");
+                     ::"r"(smem_u32(&tmem_slot)), "r"(2 * TN) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -102,117 +117,182 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = tmem_slot;
     volatile int* abortp = &abort_flag;
+    int never = 0;
     pdl_wait();
 
     if (warp == 0) {
+        // ---------------- TMA producer ----------------
         if (lane == 0) {
-            const int wr0 = z * a.w_rows + n0, wr1 = a.glu ? wr0 + a.N : wr0 + TN / 2;
-            int it = 0;
-            for (; it < nk; it++) {
-                const int s = it % kStages;
-                if (!mbar_wait(empty(s), ((it / kStages) & 1) ^ 1, abortp)) { abort_flag = 1; break; }
-                mbar_expect_tx(full(s), kStage);
-                const uint32_t dst = smem_u32(smem + (size_t)s * kStage);
-                tma_load_2d(dst, &map_x, z * a.x_batch + it * kBlkK, m0, full(s));
-                tma_load_2d(dst + kXBytes, &map_w, it * kBlkK, wr0, full(s));
-                tma_load_2d(dst + kXBytes + TN / 2 * kBlkK * 2, &map_w, it * kBlkK, wr1, full(s));
+            int it = 0;                                  // stages filled so far, over all tiles
+            bool ok = true;
+            for (int tile = blockIdx.x; ok && tile < a.tiles; tile += gridDim.x) {
+                int m0, n0, z;
+                where(tile, m0, n0, z);
+                const int wr0 = z * a.w_rows + n0, wr1 = a.glu ? wr0 + a.N : wr0 + TN / 2;
+                for (int k = 0; k < nk; k++, it++) {
+                    const int s = it % kStages;
+                    if (!mbar_wait(empty(s), ((it / kStages) & 1) ^ 1, abortp)) {
+                        abort_flag = 1;
+                        ok = false;
+                        break;
+                    }
+                    mbar_expect_tx(full(s), kStage);
+                    const uint32_t dst = smem_u32(smem + (size_t)s * kStage);
+                    tma_load_2d(dst, &map_x, z * a.x_batch + k * kBlkK, m0, full(s));
+                    tma_load_2d(dst + kXBytes, &map_w, k * kBlkK, wr0, full(s));
+                    tma_load_2d(dst + kXBytes + TN / 2 * kBlkK * 2, &map_w, k * kBlkK, wr1, full(s));
+                }
             }
-            // normally the MMAs have consumed every stage; after an abort the copies still in
-            // flight must land before the shared memory goes away
-            if (it < nk || *abortp) {
-                int never = 0;
+            // normally the MMAs consume every stage; after an abort the copies still in flight
+            // must land before the shared memory goes away
+            if (*abortp)
                 for (int j = it > kStages ? it - kStages : 0; j < it; j++) mbar_wait(full(j % kStages), (j / kStages) & 1, &never);
-            }
         }
     } else if (warp == 1) {
+        // ---------------- MMA issuer ----------------
         if (lane == 0) {
             const uint32_t idesc = idesc_bf16<TN>();
-            for (int it = 0; it < nk; it++) {
-                const int s = it % kStages;
-                if (!mbar_wait(full(s), (it / kStages) & 1, abortp)) { abort_flag = 1; break; }
+            int it = 0, i = 0;                           // i: tiles of this CTA so far
+            bool ok = true;
+            for (int tile = blockIdx.x; ok && tile < a.tiles; tile += gridDim.x, i++) {
+                const int buf = i & 1;
+                if (!mbar_wait(acc_empty(buf), ((i >> 1) & 1) ^ 1, abortp)) {
+                    abort_flag = 1;
+                    break;
+                }
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const uint32_t xb = smem_u32(smem + (size_t)s * kStage), wb = xb + kXBytes;
+                const uint32_t acc = tmem + buf * TN;
+                for (int k = 0; k < nk; k++, it++) {
+                    const int s = it % kStages;
+                    if (!mbar_wait(full(s), (it / kStages) & 1, abortp)) {
+                        abort_flag = 1;
+                        ok = false;
+                        break;
+                    }
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    const uint32_t xb = smem_u32(smem + (size_t)s * kStage), wb = xb + kXBytes;
 #pragma unroll
-                for (int k = 0; k < kBlkK / 16; k++)
-                    mma_ss(tmem, make_sw128_desc(xb + k * 32), make_sw128_desc(wb + k * 32), idesc, (it > 0 || k > 0) ? 1u : 0u);
-                mma_commit(empty(s));
+                    for (int kk = 0; kk < kBlkK / 16; kk++)
+                        mma_ss(acc, make_sw128_desc(xb + kk * 32), make_sw128_desc(wb + kk * 32), idesc, (k > 0 || kk > 0) ? 1u : 0u);
+                    mma_commit(empty(s));
+                }
+                // arrives after everything issued so far, on the abort path too
+                mma_commit(acc_full(buf));
             }
-            mma_commit(done);
-            int never = 0;
-            if (!mbar_wait(done, 0, &never)) abort_flag = 1;
+            // the last accumulators complete before TMEM and shared memory are given up
+            for (int j = i > 2 ? i - 2 : 0; j < i; j++)
+                if (!mbar_wait(acc_full(j & 1), (j >> 1) & 1, &never)) abort_flag = 1;
         }
     } else if (warp >= 4) {
-        const int row = tid - 128, m = m0 + row;
-        int never = 0;
-        // `done` arrives on every path of the issuer, an aborted one included
-        const bool ok = __all_sync(0xffffffffu, mbar_wait(done, 0, &never) && !*abortp);
-        if (ok) {
+        // ---------------- epilogue ----------------
+        const int ew = warp - 4, row0 = (ew & 3) * 32, half = ew >> 2;
+        const uint32_t lane_base = tmem + ((uint32_t)row0 << 16);
+        uint32_t* st = reinterpret_cast<uint32_t*>(smem + (size_t)kStages * kStage) + ew * 32 * kStageLd;
+        const int sr = lane >> 2, sw = (lane & 3) * 4;   // row (of eight) and words this lane stores
+        const int wcols = a.y_f32 ? 1 : 2;               // columns per staged word
+        int i = 0;
+        for (int tile = blockIdx.x; tile < a.tiles; tile += gridDim.x, i++) {
+            const int buf = i & 1;
+            if (!__all_sync(0xffffffffu, mbar_wait(acc_full(buf), (i >> 1) & 1, abortp))) {
+                abort_flag = 1;
+                break;
+            }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint32_t lane_base = tmem + ((uint32_t)(row & ~31) << 16);
-            const float hg = (a.gate && m < a.M) ? sigmoid_f(__bfloat162float(a.gate[(size_t)m * a.gate_ld + z])) : 1.f;
+            int m0, n0, z;
+            where(tile, m0, n0, z);
+            const int mrow = m0 + row0;
+            const float hg = (a.gate && mrow + lane < a.M) ? sigmoid_f(__bfloat162float(a.gate[(size_t)(mrow + lane) * a.gate_ld + z])) : 1.f;
+            const int ncols = min(outs, a.N - n0);
+            const uint32_t acc = lane_base + buf * TN;
+            if (mrow < a.M)
 #pragma unroll 1
-            for (int c = 0; c < outs; c += 32) {
-                if (n0 + c >= a.N) break;
+            for (int c = half * 32; c < ncols; c += 64) {
                 uint32_t v[32];
                 __syncwarp();
-                tmem_ld32(lane_base + c, v);
+                tmem_ld32(acc + c, v);
                 float f[32];
                 if (a.glu) {
                     uint32_t u[32];
-                    tmem_ld32(lane_base + TN / 2 + c, u);
+                    tmem_ld32(acc + TN / 2 + c, u);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
-                    for (int j = 0; j < 32; j++) f[j] = apply_act(a.act, __uint_as_float(v[j])) * __uint_as_float(u[j]);
+                    for (int j = 0; j < 32; j++) f[j] = __uint_as_float(v[j]);
+                    apply_act_n<32>(a.act, f);
+#pragma unroll
+                    for (int j = 0; j < 32; j++) f[j] *= __uint_as_float(u[j]);
                 } else {
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
                     for (int j = 0; j < 32; j++) f[j] = __uint_as_float(v[j]);
                     if (a.bias) {
-                        const float* b = a.bias + (size_t)z * a.N + n0 + c;
+                        const float* bp = a.bias + (size_t)z * a.N + n0 + c;
+                        if (a.bias_vec && c + 32 <= ncols) {
 #pragma unroll
-                        for (int j = 0; j < 32; j++)
-                            if (n0 + c + j < a.N) f[j] += __ldg(b + j);
-                    }
-                    if (a.act != kActNone) {
+                            for (int j = 0; j < 8; j++) {
+                                const float4 t = __ldg(reinterpret_cast<const float4*>(bp) + j);
+                                f[4 * j] += t.x;
+                                f[4 * j + 1] += t.y;
+                                f[4 * j + 2] += t.z;
+                                f[4 * j + 3] += t.w;
+                            }
+                        } else {
 #pragma unroll
-                        for (int j = 0; j < 32; j++) f[j] = apply_act(a.act, f[j]);
+                            for (int j = 0; j < 32; j++)
+                                if (c + j < ncols) f[j] += __ldg(bp + j);
+                        }
                     }
+                    apply_act_n<32>(a.act, f);
                     if (a.gate) {
 #pragma unroll
                         for (int j = 0; j < 32; j++) f[j] *= hg;
                     }
                 }
-                if (m >= a.M) continue;
-                const size_t o = (size_t)m * a.ldy + (size_t)z * a.y_batch + n0 + c;
-                if (a.vec && n0 + c + 32 <= a.N) {
-                    if (a.y_f32) {
-                        float4* p = reinterpret_cast<float4*>(static_cast<float*>(a.y) + o);
+                // through shared memory, 16 words of a row at a time: FP32 in two halves, BF16 at once
 #pragma unroll
-                        for (int j = 0; j < 8; j++) p[j] = make_float4(f[4 * j], f[4 * j + 1], f[4 * j + 2], f[4 * j + 3]);
-                    } else {
-                        uint4* p = reinterpret_cast<uint4*>(static_cast<bf16*>(a.y) + o);
+                for (int part = 0; part < 2; part++) {
+                    if (part == 1 && !a.y_f32) break;
+                    __syncwarp();
 #pragma unroll
-                        for (int j = 0; j < 4; j++) {
-                            uint32_t w[4];
+                    for (int j = 0; j < 4; j++) {
+                        uint32_t w[4];
 #pragma unroll
-                            for (int q = 0; q < 4; q++) {
-                                const __nv_bfloat162 t = __floats2bfloat162_rn(f[8 * j + 2 * q], f[8 * j + 2 * q + 1]);
+                        for (int q = 0; q < 4; q++) {
+                            const int e = 4 * j + q;
+                            if (a.y_f32) {
+                                w[q] = __float_as_uint(f[part * 16 + e]);
+                            } else {
+                                const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * e], f[2 * e + 1]);
                                 w[q] = *reinterpret_cast<const uint32_t*>(&t);
                             }
-                            p[j] = make_uint4(w[0], w[1], w[2], w[3]);
                         }
+                        *reinterpret_cast<uint4*>(st + lane * kStageLd + 4 * j) = make_uint4(w[0], w[1], w[2], w[3]);
                     }
-                } else {
+                    __syncwarp();
+                    const int col = c + part * 16 + sw * wcols;      // first of this lane's columns inside the tile
+                    if (col < ncols) {
+                        const bool vec = a.vec && col + 4 * wcols <= ncols;
 #pragma unroll
-                    for (int j = 0; j < 32; j++) {
-                        if (n0 + c + j >= a.N) continue;
-                        if (a.y_f32) static_cast<float*>(a.y)[o + j] = f[j];
-                        else static_cast<bf16*>(a.y)[o + j] = __float2bfloat16_rn(f[j]);
+                        for (int r = 0; r < 4; r++) {
+                            const int rr = r * 8 + sr, m = mrow + rr;
+                            if (m >= a.M) break;
+                            const uint4 t = *reinterpret_cast<const uint4*>(st + rr * kStageLd + sw);
+                            const size_t o = (size_t)m * a.ldy + (size_t)z * a.y_batch + n0 + col;
+                            if (vec) {
+                                if (a.y_f32) *reinterpret_cast<uint4*>(static_cast<float*>(a.y) + o) = t;
+                                else *reinterpret_cast<uint4*>(static_cast<bf16*>(a.y) + o) = t;
+                            } else {
+                                const uint32_t w[4] = {t.x, t.y, t.z, t.w};
+                                for (int q = 0; q < 4 * wcols && col + q < ncols; q++) {
+                                    if (a.y_f32) static_cast<uint32_t*>(a.y)[o + q] = w[q];
+                                    else static_cast<uint16_t*>(a.y)[o + q] = (uint16_t)(w[q >> 1] >> ((q & 1) * 16));
+                                }
+                            }
+                        }
                     }
                 }
             }
-        } else {
-            abort_flag = 1;
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            mbar_arrive(acc_empty(buf));
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -220,7 +300,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
     if (abort_flag && tid == 0) atomicExch(a.err, TLLM_ERR_TIMEOUT);
     if (warp == 1) {
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(TN) : "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(2 * TN) : "memory");
     }
 }
 
@@ -238,7 +318,7 @@ int encode(EncodeTiledFn enc, CUtensorMap* map, const bf16* p, int cols, int row
 }
 
 template <int TN>
-int launch_tn(EncodeTiledFn enc, const LinearArgs<bf16>& l, DenseEpi e, cudaStream_t stream)
+int launch_tn(EncodeTiledFn enc, const LinearArgs<bf16>& l, DenseEpi e, int sms, cudaStream_t stream)
 {
     CUtensorMap mx, mw;
     int st;
@@ -252,8 +332,10 @@ int launch_tn(EncodeTiledFn enc, const LinearArgs<bf16>& l, DenseEpi e, cudaStre
         attr[dev] = true;
     }
     const int outs = l.glu ? TN / 2 : TN;
-    return launch_pdl("dense_gemm", dense_gemm_kernel<TN>, dim3((l.M + kTok - 1) / kTok, (l.N + outs - 1) / outs, l.batch),
-                      dim3(kThr), DCfg<TN>::kSmem, stream, mx, mw, e);
+    e.mt = (l.M + kTok - 1) / kTok;
+    e.nt = (l.N + outs - 1) / outs;
+    e.tiles = e.mt * e.nt * l.batch;
+    return launch_pdl("dense_gemm", dense_gemm_kernel<TN>, dim3(e.tiles < sms ? e.tiles : sms), dim3(kThr), DCfg<TN>::kSmem, stream, mx, mw, e);
 }
 
 }  // namespace
@@ -286,6 +368,7 @@ int launch_dense_gemm_tcgen05(const LinearArgs<bf16>& l, cudaStream_t stream)
     e.y_f32 = l.y_f32;
     const size_t es = l.y_f32 ? 4 : 2;
     e.vec = ((l.ldy * es) % 16 == 0 && (l.y_batch * es) % 16 == 0 && (reinterpret_cast<uintptr_t>(l.y) & 15) == 0);
+    e.bias_vec = l.N % 4 == 0 && (reinterpret_cast<uintptr_t>(l.bias) & 15) == 0;
     e.err = device_error_flag();
     if (!e.err) return fail(TLLM_ERR_LAUNCH, "device scratch unavailable");
     static int sms[64] = {};
@@ -299,9 +382,9 @@ int launch_dense_gemm_tcgen05(const LinearArgs<bf16>& l, cudaStream_t stream)
         const int outs = l.glu ? tn / 2 : tn;
         return mt * ((l.N + outs - 1) / outs) * l.batch;
     };
-    if (tiles(256) * 10 >= 7LL * sms[dev]) return launch_tn<256>(enc, l, e, stream);
-    if (tiles(128) * 10 >= 7LL * sms[dev]) return launch_tn<128>(enc, l, e, stream);
-    return launch_tn<64>(enc, l, e, stream);
+    if (tiles(256) * 10 >= 7LL * sms[dev]) return launch_tn<256>(enc, l, e, sms[dev], stream);
+    if (tiles(128) * 10 >= 7LL * sms[dev]) return launch_tn<128>(enc, l, e, sms[dev], stream);
+    return launch_tn<64>(enc, l, e, sms[dev], stream);
 }
 
 }  // namespace tllm

@@ -4,8 +4,11 @@
 // HBM-bound: a row of W is read once for up to eight vectors, which are staged in shared
 // memory.  A row is served by a power-of-two group of lanes (a whole warp for rows of 32 or
 // more 16-byte pieces, fewer lanes for short rows such as the step-size projection of a
-// selective scan), each lane keeping eight 16-byte loads in flight.  The first loads are
-// issued before the wait on the previous kernel: weights depend on nothing in the stream.
+// selective scan).  Every lane streams its pieces through a ring of its own in shared memory
+// (cp.async, three groups of four pieces; a lane reads back only what it copied, so no barrier
+// is involved), and the ring runs across the ends of rows.  The first groups are requested
+// before the wait on the previous kernel -- weights depend on nothing in the stream -- and a
+// launch leaves room on the SM for the next one to do the same.
 #include "dense.cuh"
 #include "launch.cuh"
 
@@ -14,62 +17,194 @@ namespace tllm {
 namespace {
 
 constexpr int kWarps = 8;
-constexpr int kAhead = 8;      // 16-byte loads in flight per lane
+constexpr int kPieces = 4, kGroups = 3;        // ring of a lane: groups of 16-byte pieces
+constexpr int kNormVecs = 4;                   // float4s of the residual row per thread (norm staging)
+constexpr int kNormMaxK = kNormVecs * kWarps * 32 * 4;
+constexpr size_t kRingBytes = (size_t)kGroups * kPieces * kWarps * 32 * 16;
 
-template <typename T, int MB>
+__device__ __forceinline__ void ring_copy(uint32_t dst, const void* src, bool valid)
+{
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+
+// sh: one word per warp, not used by an earlier sum that is still being read
+__device__ __forceinline__ float gemv_cta_sum(float v, float* sh)
+{
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int i = 0; i < kWarps; i++) t += sh[i];
+    return t;
+}
+
+__device__ __forceinline__ float4 gemv_ld4(const float* p, int i) { return *(reinterpret_cast<const float4*>(p) + i); }
+
+// One vector of the residual chain into shared memory; wp, wn: the norm weights, staged before
+// the wait on the previous kernel.  sh: 2 * kWarps words.
+template <typename T>
+__device__ __forceinline__ void stage_norm(const GemvNorm& f, int m, int K, T* xs, const float* wp, const float* wn, float* sh)
+{
+    const size_t row = (size_t)m * K;
+    const int n4 = K >> 2;
+    float4 y[kNormVecs], x[kNormVecs];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < kNormVecs; j++) {
+        const int i = threadIdx.x + j * kWarps * 32;
+        y[j] = x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < n4) {
+            y[j] = gemv_ld4(f.y + row, i);
+            x[j] = gemv_ld4(f.x_in + row, i);
+            if (f.extra) {
+                const float4 e = gemv_ld4(f.extra + row, i);
+                x[j].x += e.x;
+                x[j].y += e.y;
+                x[j].z += e.z;
+                x[j].w += e.w;
+            }
+        }
+        ss += (y[j].x * y[j].x + y[j].y * y[j].y) + (y[j].z * y[j].z + y[j].w * y[j].w);
+    }
+    float rinv = 1.f;
+    if (f.w_post) rinv = 1.0f / sqrtf(gemv_cta_sum(ss, sh) / (float)f.width + f.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < kNormVecs; j++) {
+        const int i = threadIdx.x + j * kWarps * 32;
+        if (i >= n4) continue;
+        float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (f.w_post) w = reinterpret_cast<const float4*>(wp)[i];
+        x[j].x += y[j].x * rinv * w.x;
+        x[j].y += y[j].y * rinv * w.y;
+        x[j].z += y[j].z * rinv * w.z;
+        x[j].w += y[j].w * rinv * w.w;
+        if (blockIdx.x == 0 && blockIdx.y == 0) reinterpret_cast<float4*>(f.x_out + row)[i] = x[j];
+        ss += (x[j].x * x[j].x + x[j].y * x[j].y) + (x[j].z * x[j].z + x[j].w * x[j].w);
+    }
+    rinv = 1.0f / sqrtf(gemv_cta_sum(ss, sh + kWarps) / (float)f.width + f.eps);
+#pragma unroll
+    for (int j = 0; j < kNormVecs; j++) {
+        const int i = threadIdx.x + j * kWarps * 32;
+        if (i >= n4) continue;
+        const float4 w = reinterpret_cast<const float4*>(wn)[i];
+        T* d = xs + 4 * i;
+        d[0] = from_f<T>(x[j].x * rinv * w.x);
+        d[1] = from_f<T>(x[j].y * rinv * w.y);
+        d[2] = from_f<T>(x[j].z * rinv * w.z);
+        d[3] = from_f<T>(x[j].w * rinv * w.w);
+    }
+    __syncthreads();             // the next vector's sums reuse sh
+}
+
+template <typename T, int MB, bool NORM, int TAIL>
 __global__ void __launch_bounds__(kWarps * 32)
-dense_gemv_kernel(const LinearArgs<T> a, int lanes_per_row, int m0)
+dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, int lanes_per_row, int m0)
 {
     constexpr int V = Vec16<T>::n;
     extern __shared__ __align__(16) uint8_t smem_raw[];
-    T* xs = reinterpret_cast<T*>(smem_raw);                  // [MB][K]
+    __shared__ float sh[2 * kWarps];
+    // ring, then the vectors [MB][K], then with NORM the two norm weights [K] each
+    T* xs = reinterpret_cast<T*>(smem_raw + kRingBytes);
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int sub = lane / lanes_per_row, l = lane - sub * lanes_per_row, rpw = 32 / lanes_per_row;
     const int z = blockIdx.y;
     const int nv = a.K / V;                                  // 16-byte pieces per row
     const int stride = gridDim.x * kWarps * rpw;
-    const int first = (blockIdx.x * kWarps + warp) * rpw + sub;
+    const int nb0 = (blockIdx.x * kWarps + warp) * rpw;
+    const int parts = (TAIL == kTailGate || a.glu) ? 2 : 1;
     const T* wz = a.w + (size_t)z * a.w_rows * a.ldw;
 
-    uint4 pre[kAhead];
-    auto fetch = [&](const T* row, int c0, bool valid) {
+    // ring of this lane: piece u of slot s at ring[(s * kPieces + u) * threads]
+    const uint4* ring = reinterpret_cast<const uint4*>(smem_raw) + threadIdx.x;
+    const uint32_t ring32 = (uint32_t)__cvta_generic_to_shared(ring);
+    int f_nb = nb0, f_part = 0, f_c = 0, f_slot = 0;         // what is requested next
+    auto request = [&]() {
+        if (f_nb < a.N) {
+            const int n = f_nb + sub;
+            const T* row = wz + (size_t)(n < a.N ? n + f_part * a.N : 0) * a.ldw;
 #pragma unroll
-        for (int u = 0; u < kAhead; u++) {
-            const int c = c0 + u * lanes_per_row;
-            pre[u] = (valid && c < nv) ? __ldcs(reinterpret_cast<const uint4*>(row) + c) : make_uint4(0, 0, 0, 0);
+            for (int u = 0; u < kPieces; u++) {
+                const int c = f_c + u * lanes_per_row + l;
+                const bool v = n < a.N && c < nv;
+                ring_copy(ring32 + (uint32_t)((f_slot * kPieces + u) * kWarps * 32 * 16), v ? row + (size_t)c * V : wz, v);
+            }
+            f_c += kPieces * lanes_per_row;
+            if (f_c >= nv) {
+                f_c = 0;
+                if (++f_part == parts) {
+                    f_part = 0;
+                    f_nb += stride;
+                }
+            }
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        f_slot = f_slot == kGroups - 1 ? 0 : f_slot + 1;
     };
-    fetch(wz + (size_t)first * a.ldw, l, first < a.N);
+#pragma unroll
+    for (int g = 0; g < kGroups; g++) request();
+    if (NORM) {
+        float* wn = reinterpret_cast<float*>(xs + (size_t)MB * a.K);
+        for (int i = threadIdx.x; i < a.K / 4; i += kWarps * 32) {
+            reinterpret_cast<float4*>(wn)[i] = gemv_ld4(f.w_next, i);
+            if (f.w_post) reinterpret_cast<float4*>(wn + a.K)[i] = gemv_ld4(f.w_post, i);
+        }
+    }
 
     pdl_wait();
     const int mb = min(MB, a.M - m0);
-    for (int i = threadIdx.x; i < mb * nv; i += kWarps * 32) {
-        const int m = i / nv, c = i - m * nv;
-        reinterpret_cast<uint4*>(xs + (size_t)m * a.K)[c] =
-            *(reinterpret_cast<const uint4*>(a.x + (size_t)(m0 + m) * a.ldx + (size_t)z * a.x_batch) + c);
+    if (NORM) {
+        const float* wn = reinterpret_cast<const float*>(xs + (size_t)MB * a.K);
+        for (int m = 0; m < mb; m++) stage_norm<T>(f, m, a.K, xs + (size_t)m * a.K, wn + a.K, wn, sh);
+    } else {
+        for (int i = threadIdx.x; i < mb * nv; i += kWarps * 32) {
+            const int m = i / nv, c = i - m * nv;
+            reinterpret_cast<uint4*>(xs + (size_t)m * a.K)[c] =
+                *(reinterpret_cast<const uint4*>(a.x + (size_t)(m0 + m) * a.ldx + (size_t)z * a.x_batch) + c);
+        }
     }
     for (int i = threadIdx.x + mb * nv; i < MB * nv; i += kWarps * 32) reinterpret_cast<uint4*>(xs)[i] = make_uint4(0, 0, 0, 0);
+    const bool fresh = TAIL != kTailNone && (t.pos_dev ? *t.pos_dev : t.start_pos) == 0;
     __syncthreads();
 
-    const int parts = a.glu ? 2 : 1;
+    int slot = 0;
     // all lanes of a warp take the same number of trips (the shuffles name all of them)
-    for (int nb = (blockIdx.x * kWarps + warp) * rpw; nb < a.N; nb += stride) {
+    for (int nb = nb0; nb < a.N; nb += stride) {
         const int n = nb + sub;
+        const bool valid = n < a.N;
+        // what the tail needs of this row is requested before the row itself
+        float hist[MB], tw = 0.f;
+        const bool conv = TAIL == kTailConv && valid && n >= t.lo && n < t.hi;
+        const int ch = TAIL == kTailConv ? n - t.lo : z * a.N + n, width = t.hi - t.lo;
+        if (TAIL == kTailConv) {
+            if (conv && l < t.taps) tw = t.w[(size_t)ch * t.taps + l];
+#pragma unroll
+            for (int m = 0; m < MB; m++)
+                hist[m] = (conv && m < mb && l + 1 < t.taps && !fresh)
+                              ? to_f<T>(t.carried[(size_t)(t.first_slot + m) * t.slot_stride + (size_t)l * width + ch]) : 0.f;
+        } else if (TAIL == kTailGate) {
+#pragma unroll
+            for (int m = 0; m < MB; m++)
+                hist[m] = (valid && m < mb && !fresh) ? t.state[(size_t)(t.first_slot + m) * t.slot_stride + ch] : 0.f;
+            if (valid) tw = -t.decay * t.soft_lam[ch];
+        }
         float res[2][MB];
+#pragma unroll
+        for (int m = 0; m < MB; m++) res[1][m] = 0.f;
         for (int part = 0; part < parts; part++) {
-            const bool valid = n < a.N;
-            const T* row = wz + (size_t)(valid ? n + part * a.N : 0) * a.ldw;
             float acc[MB];
 #pragma unroll
             for (int m = 0; m < MB; m++) acc[m] = 0.f;
-            for (int c0 = l; c0 < nv; c0 += kAhead * lanes_per_row) {
-                if (!(nb == (blockIdx.x * kWarps + warp) * rpw && part == 0 && c0 == l)) fetch(row, c0, valid);
+            for (int cb = l; cb - l < nv; cb += kPieces * lanes_per_row) {
+                asm volatile("cp.async.wait_group %0;" ::"n"(kGroups - 1) : "memory");
+                const uint4* rs = ring + slot * kPieces * kWarps * 32;
 #pragma unroll
-                for (int u = 0; u < kAhead; u++) {
-                    const int c = min(c0 + u * lanes_per_row, nv - 1);     // pieces past the row are zero
+                for (int u = 0; u < kPieces; u++) {
+                    const int c = min(cb + u * lanes_per_row, nv - 1);     // pieces past the row are zero
                     float wf[V];
-                    Vec16<T>::unpack(pre[u], wf);
+                    Vec16<T>::unpack(rs[u * kWarps * 32], wf);
 #pragma unroll
                     for (int m = 0; m < MB; m++) {
                         float xf[V];
@@ -78,17 +213,47 @@ dense_gemv_kernel(const LinearArgs<T> a, int lanes_per_row, int m0)
                         for (int j = 0; j < V; j++) acc[m] = fmaf(wf[j], xf[j], acc[m]);
                     }
                 }
+                request();
+                slot = slot == kGroups - 1 ? 0 : slot + 1;
             }
 #pragma unroll
             for (int m = 0; m < MB; m++) {
                 for (int o = lanes_per_row >> 1; o > 0; o >>= 1) acc[m] += __shfl_xor_sync(0xffffffffu, acc[m], o);
-                res[part][m] = acc[m];
+                if (part == 0) res[0][m] = acc[m];
+                else res[1][m] = acc[m];
             }
         }
-        if (n >= a.N) continue;
+        if (TAIL == kTailConv) {
+            // every lane of the group holds the row's new input; lane j weighs carried input j,
+            // lane taps - 1 the new one
+#pragma unroll
+            for (int m = 0; m < MB; m++) {
+                const float v = to_f<T>(from_f<T>(res[0][m] + ((a.bias && valid) ? a.bias[n] : 0.f)));
+                float s = 0.f;
+                if (conv && m < mb) s = l + 1 < t.taps ? tw * hist[m] : l + 1 == t.taps ? tw * v : 0.f;
+                for (int o = lanes_per_row >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+                if (conv && m < mb) {
+                    T* cr = t.carried + (size_t)(t.first_slot + m) * t.slot_stride + ch;
+                    if (l > 0 && l + 1 < t.taps) cr[(size_t)(l - 1) * width] = from_f<T>(hist[m]);
+                    if (l + 1 == t.taps && t.taps > 1) cr[(size_t)(t.taps - 2) * width] = from_f<T>(v);
+                    if (l == 0) t.out[(size_t)m * t.ld_out + ch] = from_f<T>(apply_act(t.act, s + (t.bias ? t.bias[ch] : 0.f)));
+                }
+            }
+            if (conv) continue;
+        }
+        if (!valid) continue;
 #pragma unroll
         for (int m = 0; m < MB; m++) {
             if (m >= mb || l != m % lanes_per_row) continue;     // one lane of the group per vector
+            if (TAIL == kTailGate) {
+                const float* b = a.bias + (size_t)z * 2 * a.N;
+                const float r = sigmoid_f(res[0][m] + b[n]), i = sigmoid_f(res[1][m] + b[a.N + n]);
+                const float log_a = tw * r, A = expf(log_a);
+                const float S = fmaf(A, hist[m], sqrtf(one_minus_exp(2.f * log_a, A * A)) * i * to_f<T>(xs[(size_t)m * a.K + n]));
+                t.state[(size_t)(t.first_slot + m) * t.slot_stride + ch] = S;
+                t.out[(size_t)m * t.ld_out + ch] = from_f<T>(S * apply_act(t.act, to_f<T>(t.y[(size_t)m * t.ld_y + ch])));
+                continue;
+            }
             float v = res[0][m];
             if (a.bias) v += a.bias[(size_t)z * a.N + n];
             v = apply_act(a.act, v);
@@ -101,54 +266,109 @@ dense_gemv_kernel(const LinearArgs<T> a, int lanes_per_row, int m0)
     }
 }
 
-template <typename T, int MB>
-int launch_mb(const LinearArgs<T>& a, int m0, cudaStream_t stream)
+template <typename T>
+int row_lanes(int k)
+{
+    const int nv = k / Vec16<T>::n;
+    int lpr = 1;
+    while (lpr < 32 && lpr < nv) lpr *= 2;
+    return lpr;
+}
+
+constexpr size_t kSmemLimit = 220 * 1024;
+
+template <typename T, int MB, bool NORM, int TAIL>
+int launch_mb(const LinearArgs<T>& a, const GemvNorm& f, const GemvTail<T>& t, int m0, cudaStream_t stream)
 {
     static bool attr[64] = {};
     static int sms[64] = {};
     int dev = 0;
     cudaGetDevice(&dev);
     if (!attr[dev]) {
-        cudaFuncSetAttribute(dense_gemv_kernel<T, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        cudaFuncSetAttribute(dense_gemv_kernel<T, MB, NORM, TAIL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemLimit);
         cudaDeviceGetAttribute(&sms[dev], cudaDevAttrMultiProcessorCount, dev);
         attr[dev] = true;
     }
-    const int nv = a.K / Vec16<T>::n;
-    int lpr = 1;
-    while (lpr < 32 && lpr < nv) lpr *= 2;
+    const int lpr = row_lanes<T>(a.K);
     const int rows_per_cta = kWarps * (32 / lpr);
     int grid = (a.N + rows_per_cta - 1) / rows_per_cta;
-    const int cap = sms[dev] * 8;
+    // two CTAs per SM: the next launch finds room and requests its weights early
+    const int cap = (2 * sms[dev] + a.batch - 1) / a.batch;
     if (grid > cap) grid = cap;
-    return launch_pdl("dense_gemv", dense_gemv_kernel<T, MB>, dim3(grid, a.batch), dim3(kWarps * 32),
-                      (size_t)MB * a.K * sizeof(T), stream, a, lpr, m0);
+    const size_t smem = kRingBytes + (size_t)MB * a.K * sizeof(T) + (NORM ? (size_t)2 * a.K * sizeof(float) : 0);
+    if (smem > kSmemLimit || (NORM && a.K > kNormMaxK)) return fail(TLLM_ERR_SHAPE, "dense_gemv: %d vectors of %d", MB, a.K);
+    return launch_pdl("dense_gemv", dense_gemv_kernel<T, MB, NORM, TAIL>, dim3(grid, a.batch), dim3(kWarps * 32), smem, stream, a, f, t, lpr, m0);
+}
+
+template <typename T, bool NORM, int TAIL>
+int launch_any(const LinearArgs<T>& a, const GemvNorm& f, const GemvTail<T>& t, int mb, int m0, cudaStream_t stream)
+{
+    switch (mb) {
+        case 8: return launch_mb<T, 8, NORM, TAIL>(a, f, t, m0, stream);
+        case 4: return launch_mb<T, 4, NORM, TAIL>(a, f, t, m0, stream);
+        case 2: return launch_mb<T, 2, NORM, TAIL>(a, f, t, m0, stream);
+        default: return launch_mb<T, 1, NORM, TAIL>(a, f, t, m0, stream);
+    }
+}
+
+template <typename T>
+int check_gemv(const LinearArgs<T>& a)
+{
+    if (a.K < 8 || a.K % 8 || a.ldw % 8 || a.ldx % 8 || a.x_batch % 8)
+        return fail(TLLM_ERR_SHAPE, "dense_gemv: K=%d ldw=%d ldx=%d x_batch=%d must be multiples of 8", a.K, a.ldw, a.ldx, a.x_batch);
+    if ((size_t)a.K * sizeof(T) > kSmemLimit - kRingBytes)
+        return fail(TLLM_ERR_SHAPE, "dense_gemv: K=%d exceeds %d", a.K, (int)((kSmemLimit - kRingBytes) / sizeof(T)));
+    return TLLM_OK;
 }
 
 }  // namespace
 
 template <typename T>
+bool gemv_tail_fits(int k, int taps)
+{
+    return row_lanes<T>(k) >= taps;
+}
+template <typename T>
+bool gemv_norm_fits(int k)
+{
+    return k <= kNormMaxK && kRingBytes + (size_t)k * (8 * sizeof(T) + 2 * sizeof(float)) <= kSmemLimit;
+}
+template bool gemv_norm_fits<bf16>(int);
+template bool gemv_norm_fits<float>(int);
+template bool gemv_tail_fits<bf16>(int, int);
+template bool gemv_tail_fits<float>(int, int);
+
+template <typename T>
+int launch_dense_gemv_fused(const LinearArgs<T>& a, const GemvNorm& f, const GemvTail<T>& t, cudaStream_t stream)
+{
+    if (a.M == 0 || a.N == 0 || a.batch == 0) return TLLM_OK;
+    const int st = check_gemv(a);
+    if (st) return st;
+    if (a.M > 8 || (f.y && (a.batch != 1 || f.x_in == f.x_out))) return fail(TLLM_ERR_SHAPE, "dense_gemv (fused): %d vectors", a.M);
+    if (t.kind == kTailConv && !gemv_tail_fits<T>(a.K, t.taps)) return fail(TLLM_ERR_SHAPE, "dense_gemv (fused): %d taps for K=%d", t.taps, a.K);
+    const int mb = a.M >= 5 ? 8 : a.M >= 3 ? 4 : a.M;
+    if (f.y)
+        return t.kind == kTailConv ? launch_any<T, true, kTailConv>(a, f, t, mb, 0, stream) : launch_any<T, true, kTailNone>(a, f, t, mb, 0, stream);
+    if (t.kind == kTailConv) return launch_any<T, false, kTailConv>(a, f, t, mb, 0, stream);
+    if (t.kind == kTailGate) return launch_any<T, false, kTailGate>(a, f, t, mb, 0, stream);
+    return launch_any<T, false, kTailNone>(a, f, t, mb, 0, stream);
+}
+template int launch_dense_gemv_fused<bf16>(const LinearArgs<bf16>&, const GemvNorm&, const GemvTail<bf16>&, cudaStream_t);
+template int launch_dense_gemv_fused<float>(const LinearArgs<float>&, const GemvNorm&, const GemvTail<float>&, cudaStream_t);
+
+template <typename T>
 int launch_dense_gemv(const LinearArgs<T>& a, cudaStream_t stream)
 {
     if (a.M == 0 || a.N == 0 || a.batch == 0) return TLLM_OK;
-    if (a.K < 8 || a.K % 8 || a.ldw % 8 || a.ldx % 8 || a.x_batch % 8)
-        return fail(TLLM_ERR_SHAPE, "dense_gemv: K=%d ldw=%d ldx=%d x_batch=%d must be multiples of 8", a.K, a.ldw, a.ldx, a.x_batch);
-    const size_t limit = 200 * 1024;
-    if ((size_t)a.K * sizeof(T) > limit) return fail(TLLM_ERR_SHAPE, "dense_gemv: K=%d exceeds %d", a.K, (int)(limit / sizeof(T)));
-    for (int m0 = 0; m0 < a.M;) {
+    int st = check_gemv(a);
+    for (int m0 = 0; !st && m0 < a.M;) {
         const int left = a.M - m0;
         int mb = left >= 5 ? 8 : left >= 3 ? 4 : left;
-        while ((size_t)mb * a.K * sizeof(T) > limit) mb /= 2;
-        int st = TLLM_OK;
-        switch (mb) {
-            case 8: st = launch_mb<T, 8>(a, m0, stream); break;
-            case 4: st = launch_mb<T, 4>(a, m0, stream); break;
-            case 2: st = launch_mb<T, 2>(a, m0, stream); break;
-            default: st = launch_mb<T, 1>(a, m0, stream); break;
-        }
-        if (st) return st;
+        while ((size_t)mb * a.K * sizeof(T) > kSmemLimit - kRingBytes) mb /= 2;
+        st = launch_any<T, false, kTailNone>(a, GemvNorm(), GemvTail<T>(), mb, m0, stream);
         m0 += mb;
     }
-    return TLLM_OK;
+    return st;
 }
 template int launch_dense_gemv<bf16>(const LinearArgs<bf16>&, cudaStream_t);
 template int launch_dense_gemv<float>(const LinearArgs<float>&, cudaStream_t);

@@ -27,7 +27,7 @@ constexpr float kLog2e = 1.4426950408889634f;
 // ---------------------------------------------------------------------------
 // Latent norm, rotations, cache append
 // ---------------------------------------------------------------------------
-constexpr int kPrepThreads = 128;
+constexpr int kPrepThreads = 256;
 
 template <typename T>
 __global__ void __launch_bounds__(kPrepThreads)
@@ -44,21 +44,27 @@ latent_prep_kernel(const LatentArgs<T> a, T* __restrict__ q_abs)
     T* cache = a.cache + (size_t)(a.g.first_slot + b) * a.slot_stride + (size_t)pos * (a.rank + a.rot);
     const float2* cs = a.rope + (size_t)pos * half_dims;
 
-    float ss = 0.f;
-    for (int i = tid; i < a.rank; i += kPrepThreads) {
-        const float v = to_f<T>(proj[a.kv_off + i]);
-        ss += v * v;
+    if (blockIdx.y == 0) {       // the latent
+        float ss = 0.f;
+        for (int i = tid; i < a.rank; i += kPrepThreads) {
+            const float v = to_f<T>(proj[a.kv_off + i]);
+            ss += v * v;
+        }
+        ss = warp_sum(ss);
+        if ((tid & 31) == 0) sh[tid >> 5] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < kPrepThreads / 32; i++) ss += sh[i];
+        const float rinv = 1.0f / sqrtf(ss / (float)a.rank_true + a.eps);
+        for (int i = tid; i < a.rank; i += kPrepThreads) cache[i] = from_f<T>(to_f<T>(proj[a.kv_off + i]) * rinv * a.kv_norm[i]);
+        return;
     }
-    ss = warp_sum(ss);
-    if ((tid & 31) == 0) sh[tid >> 5] = ss;
-    __syncthreads();
-    ss = (sh[0] + sh[1]) + (sh[2] + sh[3]);
-    const float rinv = 1.0f / sqrtf(ss / (float)a.rank_true + a.eps);
-    for (int i = tid; i < a.rank; i += kPrepThreads) cache[i] = from_f<T>(to_f<T>(proj[a.kv_off + i]) * rinv * a.kv_norm[i]);
 
     // rotated parts: head -1 is the shared key part
     const int per = a.rot - half_dims;                      // half_dims pairs, then the entries that pass
     const int dk = a.rank + a.rot;
+#pragma unroll 2
     for (int i = tid; i < (a.heads + 1) * per; i += kPrepThreads) {
         const int h = i / per - 1, e = i - (h + 1) * per;
         const T* src = (h < 0) ? proj + a.kv_off + a.rank : proj + a.q_off + (size_t)h * (a.dim + a.rot) + a.dim;
@@ -326,7 +332,7 @@ latent_absorbed_mma_kernel(const LatentArgs<bf16> a, const bf16* __restrict__ q_
             float sum = 0.f;
 #pragma unroll
             for (int j = 0; j < TK / 32; j++) {
-                const float p = (s[j] == -INFINITY) ? 0.f : exp2f(s[j] - m_new);
+                const float p = (s[j] == -INFINITY) ? 0.f : exp2_neg(s[j] - m_new);
                 sum += p;
                 const bf16 h = __float2bfloat16_rn(p);
                 ph[r * (TK + 8) + lane + 32 * j] = h;
@@ -403,6 +409,14 @@ latent_merge_kernel(const LatentArgs<bf16> a, const float* __restrict__ ws, bf16
     const int total = min((a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) + a.g.seq_len, a.max_seq);
     const int len = split_len(total, nsplit), active = (total + len - 1) / len, rec = a.rank + 2;
     const float* base = ws + (size_t)row * nsplit * rec;
+    // the first half of the partial sums is requested before the weights are known
+    constexpr int kAtOnce = kAbsMaxSplit / 2;
+    float v[kAtOnce];
+    auto load = [&](int s0) {
+#pragma unroll
+        for (int u = 0; u < kAtOnce; u++) v[u] = (c < a.rank && s0 + u < active) ? __ldcg(base + (size_t)(s0 + u) * rec + c) : 0.f;
+    };
+    load(0);
     if (threadIdx.x < 32) {
         const int s0 = threadIdx.x, s1 = threadIdx.x + 32;
         const float m0 = s0 < active ? base[(size_t)s0 * rec + a.rank] : -INFINITY, m1 = s1 < active ? base[(size_t)s1 * rec + a.rank] : -INFINITY;
@@ -421,13 +435,11 @@ latent_merge_kernel(const LatentArgs<bf16> a, const float* __restrict__ ws, bf16
     __syncthreads();
     if (c >= a.rank) return;
     float o = 0.f;
-    for (int s = 0; s < active; s += 8) {
-        float v[8];
+    for (int s0 = 0; s0 < active; s0 += kAtOnce) {
+        if (s0) load(s0);
 #pragma unroll
-        for (int u = 0; u < 8; u++) v[u] = (s + u < active) ? __ldcg(base + (size_t)(s + u) * rec + c) : 0.f;
-#pragma unroll
-        for (int u = 0; u < 8; u++)
-            if (s + u < active) o = fmaf(wgt[s + u], v[u], o);
+        for (int u = 0; u < kAtOnce; u++)
+            if (s0 + u < active) o = fmaf(wgt[s0 + u], v[u], o);
     }
     o_lat[(size_t)row * a.rank + c] = __float2bfloat16_rn(o);
 }
@@ -477,16 +489,23 @@ latent_expanded_kernel(const LatentArgs<bf16> a, const bf16* __restrict__ kx, co
             cp16(qs + r * ldq + c * 8, v ? a.proj + (size_t)(q0 + r) * a.ld + a.q_off + (size_t)h * dq + c * 8 : a.proj, v);
         }
     }
+    // pieces of 16 bytes per row: unrotated key, shared key part, value; i / pieces as a multiplication
+    const int pk = a.dim / 8, pr = a.rot / 8, pv = a.vdim / 8;
+    const uint32_t mk = 0xffffffffu / pk + 1, mr = pr ? 0xffffffffu / pr + 1 : 0, mv = 0xffffffffu / pv + 1;
+    const bf16 *kxh = kx + (size_t)h * a.dim, *vxh = vx + (size_t)h * a.vdim, *krh = cache + a.rank;
+    const size_t kx_ld = (size_t)a.heads * a.dim, vx_ld = (size_t)a.heads * a.vdim;
+    auto load_part = [&](bf16* dst, int ld, const bf16* src, size_t src_ld, int pieces, uint32_t magic, int k0) {
+        for (int i = tid; i < kExpK * pieces; i += kExpThreads) {
+            const int r = pieces == 1 ? i : (int)__umulhi((uint32_t)i, magic), c = (i - r * pieces) * 8;
+            const bool v = k0 + r < hi;
+            cp16(dst + r * ld + c, v ? src + (size_t)(k0 + r) * src_ld + c : src, v);
+        }
+    };
     auto load_tile = [&](int k0, int stage) {
         bf16 *kd = ks + (size_t)stage * kExpK * ldq, *vd = vs + (size_t)stage * kExpK * ldv;
-        const int pk = a.dim / 8, pr = a.rot / 8, pv = a.vdim / 8, pall = pk + pr + pv;
-        for (int i = tid; i < kExpK * pall; i += kExpThreads) {
-            const int r = i / pall, c = i - r * pall, k = k0 + r;
-            const bool v = k < hi;
-            if (c < pk) cp16(kd + r * ldq + c * 8, v ? kx + ((size_t)k * a.heads + h) * a.dim + c * 8 : kx, v);
-            else if (c < pk + pr) cp16(kd + r * ldq + c * 8, v ? cache + (size_t)k * dk + a.rank + (c - pk) * 8 : cache, v);
-            else cp16(vd + r * ldv + (c - pk - pr) * 8, v ? vx + ((size_t)k * a.heads + h) * a.vdim + (c - pk - pr) * 8 : vx, v);
-        }
+        load_part(kd, ldq, kxh, kx_ld, pk, mk, k0);
+        if (pr) load_part(kd + a.dim, ldq, krh, (size_t)dk, pr, mr, k0);
+        load_part(vd, ldv, vxh, vx_ld, pv, mv, k0);
         cp_commit();
     };
     float o[NV][4];
@@ -542,16 +561,18 @@ latent_expanded_kernel(const LatentArgs<bf16> a, const bf16* __restrict__ kx, co
             mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
             mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
             const float m_new = fmaxf(m_run[e], mx[e]);
-            cr[e] = (m_run[e] == -INFINITY) ? 0.f : exp2f(m_run[e] - m_new);
+            cr[e] = exp2_neg(m_run[e] - m_new);                // 0 at first: position 0 is seen by every query
             m_run[e] = m_new;
             l_run[e] *= cr[e];
         }
+        if (__any_sync(0xffffffffu, cr[0] != 1.f || cr[1] != 1.f)) {
 #pragma unroll
-        for (int j = 0; j < NV; j++) {
-            o[j][0] *= cr[0];
-            o[j][1] *= cr[0];
-            o[j][2] *= cr[1];
-            o[j][3] *= cr[1];
+            for (int j = 0; j < NV; j++) {
+                o[j][0] *= cr[0];
+                o[j][1] *= cr[0];
+                o[j][2] *= cr[1];
+                o[j][3] *= cr[1];
+            }
         }
 #pragma unroll
         for (int k = 0; k < 4; k++) {                          // 16 positions per step
@@ -561,7 +582,7 @@ latent_expanded_kernel(const LatentArgs<bf16> a, const bf16* __restrict__ kx, co
                 float (&v)[4] = s[2 * k + q];
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
-                    v[e] = (v[e] == -INFINITY) ? 0.f : exp2f(v[e] - m_run[e >> 1]);
+                    v[e] = exp2_neg(v[e] - m_run[e >> 1]);
                     l_run[e >> 1] += v[e];
                 }
                 split2(v[0], v[1], fh[2 * q], fl[2 * q]);
@@ -690,7 +711,7 @@ int launch_latent_prep(const LatentArgs<T>& a, T* q_abs, cudaStream_t stream)
     if (a.g.rows() == 0) return TLLM_OK;
     int st = check_latent(a);
     if (st) return st;
-    return launch_pdl("latent_prep", latent_prep_kernel<T>, dim3(a.g.rows()), dim3(kPrepThreads), 0, stream, a, q_abs);
+    return launch_pdl("latent_prep", latent_prep_kernel<T>, dim3(a.g.rows(), 2), dim3(kPrepThreads), 0, stream, a, q_abs);
 }
 template int launch_latent_prep<bf16>(const LatentArgs<bf16>&, bf16*, cudaStream_t);
 template int launch_latent_prep<float>(const LatentArgs<float>&, float*, cudaStream_t);

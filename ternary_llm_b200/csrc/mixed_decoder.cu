@@ -74,12 +74,12 @@ struct MixedDecoder : Decoder {
     std::vector<RunState<T>> runs;
     Mat<T> embed;
     float* final_norm = nullptr;
-    bool recurrent = false, inject = false;
+    bool recurrent = false, inject = false, fused_ok = true;
     int rows_cap = 0;
     std::vector<int> len;                  // tokens each slot's sequence has consumed
     std::map<std::pair<double, int>, float2*> ropes;
     // activations
-    float *x = nullptr, *emb = nullptr, *y = nullptr, *f32buf = nullptr, *ws = nullptr, *logits = nullptr;
+    float *x = nullptr, *x2 = nullptr, *emb = nullptr, *y = nullptr, *f32buf = nullptr, *ws = nullptr, *rec = nullptr, *logits = nullptr;
     T *h = nullptr, *proj = nullptr, *mixed = nullptr, *conv_out = nullptr, *xdbc = nullptr, *q_abs = nullptr, *o_lat = nullptr;
     T *kx = nullptr, *vx = nullptr;
     int* want_dev = nullptr;
@@ -113,13 +113,20 @@ private:
     int load_layer(const tllm_b200_mixed_layer& s, MixLayer<T>& L);
     int rope_table(double base, int dims, const float2** out);
     int layers_pass(const int* tokens, const StepGeo& g, float* taps, size_t tap_stride, cudaStream_t s);
+    int embed_rows(const int* tokens, int rows, cudaStream_t s);
+    int decode_step(const int* tokens, const StepGeo& g, float* out, cudaStream_t s);
+    bool fuses(const StepGeo& g) const { return g.seq_len == 1 && g.rows() <= kFewRows && fused_ok; }
     int head(const float* rows_x, const int* row_map, int n, float* out, cudaStream_t s);
     int mixer(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s);
-    int attention(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s);
+    int mixer_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s);
+    int attention_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s);
+    ScanArgs<T> scan_args(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g) const;
+    LinearArgs<T> gates_args(const MixLayer<T>& L, int n_rows) const;
+    int feed_forward(const MixLayer<T>& L, int n_rows, const GemvNorm* norm, cudaStream_t s);
     bool use_expanded(const LatentArgs<T>& a) const;
     int expanded(const MixLayer<T>& L, const RunState<T>& R, const LatentArgs<T>& a, cudaStream_t s);
-    int project(const Mat<T>& m, const T* in, int ldx, int k, void* out, int ldy, bool f32, int n_rows, cudaStream_t s,
-                const float* bias = nullptr, int act = kActNone)
+    LinearArgs<T> product(const Mat<T>& m, const T* in, int ldx, int k, void* out, int ldy, bool f32, int n_rows,
+                          const float* bias = nullptr, int act = kActNone) const
     {
         LinearArgs<T> l;
         l.w = m.p;
@@ -135,7 +142,12 @@ private:
         l.K = k;
         l.bias = bias;
         l.act = act;
-        return linear(l, s);
+        return l;
+    }
+    int project(const Mat<T>& m, const T* in, int ldx, int k, void* out, int ldy, bool f32, int n_rows, cudaStream_t s,
+                const float* bias = nullptr, int act = kActNone)
+    {
+        return linear(product(m, in, ldx, k, out, ldy, f32, n_rows, bias, act), s);
     }
 };
 
@@ -343,6 +355,11 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
     layers.resize(c.n_layers);
     for (int i = 0; i < c.n_layers; i++) TRY(load_layer(c.layers[i], layers[i]));
 
+    // a convolution in the tail of a GEMV needs a lane per tap; norm staging rows in shared memory
+    for (const MixLayer<T>& L : layers)
+        if (L.ch && !gemv_tail_fits<T>(w, L.taps)) fused_ok = false;
+    if (!gemv_norm_fits<T>(w)) fused_ok = false;
+
     const bool loop = c.loop_times != 1 && c.loop_stop > c.loop_start;
     for (int i = 0; i < c.n_layers;) {
         if (loop && i == c.loop_start) {
@@ -359,7 +376,7 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
     if (rows_cap < max_batch) rows_cap = max_batch;
     const size_t R = rows_cap;
     const int ar = rows_cap < kAbsorbRows ? rows_cap : kAbsorbRows;
-    size_t n_proj = 0, n_mixed = 0, n_ch = 0, n_x = 0, n_f32 = 0, n_q = 0, n_o = 0, n_ws = 0, n_k = 0, n_v = 0;
+    size_t n_proj = 0, n_mixed = 0, n_ch = 0, n_x = 0, n_f32 = 0, n_q = 0, n_o = 0, n_ws = 0, n_k = 0, n_v = 0, n_rec = 0;
     auto up = [](size_t& a, size_t b) { if (b > a) a = b; };
     for (const MixLayer<T>& L : layers) {
         up(n_mixed, L.ff);
@@ -375,10 +392,12 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
             up(n_ch, L.ch);
             up(n_x, L.x.rows);
             up(n_f32, L.type == TLLM_MIXER_SELECTIVE_SCAN ? L.ch : 2 * L.ch);
+            up(n_rec, scan_record_floats(1, rows_cap, L.ch, L.type == TLLM_MIXER_SELECTIVE_SCAN ? L.state : 1));
         }
     }
     auto some = [](size_t n) { return n ? n : (size_t)8; };
     TRY(dev_alloc(&x, R * w, true));
+    TRY(dev_alloc(&x2, (size_t)kFewRows * w, true));
     if (inject) TRY(dev_alloc(&emb, R * w, true));
     TRY(dev_alloc(&y, R * w, true));
     TRY(dev_alloc(&h, R * w, true));
@@ -390,6 +409,7 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
     TRY(dev_alloc(&q_abs, some(ar * n_q), true));
     TRY(dev_alloc(&o_lat, some(ar * n_o), true));
     TRY(dev_alloc(&ws, some(n_ws), true));
+    TRY(dev_alloc(&rec, some(n_rec), true));
     if (sizeof(T) == 2) {
         TRY(dev_alloc(&kx, some(max_seq * n_k), true));
         TRY(dev_alloc(&vx, some(max_seq * n_v), true));
@@ -480,11 +500,10 @@ int MixedDecoder<bf16>::expanded(const MixLayer<bf16>& L, const RunState<bf16>& 
 }
 
 template <typename T>
-int MixedDecoder<T>::attention(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s)
+int MixedDecoder<T>::attention_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s)
 {
     int st;
     const int rows = g.rows(), ldp = L.in.rows, H = L.heads, dq = L.dim + L.rot, dk = L.rank + L.rot;
-    TRY(project(L.in, h, w, w, proj, ldp, false, rows, s));
     LatentArgs<T> a;
     a.proj = proj;
     a.ld = ldp;
@@ -559,16 +578,72 @@ int MixedDecoder<T>::attention(const MixLayer<T>& L, const RunState<T>& R, const
             TRY(linear(v, s));
         }
     }
-    return project(L.out, mixed, L.out.ld, L.out.ld, y, w, true, rows, s);
+    return TLLM_OK;
 }
 
-// h -> y
 template <typename T>
-int MixedDecoder<T>::mixer(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s)
+ScanArgs<T> MixedDecoder<T>::scan_args(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g) const
 {
-    if (L.type == TLLM_MIXER_LATENT_ATTENTION) return attention(L, R, g, s);
+    ScanArgs<T> a;
+    a.x = conv_out;
+    a.bc = xdbc;
+    a.ld_bc = L.x.rows;
+    a.b_off = L.dt8;
+    a.c_off = L.dt8 + L.st8;
+    if (scan_takes_dt(g.seq_len, L.state)) {
+        a.dt_w = L.dt.p;
+        a.dt_bias = L.dt_bias;
+        a.dt_rank = L.dt8;
+    } else {
+        a.dt = f32buf;
+    }
+    a.z = proj + L.ch;
+    a.ld_z = 2 * L.ch;
+    a.a2 = L.a2;
+    a.d = L.d;
+    a.state = R.rec;
+    a.slot_stride = R.rec_slot;
+    a.y = mixed;
+    a.channels = L.ch;
+    a.states = L.state;
+    a.rec = rec;
+    a.g = g;
+    return a;
+}
+
+template <typename T>
+LinearArgs<T> MixedDecoder<T>::gates_args(const MixLayer<T>& L, int n_rows) const
+{
+    LinearArgs<T> l;
+    l.w = L.gates.p;
+    l.ldw = L.block;
+    l.w_rows = 2 * L.block;
+    l.x = conv_out;
+    l.ldx = L.ch;
+    l.x_batch = L.block;
+    l.y = f32buf;
+    l.ldy = 2 * L.ch;
+    l.y_batch = 2 * L.block;
+    l.y_f32 = true;
+    l.M = n_rows;
+    l.N = 2 * L.block;
+    l.K = L.block;
+    l.batch = L.blocks;
+    l.bias = L.gate_bias;
+    l.act = kActSigmoid;
+    return l;
+}
+
+// h -> mixed, the input of the output projection
+template <typename T>
+int MixedDecoder<T>::mixer_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s)
+{
     int st;
     const int rows = g.rows(), ch = L.ch;
+    if (L.type == TLLM_MIXER_LATENT_ATTENTION) {
+        TRY(project(L.in, h, w, w, proj, L.in.rows, false, rows, s));
+        return attention_inner(L, R, g, s);
+    }
     const bool scan = L.type == TLLM_MIXER_SELECTIVE_SCAN;
     TRY(project(L.in, h, w, w, proj, 2 * ch, false, rows, s, L.in_bias));
     ConvArgs<T> c;
@@ -586,61 +661,157 @@ int MixedDecoder<T>::mixer(const MixLayer<T>& L, const RunState<T>& R, const Ste
     TRY(launch_causal_conv<T>(c, s));
     if (scan) {
         TRY(project(L.x, conv_out, ch, ch, xdbc, L.x.rows, false, rows, s));
-        TRY(project(L.dt, xdbc, L.x.rows, L.dt8, f32buf, ch, true, rows, s, L.dt_bias, kActSoftplus));
-        ScanArgs<T> a;
-        a.x = conv_out;
-        a.dt = f32buf;
-        a.bc = xdbc;
-        a.ld_bc = L.x.rows;
-        a.b_off = L.dt8;
-        a.c_off = L.dt8 + L.st8;
-        a.z = proj + ch;
-        a.ld_z = 2 * ch;
-        a.a2 = L.a2;
-        a.d = L.d;
-        a.state = R.rec;
-        a.slot_stride = R.rec_slot;
-        a.y = mixed;
-        a.channels = ch;
-        a.states = L.state;
-        a.g = g;
-        TRY(launch_selective_scan<T>(a, s));
-    } else {
-        LinearArgs<T> l;
-        l.w = L.gates.p;
-        l.ldw = L.block;
-        l.w_rows = 2 * L.block;
-        l.x = conv_out;
-        l.ldx = ch;
-        l.x_batch = L.block;
-        l.y = f32buf;
-        l.ldy = 2 * ch;
-        l.y_batch = 2 * L.block;
-        l.y_f32 = true;
-        l.M = rows;
-        l.N = 2 * L.block;
-        l.K = L.block;
-        l.batch = L.blocks;
-        l.bias = L.gate_bias;
-        l.act = kActSigmoid;
-        TRY(linear(l, s));
-        GatedScanArgs<T> a;
-        a.u = conv_out;
-        a.gates = f32buf;
-        a.soft_lam = L.soft_lam;
-        a.c = L.decay;
-        a.y = proj;
-        a.ld_y = 2 * ch;
-        a.act = L.gate_act;
-        a.state = R.rec;
-        a.slot_stride = R.rec_slot;
-        a.out = mixed;
-        a.channels = ch;
-        a.block = L.block;
-        a.g = g;
-        TRY(launch_gated_scan<T>(a, s));
+        const ScanArgs<T> a = scan_args(L, R, g);
+        if (!a.dt_w) TRY(project(L.dt, xdbc, L.x.rows, L.dt8, f32buf, ch, true, rows, s, L.dt_bias, kActSoftplus));
+        return launch_selective_scan<T>(a, s);
     }
-    return project(L.out, mixed, L.out.ld, L.out.ld, y, w, true, rows, s);
+    TRY(linear(gates_args(L, rows), s));
+    GatedScanArgs<T> a;
+    a.u = conv_out;
+    a.gates = f32buf;
+    a.soft_lam = L.soft_lam;
+    a.c = L.decay;
+    a.y = proj;
+    a.ld_y = 2 * ch;
+    a.act = L.gate_act;
+    a.state = R.rec;
+    a.slot_stride = R.rec_slot;
+    a.out = mixed;
+    a.channels = ch;
+    a.block = L.block;
+    a.rec = rec;
+    a.g = g;
+    return launch_gated_scan<T>(a, s);
+}
+
+// h -> y
+template <typename T>
+int MixedDecoder<T>::mixer(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s)
+{
+    int st;
+    TRY(mixer_inner(L, R, g, s));
+    return project(L.out, mixed, L.out.ld, L.out.ld, y, w, true, g.rows(), s);
+}
+
+// h (or the residual chain staged in the first product) -> y
+template <typename T>
+int MixedDecoder<T>::feed_forward(const MixLayer<T>& L, int n_rows, const GemvNorm* norm, cudaStream_t s)
+{
+    int st;
+    LinearArgs<T> l;
+    l.w = L.gate_up.p;
+    l.ldw = w;
+    l.w_rows = 2 * L.ff;
+    l.x = h;
+    l.ldx = w;
+    l.y = mixed;
+    l.ldy = L.ff;
+    l.M = n_rows;
+    l.N = L.ff;
+    l.K = w;
+    l.act = L.ff_act;
+    l.glu = true;
+    TRY(norm ? launch_dense_gemv_fused<T>(l, *norm, GemvTail<T>(), s) : linear(l, s));
+    return project(L.down, mixed, L.ff, L.ff, y, w, true, n_rows, s);
+}
+
+// residual = table[token]; h = its norm for the first layer
+template <typename T>
+int MixedDecoder<T>::embed_rows(const int* tokens, int rows, cudaStream_t s)
+{
+    NormArgs<T> a;
+    a.x = x;
+    a.h = h;
+    a.rows = rows;
+    a.width = width;
+    a.w = w;
+    a.eps = eps;
+    a.table = embed.p;
+    a.tokens = tokens;
+    a.emb = inject ? emb : nullptr;
+    a.w_next = layers[order[0].first].norm1;
+    return launch_norm_chain<T>(a, s);
+}
+
+// One new token of each of a few sequences, logits of all of them: the residual chain is staged
+// in the products behind it, the convolution step and the gated recurrence step are tails of
+// the products in front of them.  Launches per layer without / with feed-forward: attention
+// 7 / 9, scan 4 / 6, recurrence 3 / 5.
+template <typename T>
+int MixedDecoder<T>::decode_step(const int* tokens, const StepGeo& g, float* out, cudaStream_t s)
+{
+    int st;
+    const int rows = g.rows();
+    TRY(embed_rows(tokens, rows, s));
+    float *cur = x, *next = x2;
+    const float* post = nullptr;
+    auto chain = [&](const float* w_next, const float* extra) {
+        GemvNorm f;
+        f.y = y;
+        f.w_post = post;
+        f.x_in = cur;
+        f.x_out = next;
+        f.extra = extra;
+        f.w_next = w_next;
+        f.width = width;
+        f.eps = eps;
+        std::swap(cur, next);
+        return f;
+    };
+    for (size_t r = 0; r < order.size(); r++) {
+        const MixLayer<T>& L = layers[order[r].first];
+        const RunState<T>& R = runs[r];
+        const GemvNorm f = r == 0 ? GemvNorm() : chain(L.norm1, order[r].second ? emb : nullptr);
+        const LinearArgs<T> in = product(L.in, h, w, w, proj, L.in.rows, false, rows, L.in_bias);
+        GemvTail<T> t;
+        if (L.type != TLLM_MIXER_LATENT_ATTENTION) {
+            const bool scan = L.type == TLLM_MIXER_SELECTIVE_SCAN;
+            t.kind = kTailConv;
+            t.lo = scan ? 0 : L.ch;
+            t.hi = t.lo + L.ch;
+            t.taps = L.taps;
+            t.act = scan ? kActSilu : kActNone;
+            t.w = L.conv;
+            t.bias = L.conv_bias;
+            t.carried = R.conv;
+            t.slot_stride = R.conv_slot;
+            t.first_slot = g.first_slot;
+            t.start_pos = g.start_pos;
+            t.pos_dev = g.pos_dev;
+            t.out = conv_out;
+            t.ld_out = L.ch;
+        }
+        TRY(launch_dense_gemv_fused<T>(in, f, t, s));
+        if (L.type == TLLM_MIXER_LATENT_ATTENTION) {
+            TRY(attention_inner(L, R, g, s));
+        } else if (L.type == TLLM_MIXER_SELECTIVE_SCAN) {
+            TRY(project(L.x, conv_out, L.ch, L.ch, xdbc, L.x.rows, false, rows, s));
+            const ScanArgs<T> a = scan_args(L, R, g);
+            if (!a.dt_w) TRY(project(L.dt, xdbc, L.x.rows, L.dt8, f32buf, L.ch, true, rows, s, L.dt_bias, kActSoftplus));
+            TRY(launch_selective_scan<T>(a, s));
+        } else {
+            LinearArgs<T> l = gates_args(L, rows);
+            l.N = L.block;
+            t.kind = kTailGate;
+            t.act = L.gate_act;
+            t.soft_lam = L.soft_lam;
+            t.decay = L.decay;
+            t.y = proj;
+            t.ld_y = 2 * L.ch;
+            t.state = R.rec;
+            t.slot_stride = R.rec_slot;
+            t.out = mixed;
+            TRY(launch_dense_gemv_fused<T>(l, GemvNorm(), t, s));
+        }
+        TRY(project(L.out, mixed, L.out.ld, L.out.ld, y, w, true, rows, s));
+        post = L.norm1b;
+        if (L.ff) {
+            const GemvNorm n2 = chain(L.norm2, nullptr);
+            TRY(feed_forward(L, rows, &n2, s));
+            post = L.norm2b;
+        }
+    }
+    return launch_dense_gemv_fused<T>(product(embed, h, w, w, out, vocab, true, rows), chain(final_norm, nullptr), GemvTail<T>(), s);
 }
 
 template <typename T>
@@ -655,14 +826,7 @@ int MixedDecoder<T>::layers_pass(const int* tokens, const StepGeo& g, float* tap
     base.width = width;
     base.w = w;
     base.eps = eps;
-    {
-        NormArgs<T> a = base;
-        a.table = embed.p;
-        a.tokens = tokens;
-        a.emb = inject ? emb : nullptr;
-        a.w_next = layers[order[0].first].norm1;
-        TRY(launch_norm_chain<T>(a, s));
-    }
+    TRY(embed_rows(tokens, rows, s));
     base.y = y;
     for (size_t r = 0; r < order.size(); r++) {
         const MixLayer<T>& L = layers[order[r].first];
@@ -673,21 +837,7 @@ int MixedDecoder<T>::layers_pass(const int* tokens, const StepGeo& g, float* tap
             a.w_post = post;
             a.w_next = L.norm2;
             TRY(launch_norm_chain<T>(a, s));
-            LinearArgs<T> l;
-            l.w = L.gate_up.p;
-            l.ldw = w;
-            l.w_rows = 2 * L.ff;
-            l.x = h;
-            l.ldx = w;
-            l.y = mixed;
-            l.ldy = L.ff;
-            l.M = rows;
-            l.N = L.ff;
-            l.K = w;
-            l.act = L.ff_act;
-            l.glu = true;
-            TRY(linear(l, s));
-            TRY(project(L.down, mixed, L.ff, L.ff, y, w, true, rows, s));
+            TRY(feed_forward(L, rows, nullptr, s));
             post = L.norm2b;
         }
         NormArgs<T> a = base;
@@ -729,6 +879,7 @@ int MixedDecoder<T>::forward(const int* tokens, int n, int start_pos, const int*
         StepGeo g;
         g.n_seq = batch;
         g.start_pos = start_pos;
+        if (fuses(g)) return decode_step(tokens, g, logits, s);
         TRY(layers_pass(tokens, g, nullptr, 0, s));
         return head(x, nullptr, batch, logits, s);
     }
@@ -739,6 +890,7 @@ int MixedDecoder<T>::forward(const int* tokens, int n, int start_pos, const int*
         g.first_slot = seq;
         g.start_pos = start_pos + t0;
         g.pos_dev = pos_dev;
+        if (n == 1 && fuses(g)) return decode_step(tokens, g, logits + (size_t)seq * vocab, s);
         TRY(layers_pass(tokens + t0, g, nullptr, 0, s));
         last = g.seq_len - 1;
     }
@@ -755,6 +907,12 @@ int MixedDecoder<T>::forward_logits(const int* tokens, int n, int start_pos, int
         g.seq_len = n - t0 < rows_cap ? n - t0 : rows_cap;
         g.first_slot = seq;
         g.start_pos = start_pos + t0;
+        if (n == 1 && !taps && fuses(g)) {                       // the step that generation runs
+            TRY(decode_step(tokens, g, logits + (size_t)seq * vocab, s));
+            for (int i = 0; i < n_want; i++)
+                cudaMemcpyAsync(out + (size_t)i * vocab, logits + (size_t)seq * vocab, (size_t)vocab * sizeof(float), cudaMemcpyDeviceToDevice, s);
+            return check_launch("decoder_forward_logits");
+        }
         TRY(layers_pass(tokens + t0, g, taps ? taps + (size_t)t0 * width : nullptr, (size_t)n * width, s));
         // runs of wanted tokens that lie in this portion
         for (int i = 0; i < n_want;) {

@@ -1,10 +1,11 @@
 // Residual chain, causal convolution and the two recurrences of the mixed-layer decoder.
 //
-// All of them are bound by memory or by the length of the sequence, not by arithmetic.  A
-// recurrence over many tokens is cut into time chunks inside one CTA: every chunk first runs
-// from a zero state and records its final state and its total decay, the chunks' true initial
-// states follow from those records, and a second pass over the chunk produces the outputs.
-// A single token takes the same code with one chunk.
+// A recurrence over many tokens is cut into time chunks: a first launch runs every chunk but the
+// last from a zero state and records its final state and its total decay, a second one derives
+// each chunk's true initial state from the records before it and produces the outputs.  The
+// first launch also copies the carried state into the records: in the second one the last chunk
+// overwrites it while others may not have started.  Short portions and single tokens are one
+// chunk and need the second launch only.
 #include "launch.cuh"
 #include "mixers.cuh"
 
@@ -154,7 +155,7 @@ causal_conv_kernel(const ConvArgs<T> a, int chunk)
         }
 #pragma unroll
         for (int j = 1; j < TAPS; j++) win[j] = input(t0 - TAPS + j);
-#pragma unroll 4
+#pragma unroll 8
         for (int t = t0; t < t1; t++) {
 #pragma unroll
             for (int j = 0; j + 1 < TAPS; j++) win[j] = win[j + 1];
@@ -186,174 +187,214 @@ causal_conv_kernel(const ConvArgs<T> a, int chunk)
 // ---------------------------------------------------------------------------
 // Selective scan
 // ---------------------------------------------------------------------------
-constexpr int kScanCh = 16;          // channels per CTA
-constexpr int kScanMaxThreads = 512;
-constexpr int kScanU = 4;            // tokens loaded together
+constexpr int kScanThreads = 128;
+constexpr int kMaxChunks = 16, kMinChunk = 32;     // time chunks; tokens of a chunk at least
 
-// A channel is served by `lpc` lanes with NS states each; lane l holds states l * NS ...
-template <typename T, int NS>
-__global__ void __launch_bounds__(kScanMaxThreads)
-selective_scan_kernel(const ScanArgs<T> a, int lpc, int nchunk)
+// a state of many entries per channel makes records expensive: fewer chunks
+inline int time_chunks(int n, int states)
 {
-    extern __shared__ __align__(16) float smem[];
-    pdl_launch_dependents();
-    const int per = kScanCh * lpc, chunk = threadIdx.x / per, rem = threadIdx.x - chunk * per;
-    const int cl = rem / lpc, l = rem - cl * lpc;
-    const int c_raw = blockIdx.x * kScanCh + cl;
-    const bool live = c_raw < a.channels;
-    const int c = live ? c_raw : a.channels - 1, b = blockIdx.y;
-    const int n = a.g.seq_len, s0 = l * NS, st8 = (a.states + 7) & ~7;
-    const int len = (n + nchunk - 1) / nchunk, t0 = min(n, chunk * len), t1 = min(n, t0 + len);
-    float* sl = smem;                                          // [nchunk][kScanCh][lpc * NS] chunk states
-    float* sd = smem + (size_t)nchunk * kScanCh * lpc * NS;    // [nchunk][kScanCh] sums of dt
+    const int c = n / kMinChunk, most = states > 1 ? kMaxChunks : 2 * kMaxChunks;
+    return c < 1 ? 1 : c > most ? most : c;
+}
 
+// A channel is served by `lpc` lanes with NS states each; lane l holds states l * NS ...  B and C
+// of TT tokens are staged in shared memory as floats, the channel's own inputs in registers.
+// Records of chunk k: [b][k][state][channel] final states, then [b][k][channel] sums of dt.
+// ONE: lpc is 1.  DT: the step sizes are computed here too (few tokens: one launch less).
+template <typename T, int NS, int TT, bool OUT, bool ONE, bool DT>
+__global__ void __launch_bounds__(kScanThreads)
+selective_scan_kernel(const ScanArgs<T> a, int lanes, int nchunk)
+{
+    const int lpc = ONE ? 1 : lanes;
+    extern __shared__ __align__(16) float bcs[];               // [TT][2][sp]
+    pdl_launch_dependents();
+    const int sp = lpc * NS, cpb = kScanThreads / lpc;
+    const int tid = threadIdx.x, cl = tid / lpc, l = tid - cl * lpc, s0 = l * NS;
+    const int c_raw = blockIdx.x * cpb + cl, chunk = blockIdx.y, b = blockIdx.z;
+    const bool live = c_raw < a.channels;
+    const int c = live ? c_raw : a.channels - 1;
+    const int n = a.g.seq_len, len = (n + nchunk - 1) / nchunk, t0 = min(n, chunk * len), t1 = min(n, t0 + len);
     float A[NS], S[NS];
 #pragma unroll
     for (int j = 0; j < NS; j++) {
         A[j] = (s0 + j < a.states) ? a.a2[(size_t)c * a.states + s0 + j] : 0.f;
         S[j] = 0.f;
     }
-    const float D = a.d ? a.d[c] : 0.f;
+    const float D = (OUT && a.d) ? a.d[c] : 0.f;
+    const float dt_bias = (DT && a.dt_bias) ? a.dt_bias[c] : 0.f;
     pdl_wait();
-    const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
-    const size_t row0 = (size_t)b * n;
-    const float* dtp = a.dt + row0 * a.channels + c;
-    const T* xp = a.x + row0 * a.channels + c;
-    const T* bp = a.bc + row0 * a.ld_bc + a.b_off + s0;
-    const T* cp = a.bc + row0 * a.ld_bc + a.c_off + s0;
+    const size_t row0 = (size_t)b * n, CH = a.channels;
+    const float* dtp = a.dt + row0 * CH + c;
+    const T* xp = a.x + row0 * CH + c;
     const T* zp = a.z ? a.z + row0 * a.ld_z + c : nullptr;
-    T* yp = a.y + row0 * a.channels + c;
+    T* yp = a.y + row0 * CH + c;
     float* stp = a.state + (size_t)(a.g.first_slot + b) * a.slot_stride + (size_t)c * a.states;
-
-    // tokens [t, t + kScanU) of the chunk; with_y: also the outputs.  Past the end dt = x = 0,
-    // which leaves the state as it is.
-    float sum_dt = 0.f;
-    auto group = [&](int t, bool with_y) {
-        float dt[kScanU], x[kScanU], Bv[kScanU][NS], Cv[kScanU][NS];
+    float* rec = a.rec + (size_t)b * nchunk * a.states * CH + c;
+    float* rec_dt = a.rec + (size_t)a.g.n_seq * nchunk * a.states * CH + (size_t)b * nchunk * CH + c;
+    const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
+    // the carried state as slot nchunk - 1 of the records (free: that chunk records nothing)
+    float* carried = rec + (size_t)(nchunk - 1) * a.states * CH;
+    if (!OUT && chunk == 0 && live) {
 #pragma unroll
-        for (int u = 0; u < kScanU; u++) {
-            const int tt = t + u;
-            const bool in = tt < t1;
-            dt[u] = in ? dtp[(size_t)tt * a.channels] : 0.f;
-            x[u] = in ? to_f<T>(xp[(size_t)tt * a.channels]) : 0.f;
+        for (int j = 0; j < NS; j++)
+            if (s0 + j < a.states) carried[(size_t)(s0 + j) * CH] = fresh ? 0.f : stp[s0 + j];
+    }
+    if (OUT) {
+#pragma unroll
+        for (int j = 0; j < NS; j++)
+            if (s0 + j < a.states) S[j] = nchunk > 1 ? carried[(size_t)(s0 + j) * CH] : fresh ? 0.f : stp[s0 + j];
+        for (int k = 0; k < chunk; k++) {
+            const float d = rec_dt[(size_t)k * CH];
+#pragma unroll
+            for (int j = 0; j < NS; j++)
+                if (s0 + j < a.states) S[j] = fmaf(exp2_neg(d * A[j]), S[j], rec[((size_t)k * a.states + s0 + j) * CH]);
+        }
+    }
+    float sum_dt = 0.f;
+    for (int t = t0; t < t1; t += TT) {
+        float dt[TT], x[TT], z[OUT ? TT : 1];
+#pragma unroll
+        for (int u = 0; u < TT; u++) {                         // past the end dt = x = 0: the state stays
+            const bool in = t + u < t1;
+            if (DT) {
+                float p = 0.f;
+                const uint4* wp = reinterpret_cast<const uint4*>(a.dt_w + (size_t)c * a.dt_rank);
+                const uint4* vp = reinterpret_cast<const uint4*>(a.bc + (row0 + min(t + u, n - 1)) * a.ld_bc + a.dt_off);
+                for (int i = l; i < a.dt_rank / Vec16<T>::n; i += lpc) {
+                    float wf[Vec16<T>::n], vf[Vec16<T>::n];
+                    Vec16<T>::unpack(__ldg(wp + i), wf);
+                    Vec16<T>::unpack(vp[i], vf);
+#pragma unroll
+                    for (int j = 0; j < Vec16<T>::n; j++) p = fmaf(wf[j], vf[j], p);
+                }
+                for (int o = lpc >> 1; o > 0; o >>= 1) p += __shfl_xor_sync(0xffffffffu, p, o);
+                dt[u] = in ? softplus_f(p + dt_bias) : 0.f;
+            } else {
+                dt[u] = in ? dtp[(size_t)(t + u) * CH] : 0.f;
+            }
+            x[u] = in ? to_f<T>(xp[(size_t)(t + u) * CH]) : 0.f;
+            if (OUT) z[u] = (in && zp) ? to_f<T>(zp[(size_t)(t + u) * a.ld_z]) : 0.f;
+        }
+        __syncthreads();
+        for (int i = tid; i < TT * 2 * sp; i += kScanThreads) {
+            const int u = i / (2 * sp), r = i - u * 2 * sp, s = r < sp ? r : r - sp;
+            const bool in = t + u < t1 && s < a.states;
+            bcs[i] = in ? to_f<T>(a.bc[(row0 + t + u) * a.ld_bc + (r < sp ? a.b_off : a.c_off) + s]) : 0.f;
+        }
+        __syncthreads();
+        float y[TT];
+#pragma unroll
+        for (int u = 0; u < TT; u++) {
+            const float dx = dt[u] * x[u];
+            const float* Bp = bcs + u * 2 * sp + s0;
+            float y0 = 0.f, y1 = 0.f;
+            if (!OUT) sum_dt += dt[u];
 #pragma unroll
             for (int j = 0; j < NS; j += 4) {
-                float4 v = make_float4(0.f, 0.f, 0.f, 0.f), w = v;
-                if (in && s0 + j < st8) {
-                    v = load4(bp + (size_t)tt * a.ld_bc + j);
-                    if (with_y) w = load4(cp + (size_t)tt * a.ld_bc + j);
+                const float4 Bv = load4(Bp + j);
+                S[j] = fmaf(exp2_neg(dt[u] * A[j]), S[j], dx * Bv.x);
+                S[j + 1] = fmaf(exp2_neg(dt[u] * A[j + 1]), S[j + 1], dx * Bv.y);
+                S[j + 2] = fmaf(exp2_neg(dt[u] * A[j + 2]), S[j + 2], dx * Bv.z);
+                S[j + 3] = fmaf(exp2_neg(dt[u] * A[j + 3]), S[j + 3], dx * Bv.w);
+                if (OUT) {
+                    const float4 Cv = load4(Bp + sp + j);
+                    y0 = fmaf(S[j], Cv.x, y0);
+                    y1 = fmaf(S[j + 1], Cv.y, y1);
+                    y0 = fmaf(S[j + 2], Cv.z, y0);
+                    y1 = fmaf(S[j + 3], Cv.w, y1);
                 }
-                Bv[u][j] = v.x; Bv[u][j + 1] = v.y; Bv[u][j + 2] = v.z; Bv[u][j + 3] = v.w;
-                Cv[u][j] = w.x; Cv[u][j + 1] = w.y; Cv[u][j + 2] = w.z; Cv[u][j + 3] = w.w;
             }
+            y[u] = y0 + y1;
         }
-        float y[kScanU];
+        if (OUT) {
+            if (!ONE)
+                for (int o = lpc >> 1; o > 0; o >>= 1) {
 #pragma unroll
-        for (int u = 0; u < kScanU; u++) {
-            const float dx = dt[u] * x[u];
-            sum_dt += dt[u];
-            y[u] = 0.f;
+                    for (int u = 0; u < TT; u++) y[u] += __shfl_xor_sync(0xffffffffu, y[u], o);
+                }
+            if (live && l == 0) {
 #pragma unroll
-            for (int j = 0; j < NS; j++) {
-                S[j] = fmaf(exp2f(dt[u] * A[j]), S[j], dx * Bv[u][j]);
-                y[u] = fmaf(S[j], Cv[u][j], y[u]);
-            }
-        }
-        if (with_y) {
-#pragma unroll
-            for (int u = 0; u < kScanU; u++)
-                for (int o = lpc >> 1; o > 0; o >>= 1) y[u] += __shfl_xor_sync(0xffffffffu, y[u], o);
-#pragma unroll
-            for (int u = 0; u < kScanU; u++) {
-                const int tt = t + u;
-                if (live && tt < t1 && l == u % lpc) {
+                for (int u = 0; u < TT; u++) {
                     float v = fmaf(D, x[u], y[u]);
-                    if (zp) {
-                        const float zz = to_f<T>(zp[(size_t)tt * a.ld_z]);
-                        v *= zz * sigmoid_f(zz);
-                    }
-                    yp[(size_t)tt * a.channels] = from_f<T>(v);
+                    if (zp) v *= z[u] * sigmoid_f(z[u]);
+                    if (t + u < t1) yp[(size_t)(t + u) * CH] = from_f<T>(v);
                 }
             }
         }
-    };
-
-    if (nchunk > 1) {
-        for (int t = t0; t < t1; t += kScanU) group(t, false);
-#pragma unroll
-        for (int j = 0; j < NS; j++) sl[((size_t)chunk * kScanCh + cl) * (lpc * NS) + s0 + j] = S[j];
-        if (l == 0) sd[chunk * kScanCh + cl] = sum_dt;
-        __syncthreads();
     }
+    if (!live) return;
+    if (OUT) {
+        if (chunk == nchunk - 1) {
 #pragma unroll
-    for (int j = 0; j < NS; j++) S[j] = (!fresh && s0 + j < a.states) ? stp[s0 + j] : 0.f;
-    for (int k = 0; k < chunk; k++) {
-        const float d = sd[k * kScanCh + cl];
+            for (int j = 0; j < NS; j++)
+                if (s0 + j < a.states) stp[s0 + j] = S[j];
+        }
+    } else {
 #pragma unroll
         for (int j = 0; j < NS; j++)
-            S[j] = fmaf(exp2f(d * A[j]), S[j], sl[((size_t)k * kScanCh + cl) * (lpc * NS) + s0 + j]);
-    }
-    if (nchunk > 1) __syncthreads();          // every chunk has read the carried state
-    for (int t = t0; t < t1; t += kScanU) group(t, true);
-    if (live && t0 < n && t1 == n) {
-#pragma unroll
-        for (int j = 0; j < NS; j++)
-            if (s0 + j < a.states) stp[s0 + j] = S[j];
+            if (s0 + j < a.states) rec[((size_t)chunk * a.states + s0 + j) * CH] = S[j];
+        if (l == 0) rec_dt[(size_t)chunk * CH] = sum_dt;
     }
 }
 
 // ---------------------------------------------------------------------------
-// Real-gated linear recurrence
+// Real-gated linear recurrence: one thread per channel and time chunk
 // ---------------------------------------------------------------------------
-constexpr int kGateCh = 32;          // channels per CTA = lanes of a warp; a warp is a time chunk
-constexpr int kGateMaxChunks = 32;
+constexpr int kGateThreads = 64;
 
-template <typename T>
-__global__ void __launch_bounds__(kGateCh * kGateMaxChunks)
-gated_scan_kernel(const GatedScanArgs<T> a)
+template <typename T, bool OUT>
+__global__ void __launch_bounds__(kGateThreads)
+gated_scan_kernel(const GatedScanArgs<T> a, int nchunk)
 {
-    __shared__ float sl[kGateMaxChunks][kGateCh], sa[kGateMaxChunks][kGateCh];
+    constexpr int TT = 8;
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31, chunk = threadIdx.x >> 5, nchunk = blockDim.x >> 5;
-    const int c_raw = blockIdx.x * kGateCh + lane, b = blockIdx.y;
-    const bool live = c_raw < a.channels;
-    const int c = live ? c_raw : a.channels - 1;
+    const int c = blockIdx.x * kGateThreads + threadIdx.x, chunk = blockIdx.y, b = blockIdx.z;
     const int n = a.g.seq_len, len = (n + nchunk - 1) / nchunk, t0 = min(n, chunk * len), t1 = min(n, t0 + len);
-    const float kc = -a.c * a.soft_lam[c];
+    const float kc = c < a.channels ? -a.c * a.soft_lam[c] : 0.f;
     pdl_wait();
-    const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
-    const size_t row0 = (size_t)b * n;
+    if (c >= a.channels) return;
+    const size_t row0 = (size_t)b * n, CH = a.channels;
     const int blk = c / a.block, ci = c - blk * a.block;
-    const float* rp = a.gates + row0 * 2 * a.channels + (size_t)blk * 2 * a.block + ci;
-    const T* up = a.u + row0 * a.channels + c;
+    const float* rp = a.gates + row0 * 2 * CH + (size_t)blk * 2 * a.block + ci;
+    const T* up = a.u + row0 * CH + c;
     const T* yp = a.y + row0 * a.ld_y + c;
-    T* op = a.out + row0 * a.channels + c;
+    T* op = a.out + row0 * CH + c;
     float* stp = a.state + (size_t)(a.g.first_slot + b) * a.slot_stride + c;
-
+    float* rec = a.rec + (size_t)b * nchunk * CH + c;
+    float* rec_log = a.rec + (size_t)(a.g.n_seq + b) * nchunk * CH + c;
     float S = 0.f, sum_log = 0.f;
-    auto step = [&](int t) {
-        const float r = rp[(size_t)t * 2 * a.channels], i = rp[(size_t)t * 2 * a.channels + a.block];
-        const float log_a = kc * r;
-        sum_log += log_a;
-        // 1 - a^2 through expm1: no cancellation when a is close to one
-        S = fmaf(expf(log_a), S, sqrtf(-expm1f(2.f * log_a)) * i * to_f<T>(up[(size_t)t * a.channels]));
-    };
-    if (nchunk > 1) {
-#pragma unroll 4
-        for (int t = t0; t < t1; t++) step(t);
-        sl[chunk][lane] = S;
-        sa[chunk][lane] = sum_log;
-        __syncthreads();
+    const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
+    float* carried = rec + (size_t)(nchunk - 1) * CH;          // see selective_scan_kernel
+    if (!OUT && chunk == 0) *carried = fresh ? 0.f : *stp;
+    if (OUT) {
+        S = nchunk > 1 ? *carried : fresh ? 0.f : *stp;
+        for (int k = 0; k < chunk; k++) S = fmaf(expf(rec_log[(size_t)k * CH]), S, rec[(size_t)k * CH]);
     }
-    S = fresh ? 0.f : *stp;
-    for (int k = 0; k < chunk; k++) S = fmaf(expf(sa[k][lane]), S, sl[k][lane]);
-    if (nchunk > 1) __syncthreads();          // every chunk has read the carried state
-#pragma unroll 4
-    for (int t = t0; t < t1; t++) {
-        step(t);
-        if (live) op[(size_t)t * a.channels] = from_f<T>(S * apply_act(a.act, to_f<T>(yp[(size_t)t * a.ld_y])));
+    for (int t = t0; t < t1; t += TT) {
+        float r[TT], i[TT], u[TT], y[OUT ? TT : 1];
+#pragma unroll
+        for (int j = 0; j < TT; j++) {
+            const bool in = t + j < t1;                        // past the end r = u = 0: the state stays
+            r[j] = in ? rp[(size_t)(t + j) * 2 * CH] : 0.f;
+            i[j] = in ? rp[(size_t)(t + j) * 2 * CH + a.block] : 0.f;
+            u[j] = in ? to_f<T>(up[(size_t)(t + j) * CH]) : 0.f;
+            if (OUT) y[j] = in ? to_f<T>(yp[(size_t)(t + j) * a.ld_y]) : 0.f;
+        }
+        if (OUT) apply_act_n(a.act, y);
+#pragma unroll
+        for (int j = 0; j < TT; j++) {
+            const float log_a = kc * r[j], A = expf(log_a);
+            if (!OUT) sum_log += log_a;
+            S = fmaf(A, S, sqrtf(one_minus_exp(2.f * log_a, A * A)) * i[j] * u[j]);
+            if (OUT && t + j < t1) op[(size_t)(t + j) * CH] = from_f<T>(S * y[j]);
+        }
     }
-    if (live && t0 < n && t1 == n) *stp = S;
+    if (OUT) {
+        if (chunk == nchunk - 1) *stp = S;
+    } else {
+        rec[(size_t)chunk * CH] = S;
+        rec_log[(size_t)chunk * CH] = sum_log;
+    }
 }
 
 }  // namespace
@@ -389,26 +430,51 @@ int launch_causal_conv(const ConvArgs<T>& a, cudaStream_t stream)
     }
 }
 
+size_t scan_record_floats(int n_seq, int seq_len, int channels, int states)
+{
+    const int nchunk = time_chunks(seq_len, states);
+    return nchunk > 1 ? (size_t)n_seq * nchunk * channels * (states + 1) : 0;
+}
+
+namespace {
+template <typename T, int NS, int TT, bool ONE, bool DT>
+int scan_passes(const ScanArgs<T>& a, int lpc, int nchunk, cudaStream_t stream)
+{
+    const int cpb = kScanThreads / lpc;
+    const size_t smem = (size_t)TT * 2 * lpc * NS * sizeof(float);
+    const auto first = selective_scan_kernel<T, NS, TT, false, ONE, DT>, second = selective_scan_kernel<T, NS, TT, true, ONE, DT>;
+    if (smem > 48 * 1024) {
+        cudaFuncSetAttribute(first, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(second, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    }
+    const unsigned gx = (a.channels + cpb - 1) / cpb;
+    if (nchunk > 1) {
+        // the last chunk's final state is nobody's initial state
+        const int st = launch_pdl("selective_scan", first, dim3(gx, nchunk - 1, a.g.n_seq), dim3(kScanThreads), smem, stream, a, lpc, nchunk);
+        if (st) return st;
+    }
+    return launch_pdl("selective_scan", second, dim3(gx, nchunk, a.g.n_seq), dim3(kScanThreads), smem, stream, a, lpc, nchunk);
+}
+}  // namespace
+
+bool scan_takes_dt(int seq_len, int states) { return seq_len <= 4 && states <= 128; }
+
 template <typename T>
 int launch_selective_scan(const ScanArgs<T>& a, cudaStream_t stream)
 {
     if (a.g.rows() == 0) return TLLM_OK;
-    const int ns = a.states <= 128 ? 4 : a.states <= 256 ? 8 : 16;
     if (a.states < 1 || a.states > 512 || a.channels < 1) return fail(TLLM_ERR_SHAPE, "selective_scan: channels=%d states=%d (1..512)", a.channels, a.states);
-    if (a.ld_bc % 4 || a.b_off % 4 || a.c_off % 4) return fail(TLLM_ERR_ALIGN, "selective_scan: B and C must start on multiples of 4");
+    const int nchunk = time_chunks(a.g.seq_len, 2);
+    if (nchunk > 1 && !a.rec) return fail(TLLM_ERR_NULL, "selective_scan: no record buffer");
+    // few tokens: more lanes per channel; many: more states per lane (fewer instructions per state)
+    const int ns = scan_takes_dt(a.g.seq_len, a.states) ? 4 : 16;
+    if (a.dt_w && (ns != 4 || a.dt_rank % 8 || a.dt_off % 8 || a.ld_bc % 8))
+        return fail(TLLM_ERR_SHAPE, "selective_scan: dt_rank=%d with %d tokens", a.dt_rank, a.g.seq_len);
     int lpc = 1;
     while (lpc * ns < a.states) lpc *= 2;
-    int nchunk = kScanMaxThreads / (kScanCh * lpc);
-    if (nchunk > a.g.seq_len / 16) nchunk = a.g.seq_len / 16;      // at least 16 tokens per chunk
-    if (nchunk < 1) nchunk = 1;
-    // records of the chunks; one chunk needs none
-    const size_t smem = nchunk > 1 ? (size_t)nchunk * kScanCh * (lpc * ns + 1) * sizeof(float) : 0;
-    const dim3 grid((a.channels + kScanCh - 1) / kScanCh, a.g.n_seq), block(kScanCh * lpc * nchunk);
-    switch (ns) {
-        case 4: return launch_pdl("selective_scan", selective_scan_kernel<T, 4>, grid, block, smem, stream, a, lpc, nchunk);
-        case 8: return launch_pdl("selective_scan", selective_scan_kernel<T, 8>, grid, block, smem, stream, a, lpc, nchunk);
-        default: return launch_pdl("selective_scan", selective_scan_kernel<T, 16>, grid, block, smem, stream, a, lpc, nchunk);
-    }
+    if (ns == 4)
+        return a.dt_w ? scan_passes<T, 4, 1, false, true>(a, lpc, nchunk, stream) : scan_passes<T, 4, 1, false, false>(a, lpc, nchunk, stream);
+    return lpc == 1 ? scan_passes<T, 16, 8, true, false>(a, lpc, nchunk, stream) : scan_passes<T, 16, 8, false, false>(a, lpc, nchunk, stream);
 }
 
 template <typename T>
@@ -416,11 +482,14 @@ int launch_gated_scan(const GatedScanArgs<T>& a, cudaStream_t stream)
 {
     if (a.g.rows() == 0) return TLLM_OK;
     if (a.channels < 1 || a.block < 1 || a.channels % a.block) return fail(TLLM_ERR_SHAPE, "gated_scan: channels=%d block=%d", a.channels, a.block);
-    int nchunk = a.g.seq_len / 16;
-    if (nchunk > kGateMaxChunks) nchunk = kGateMaxChunks;
-    if (nchunk < 1) nchunk = 1;
-    return launch_pdl("gated_scan", gated_scan_kernel<T>, dim3((a.channels + kGateCh - 1) / kGateCh, a.g.n_seq), dim3(kGateCh * nchunk),
-                      0, stream, a);
+    const int nchunk = time_chunks(a.g.seq_len, 1);
+    if (nchunk > 1 && !a.rec) return fail(TLLM_ERR_NULL, "gated_scan: no record buffer");
+    const unsigned gx = (a.channels + kGateThreads - 1) / kGateThreads;
+    if (nchunk > 1) {
+        const int st = launch_pdl("gated_scan", gated_scan_kernel<T, false>, dim3(gx, nchunk - 1, a.g.n_seq), dim3(kGateThreads), 0, stream, a, nchunk);
+        if (st) return st;
+    }
+    return launch_pdl("gated_scan", gated_scan_kernel<T, true>, dim3(gx, nchunk, a.g.n_seq), dim3(kGateThreads), 0, stream, a, nchunk);
 }
 
 #define TLLM_INSTANTIATE(T)                                                \

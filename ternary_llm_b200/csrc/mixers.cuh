@@ -67,6 +67,10 @@ struct ScanArgs {
     const float* dt = nullptr; // [rows, channels]
     const T* bc = nullptr;     // [rows, ld_bc]: B from column b_off, C from column c_off
     int ld_bc = 0, b_off = 0, c_off = 0;
+    // instead of dt (scan_takes_dt): dt = softplus(dt_w . bc[dt_off ..] + dt_bias)
+    const T* dt_w = nullptr;   // [channels, dt_rank]
+    const float* dt_bias = nullptr;
+    int dt_rank = 0, dt_off = 0;
     const T* z = nullptr;      // [rows, ld_z], null = no gate
     int ld_z = 0;
     const float* a2 = nullptr; // [channels, states], A / ln 2
@@ -75,8 +79,12 @@ struct ScanArgs {
     size_t slot_stride = 0;
     T* y = nullptr;            // [rows, channels]
     int channels = 0, states = 0;
+    float* rec = nullptr;      // scan_record_floats, when the sequence is cut into time chunks
     StepGeo g;
 };
+// records of the time chunks of a scan over n_seq x seq_len tokens (0: one chunk, none needed)
+bool scan_takes_dt(int seq_len, int states);
+size_t scan_record_floats(int n_seq, int seq_len, int channels, int states);
 template <typename T>
 int launch_selective_scan(const ScanArgs<T>& a, cudaStream_t stream);
 
@@ -94,6 +102,7 @@ struct GatedScanArgs {
     size_t slot_stride = 0;
     T* out = nullptr;              // [rows, channels]
     int channels = 0, block = 0;   // block: m (padded)
+    float* rec = nullptr;          // scan_record_floats with one state
     StepGeo g;
 };
 template <typename T>
