@@ -192,6 +192,21 @@ def test_greedy_generation_through_the_graph_replayed_loop(dtype):
     dec.close()
 
 
+def test_generation_from_the_command_line(tmp_path):
+    cfg, raw, toks, _, _ = setup("one_layer_loop", n=60)
+    write_model(str(tmp_path / "m"), cfg, raw)
+    r = subprocess.run([sys.executable, "-m", "ternary_llm_b200.generate", "--model", str(tmp_path / "m"), "--tokens",
+                        ",".join(map(str, toks[:12])), "--steps", "9", "--dtype", "float32"], capture_output=True, text=True, timeout=600, cwd=ROOT)
+    assert r.returncode == 0, r.stderr[-2000:]
+    dec = tl.Decoder(str(tmp_path / "m"), dtype="float32", max_seq_len=64)
+    tok, want = int(dec.forward(ids(toks[:12]), 0).argmax()), []
+    for i in range(9):
+        want.append(tok)
+        tok = int(dec.forward(ids([tok]), 12 + i).argmax())
+    assert [int(v) for v in r.stdout.strip().splitlines()[-1].split(",")] == want
+    dec.close()
+
+
 def test_prompt_longer_than_one_pass_through_the_layers():
     """A prompt of more tokens than the activation buffers hold goes through in portions, wanted
     logits from each; decode steps far behind it read the whole cache."""

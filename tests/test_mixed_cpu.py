@@ -12,7 +12,7 @@ import pytest
 
 from oracle import mixed_oracle as O
 from tests import _mixed as M
-from ternary_llm_b200 import _lib, mixed, models, trace
+from ternary_llm_b200 import _lib, generate, mixed, models, trace
 from ternary_llm_b200 import safetensors_io as st
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -235,3 +235,11 @@ def test_trace_replay_positions_slots_and_files(tmp_path, monkeypatch):
     with pytest.raises(RuntimeError, match="slots"):
         t = trace.SlotTable(1)
         t.slot("a"), t.slot("b")
+
+
+def test_generation_command_line_arguments(capsys):
+    assert generate.parse_tokens("5, 17,3") == [5, 17, 3]
+    for bad in (["--model", "m", "--tokens", "a"], ["--model", "m", "--tokens", "-1"], ["--tokens", "1"], ["--model", "m", "--tokens", "1", "--dtype", "int8"]):
+        with pytest.raises(SystemExit):
+            generate.main(bad)
+    capsys.readouterr()
