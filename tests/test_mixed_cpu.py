@@ -92,7 +92,7 @@ def test_a_mistake_in_any_mechanism_shows_in_the_logits(mistake, monkeypatch):
     elif mistake == "scan_skip":
         W = {k: (v * 0 if k.endswith(".D") else v) for k, v in W.items()}
     elif mistake == "lam":
-        W = {k: (v + 1 if k.endswith("lam") else v) for k, v in W.items()}
+        W = {k: (v + 3 if k.endswith("lam") else v) for k, v in W.items()}
     elif mistake == "inject":
         monkeypatch.setattr(O, "run_order", lambda c, f=O.run_order: [(i, False) for i, _ in f(c)])
     elif mistake == "post_norm":
