@@ -118,7 +118,14 @@ __device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.0f, 1.
 
 // z * sigmoid(2u) with u = sqrt(2/pi) (z + 0.044715 z^3): the same number as 0.5 z (1 + tanh(u))
 __device__ __forceinline__ float gelu_tanh_f(float z) { return z * sigmoid_f(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// max(z, 0) + log(1 + e), e = exp(-|z|): log(1 + e) = 2 artanh(e / (2 + e)) as its power series,
+// whose argument is at most 1/3 (the first term left out is below 2^-25 of the sum)
+__device__ __forceinline__ float softplus_f(float z)
+{
+    const float e = expf(-fabsf(z)), s = __fdividef(e, 2.f + e), q = s * s;
+    const float p = 1.f + q * (1.f / 3 + q * (1.f / 5 + q * (1.f / 7 + q * (1.f / 9 + q * (1.f / 11 + q * (1.f / 13))))));
+    return fmaxf(z, 0.f) + 2.f * s * p;
+}
 
 // 2^x for x <= 0, flushed to zero below the normal range
 __device__ __forceinline__ float exp2_neg(float x)
@@ -135,6 +142,15 @@ __device__ __forceinline__ float one_minus_exp(float t, float e)
     const float p = -t * (1.f + t * (1.f / 2) * (1.f + t * (1.f / 3) * (1.f + t * (1.f / 4) * (1.f + t * (1.f / 5) * (1.f + t * (1.f / 6))))));
     return t > -0.25f ? p : 1.f - e;
 }
+
+// e^t for t <= 0 given an approximation e: close to one, where the errors of a product of many
+// decays would add up, from the series (rounded once)
+__device__ __forceinline__ float decay_exp(float t, float e) { return 1.f - one_minus_exp(t, e); }
+
+// 2^x, x <= 0; the exact 32-bit mode takes the series near zero
+template <typename T> __device__ __forceinline__ float decay_exp2(float x);
+template <> __device__ __forceinline__ float decay_exp2<bf16>(float x) { return exp2_neg(x); }
+template <> __device__ __forceinline__ float decay_exp2<float>(float x) { return decay_exp(0.69314718055994531f * x, exp2_neg(x)); }
 
 // the switch stays outside the loop over the elements
 template <int N>

@@ -248,7 +248,7 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
             if (TAIL == kTailGate) {
                 const float* b = a.bias + (size_t)z * 2 * a.N;
                 const float r = sigmoid_f(res[0][m] + b[n]), i = sigmoid_f(res[1][m] + b[a.N + n]);
-                const float log_a = tw * r, A = expf(log_a);
+                const float log_a = tw * r, A = decay_exp(log_a, expf(log_a));
                 const float S = fmaf(A, hist[m], sqrtf(one_minus_exp(2.f * log_a, A * A)) * i * to_f<T>(xs[(size_t)m * a.K + n]));
                 t.state[(size_t)(t.first_slot + m) * t.slot_stride + ch] = S;
                 t.out[(size_t)m * t.ld_out + ch] = from_f<T>(S * apply_act(t.act, to_f<T>(t.y[(size_t)m * t.ld_y + ch])));

@@ -159,7 +159,7 @@ causal_conv_kernel(const ConvArgs<T> a, int chunk)
         for (int t = t0; t < t1; t++) {
 #pragma unroll
             for (int j = 0; j + 1 < TAPS; j++) win[j] = win[j + 1];
-            win[TAPS - 1] = input(t);
+            win[TAPS - 1] = ld2(x + (size_t)t * a.ldx);
             float v0 = b0, v1 = b1;
 #pragma unroll
             for (int j = 0; j < TAPS; j++) {
@@ -202,7 +202,7 @@ inline int time_chunks(int n, int states)
 // Records of chunk k: [b][k][state][channel] final states, then [b][k][channel] sums of dt.
 // ONE: lpc is 1.  DT: the step sizes are computed here too (few tokens: one launch less).
 template <typename T, int NS, int TT, bool OUT, bool ONE, bool DT>
-__global__ void __launch_bounds__(kScanThreads)
+__global__ void __launch_bounds__(kScanThreads, 4)
 selective_scan_kernel(const ScanArgs<T> a, int lanes, int nchunk)
 {
     const int lpc = ONE ? 1 : lanes;
@@ -243,19 +243,43 @@ selective_scan_kernel(const ScanArgs<T> a, int lanes, int nchunk)
 #pragma unroll
         for (int j = 0; j < NS; j++)
             if (s0 + j < a.states) S[j] = nchunk > 1 ? carried[(size_t)(s0 + j) * CH] : fresh ? 0.f : stp[s0 + j];
+#pragma unroll 2
         for (int k = 0; k < chunk; k++) {
             const float d = rec_dt[(size_t)k * CH];
 #pragma unroll
             for (int j = 0; j < NS; j++)
-                if (s0 + j < a.states) S[j] = fmaf(exp2_neg(d * A[j]), S[j], rec[((size_t)k * a.states + s0 + j) * CH]);
+                if (s0 + j < a.states) S[j] = fmaf(decay_exp2<T>(d * A[j]), S[j], rec[((size_t)k * a.states + s0 + j) * CH]);
         }
     }
     float sum_dt = 0.f;
-    for (int t = t0; t < t1; t += TT) {
-        float dt[TT], x[TT], z[OUT ? TT : 1];
+    // inputs of the next TT tokens, requested one tile ahead; B and C too when a channel is one
+    // lane (a handful of values per thread then)
+    constexpr int NB = ONE ? TT * 2 * NS / kScanThreads : 1;
+    float dt_n[TT], x_n[TT], z_n[OUT ? TT : 1], bc_n[NB];
+    auto bc_at = [&](int t, int i) -> float {
+        const int u = i / (2 * sp), r = i - u * 2 * sp, s = r < sp ? r : r - sp;
+        return (t + u < t1 && s < a.states) ? to_f<T>(a.bc[(row0 + t + u) * a.ld_bc + (r < sp ? a.b_off : a.c_off) + s]) : 0.f;
+    };
+    auto request = [&](int t) {
 #pragma unroll
         for (int u = 0; u < TT; u++) {                         // past the end dt = x = 0: the state stays
             const bool in = t + u < t1;
+            if (!DT) dt_n[u] = in ? dtp[(size_t)(t + u) * CH] : 0.f;
+            x_n[u] = in ? to_f<T>(xp[(size_t)(t + u) * CH]) : 0.f;
+            if (OUT) z_n[u] = (in && zp) ? to_f<T>(zp[(size_t)(t + u) * a.ld_z]) : 0.f;
+        }
+        if (ONE) {
+#pragma unroll
+            for (int j = 0; j < NB; j++) bc_n[j] = bc_at(t, tid + j * kScanThreads);
+        }
+    };
+    request(t0);
+    for (int t = t0; t < t1; t += TT) {
+        float dt[TT], x[TT], z[OUT ? TT : 1];
+#pragma unroll
+        for (int u = 0; u < TT; u++) {
+            x[u] = x_n[u];
+            if (OUT) z[u] = z_n[u];
             if (DT) {
                 float p = 0.f;
                 const uint4* wp = reinterpret_cast<const uint4*>(a.dt_w + (size_t)c * a.dt_rank);
@@ -268,20 +292,20 @@ selective_scan_kernel(const ScanArgs<T> a, int lanes, int nchunk)
                     for (int j = 0; j < Vec16<T>::n; j++) p = fmaf(wf[j], vf[j], p);
                 }
                 for (int o = lpc >> 1; o > 0; o >>= 1) p += __shfl_xor_sync(0xffffffffu, p, o);
-                dt[u] = in ? softplus_f(p + dt_bias) : 0.f;
+                dt[u] = t + u < t1 ? softplus_f(p + dt_bias) : 0.f;
             } else {
-                dt[u] = in ? dtp[(size_t)(t + u) * CH] : 0.f;
+                dt[u] = dt_n[u];
             }
-            x[u] = in ? to_f<T>(xp[(size_t)(t + u) * CH]) : 0.f;
-            if (OUT) z[u] = (in && zp) ? to_f<T>(zp[(size_t)(t + u) * a.ld_z]) : 0.f;
         }
         __syncthreads();
-        for (int i = tid; i < TT * 2 * sp; i += kScanThreads) {
-            const int u = i / (2 * sp), r = i - u * 2 * sp, s = r < sp ? r : r - sp;
-            const bool in = t + u < t1 && s < a.states;
-            bcs[i] = in ? to_f<T>(a.bc[(row0 + t + u) * a.ld_bc + (r < sp ? a.b_off : a.c_off) + s]) : 0.f;
+        if (ONE) {
+#pragma unroll
+            for (int j = 0; j < NB; j++) bcs[tid + j * kScanThreads] = bc_n[j];
+        } else {
+            for (int i = tid; i < TT * 2 * sp; i += kScanThreads) bcs[i] = bc_at(t, i);
         }
         __syncthreads();
+        if (t + TT < t1) request(t + TT);
         float y[TT];
 #pragma unroll
         for (int u = 0; u < TT; u++) {
@@ -292,10 +316,10 @@ selective_scan_kernel(const ScanArgs<T> a, int lanes, int nchunk)
 #pragma unroll
             for (int j = 0; j < NS; j += 4) {
                 const float4 Bv = load4(Bp + j);
-                S[j] = fmaf(exp2_neg(dt[u] * A[j]), S[j], dx * Bv.x);
-                S[j + 1] = fmaf(exp2_neg(dt[u] * A[j + 1]), S[j + 1], dx * Bv.y);
-                S[j + 2] = fmaf(exp2_neg(dt[u] * A[j + 2]), S[j + 2], dx * Bv.z);
-                S[j + 3] = fmaf(exp2_neg(dt[u] * A[j + 3]), S[j + 3], dx * Bv.w);
+                S[j] = fmaf(decay_exp2<T>(dt[u] * A[j]), S[j], dx * Bv.x);
+                S[j + 1] = fmaf(decay_exp2<T>(dt[u] * A[j + 1]), S[j + 1], dx * Bv.y);
+                S[j + 2] = fmaf(decay_exp2<T>(dt[u] * A[j + 2]), S[j + 2], dx * Bv.z);
+                S[j + 3] = fmaf(decay_exp2<T>(dt[u] * A[j + 3]), S[j + 3], dx * Bv.w);
                 if (OUT) {
                     const float4 Cv = load4(Bp + sp + j);
                     y0 = fmaf(S[j], Cv.x, y0);
@@ -368,6 +392,7 @@ gated_scan_kernel(const GatedScanArgs<T> a, int nchunk)
     if (!OUT && chunk == 0) *carried = fresh ? 0.f : *stp;
     if (OUT) {
         S = nchunk > 1 ? *carried : fresh ? 0.f : *stp;
+#pragma unroll 8
         for (int k = 0; k < chunk; k++) S = fmaf(expf(rec_log[(size_t)k * CH]), S, rec[(size_t)k * CH]);
     }
     for (int t = t0; t < t1; t += TT) {
@@ -383,7 +408,7 @@ gated_scan_kernel(const GatedScanArgs<T> a, int nchunk)
         if (OUT) apply_act_n(a.act, y);
 #pragma unroll
         for (int j = 0; j < TT; j++) {
-            const float log_a = kc * r[j], A = expf(log_a);
+            const float log_a = kc * r[j], A = decay_exp(log_a, expf(log_a));
             if (!OUT) sum_log += log_a;
             S = fmaf(A, S, sqrtf(one_minus_exp(2.f * log_a, A * A)) * i[j] * u[j]);
             if (OUT && t + j < t1) op[(size_t)(t + j) * CH] = from_f<T>(S * y[j]);
