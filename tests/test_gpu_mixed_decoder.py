@@ -89,7 +89,7 @@ def test_residual_after_every_layer_run(dtype):
 def test_a_far_token_is_found_again():
     """Attention whose query reaches a token hundreds of positions back, through the prompt and
     through the decode kernels: the logits change when that one token changes, as the oracle's do."""
-    cfg = M.config([M.attention(heads=2, dim=16, rot_dim=2, vdim=32, kv_rank=32, base=1e6, scale=2.0)], width=48, vocab=61)
+    cfg = M.config([M.attention(heads=2, dim=16, rot_dim=2, vdim=32, kv_rank=32, base=2e5, scale=2.0)], width=48, vocab=61)
     raw, W = M.finder_model(cfg, 77)
     toks = np.random.default_rng(3).integers(0, 60, 400).astype(np.int32)
     toks[3] = 60                              # the only token of its kind

@@ -152,7 +152,7 @@ def plain_attention(q, k, v, scale, sink, start):
 
 
 @pytest.mark.parametrize("dt", list(DT))
-@pytest.mark.parametrize("H,rank,rot", [(1, 8, 8), (3, 40, 8), (8, 64, 16), (20, 128, 0), (16, 512, 64), (4, 896, 128), (2, 1104, 8)])
+@pytest.mark.parametrize("H,rank,rot", [(1, 8, 8), (3, 40, 8), (7, 56, 24), (20, 128, 0), (16, 512, 64), (4, 896, 128), (2, 1104, 8)])
 def test_absorbed_attention(H, rank, rot, dt):
     """Edges: the first position, the borders of the 64-position tiles and of the splits, the
     query's own position, and the one after it (which must not be seen)."""
@@ -213,7 +213,7 @@ def test_absorbed_attention_of_several_sequences_is_each_alone(dt):
         close(o[b:b + 1], one.double().cpu().numpy(), REL[dt], f"sequence {b}")
 
 
-@pytest.mark.parametrize("H,dim,rot,vdim", [(1, 8, 8, 8), (3, 24, 8, 40), (2, 32, 16, 80), (4, 128, 64, 128), (2, 64, 0, 256), (2, 200, 56, 24)])
+@pytest.mark.parametrize("H,dim,rot,vdim", [(1, 8, 8, 8), (3, 24, 8, 40), (2, 40, 24, 72), (4, 128, 64, 128), (2, 64, 0, 256), (2, 200, 56, 24)])
 def test_expanded_attention(H, dim, rot, vdim):
     rng = np.random.default_rng(dim)
     dt, rank = "bfloat16", 16
