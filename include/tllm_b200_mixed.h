@@ -1,16 +1,18 @@
 /*
  * tllm_b200_mixed.h -- decoders whose layers are a list of different token mixers (latent
- * attention, selective scan, real-gated linear recurrence) with dense BF16 weights.
+ * attention, selective scan, real-gated linear recurrence, grouped-query attention, linear
+ * attention, gated delta rule, or two of the last three side by side) with dense or routed
+ * feed-forwards and BF16 weights.
  *
  * No counterpart in the reference engine, whose Transformer (src/transformer.cpp) has one kind
  * of layer.  A decoder made here is driven by the same entry points as every other model of
  * the library (tllm_b200_layer.h: tllm_b200_decoder_forward, _forward_seq, _forward_batch,
  * _generate, _reset, _destroy); logits are FP32.
  *
- * A sequence's state is a cache of one latent row per position for latent attention and a
- * fixed-size recurrent state otherwise.  A call with start_pos 0 starts a new sequence in its
+ * A sequence's state is a cache of one row per position for attention (with a chunk mask: a ring
+ * of as many rows as a chunk and a pass need) and a fixed-size recurrent state otherwise.  A call with start_pos 0 starts a new sequence in its
  * slot; with recurrent layers, every other call must continue where the slot's sequence ended
- * (TLLM_ERR_SHAPE otherwise).
+ * (TLLM_ERR_SHAPE otherwise), and so it must with a ring of cache rows.
  */
 #ifndef TLLM_B200_MIXED_H
 #define TLLM_B200_MIXED_H
@@ -24,23 +26,27 @@ extern "C" {
 enum {
     TLLM_MIXER_LATENT_ATTENTION = 1,
     TLLM_MIXER_SELECTIVE_SCAN = 2,   /* Mamba */
-    TLLM_MIXER_GATED_RECURRENCE = 3  /* Griffin's RG-LRU block */
+    TLLM_MIXER_GATED_RECURRENCE = 3, /* Griffin's RG-LRU block */
+    TLLM_MIXER_ATTENTION = 4,        /* grouped-query softmax attention */
+    TLLM_MIXER_LINEAR_ATTENTION = 5, /* S <- decay S + k v^T, o = S^T q, a constant decay per head */
+    TLLM_MIXER_DELTA_RULE = 6        /* S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q */
 };
-enum { TLLM_ACT_NONE = 0, TLLM_ACT_GELU_TANH = 1, TLLM_ACT_SILU = 2 };
+enum { TLLM_ACT_NONE = 0, TLLM_ACT_GELU_TANH = 1, TLLM_ACT_SILU = 2, TLLM_ACT_SIGMOID = 4 };
 
 /* Tensors of a layer: device pointers to BF16 data, row-major [out, in]; copied (and padded)
  * at creation.  Unused entries are NULL. */
 enum {
-    TLLM_T_NORM1 = 0,   /* [width], before the mixer */
+    TLLM_T_NORM1 = 0,   /* [width], before the mixer (norm_after_sum: of the sum behind it) */
     TLLM_T_NORM1B,      /* [width], after the mixer; NULL: plain residual add */
-    TLLM_T_NORM2,       /* [width], before the feed-forward */
+    TLLM_T_NORM2,       /* [width], before the feed-forward (norm_after_sum: of the sum behind it) */
     TLLM_T_NORM2B,      /* [width], after it; NULL: plain residual add */
-    TLLM_T_GATE,        /* [ff, width] */
-    TLLM_T_UP,          /* [ff, width] */
-    TLLM_T_DOWN,        /* [width, ff] */
+    TLLM_T_GATE,        /* [ff, width], or [experts, ff, width] */
+    TLLM_T_UP,          /* [ff, width], or [experts, ff, width] */
+    TLLM_T_DOWN,        /* [width, ff], or [experts, width, ff] */
     TLLM_T_OUT,         /* [width, mixer output] */
     /* latent attention */
-    TLLM_T_Q,           /* [heads * (dim + rot_dim), width], per head unrotated then rotated */
+    TLLM_T_Q,           /* [heads * (dim + rot_dim), width], per head unrotated then rotated; attention and
+                           linear attention: [heads * dim, width]; delta rule: [kv_heads * dim, width] */
     TLLM_T_KV_DOWN,     /* [kv_rank + rot_dim, width]: latent, then the shared rotated key part */
     TLLM_T_KV_NORM,     /* [kv_rank] */
     TLLM_T_K_UP,        /* [heads * dim, kv_rank] */
@@ -64,6 +70,20 @@ enum {
     TLLM_T_RI,
     TLLM_T_RI_BIAS,
     TLLM_T_LAM,         /* recurrence: [channels] */
+    /* attention, linear attention, delta rule */
+    TLLM_T_K,           /* [kv_heads * dim, width] */
+    TLLM_T_V,           /* attention: [kv_heads * vdim, width], else [heads * vdim, width] */
+    TLLM_T_Q_NORM,      /* attention: [dim], NULL: no norm */
+    TLLM_T_K_NORM,
+    TLLM_T_Q_CONV,      /* delta rule: [kv_heads * dim, taps] */
+    TLLM_T_K_CONV,
+    TLLM_T_V_CONV,      /* delta rule: [heads * vdim, taps] */
+    TLLM_T_STEP,        /* delta rule: [heads, width], before the sigmoid */
+    TLLM_T_DECAY,       /* delta rule: [heads, width]; with TLLM_T_DT_BIAS and TLLM_T_A_LOG [heads] */
+    TLLM_T_MIX_NORM,    /* of the output -- linear attention: [heads * vdim]; delta rule: [vdim], every head alone */
+    TLLM_T_MIX_GATE,    /* linear attention, delta rule: [heads * vdim, width], multiplies the normed output */
+    /* feed-forward */
+    TLLM_T_ROUTER,      /* [experts, width] */
     TLLM_T_COUNT
 };
 
@@ -76,8 +96,17 @@ typedef struct tllm_b200_mixed_layer {
     int state, dt_rank;                              /* scan */
     int blocks;                                      /* recurrence */
     float decay;                                     /* recurrence: c in log a = -c r softplus(lam) */
-    int gate_act;                                    /* recurrence: activation of the gating branch */
+    int gate_act;                                    /* activation of the gating branch or the output gate */
     int ff, ff_act;                                  /* ff = 0: no feed-forward */
+    int experts, top;                                /* experts > 0: mixture, `top` per token; ff is an expert's */
+    int kv_heads;                                    /* attention, delta rule */
+    int chunk;                                       /* attention: only positions of the same chunk; 0: all */
+    int in_act;                                      /* linear attention: of q, k, v; delta rule: of the convolutions */
+    float out_scale;                                 /* of the mixer's output (attention, linear attention, delta rule) */
+    const float* head_decay;                         /* linear attention: host array [heads] */
+    /* a second mixer of the three that reads the same input and is added (its own `beside`, feed-forward
+     * and layer norms are ignored), or NULL */
+    const struct tllm_b200_mixed_layer* beside;
     const void* t[TLLM_T_COUNT];
 } tllm_b200_mixed_layer;
 
@@ -88,7 +117,11 @@ typedef struct tllm_b200_mixed_desc {
      * pass with its own cache or state; loop_inject: the embedding output is added to the
      * residual before the first layer of every pass but the first */
     int loop_start, loop_stop, loop_times, loop_inject;
-    const void* embedding;   /* BF16 [vocab, width], also the output head */
+    int norm_after_sum;      /* x = norm(residual_scale * x + sublayer(x)) instead of x + sublayer(norm(x)) */
+    float residual_scale;
+    float logit_softcap;     /* logits = cap * tanh(logits / cap); 0: none */
+    const void* embedding;   /* BF16 [vocab, width] */
+    const void* head;        /* BF16 [vocab, width], NULL: the embedding */
     const void* final_norm;  /* BF16 [width] */
     const tllm_b200_mixed_layer* layers; /* host array of n_layers */
 } tllm_b200_mixed_desc;

@@ -73,7 +73,7 @@ SIGNATURES = {
     "tllm_b200_latent_attention_expanded": (_int, [_vp] * 7 + [_int] * 5 + [ctypes.c_float] + [_int] * 3 + [_vp]),
 }
 
-TENSORS_PER_LAYER = 31      # TLLM_T_COUNT
+TENSORS_PER_LAYER = 43      # TLLM_T_COUNT
 
 
 class TernaryWeightDesc(ctypes.Structure):
@@ -103,15 +103,18 @@ class MixedLayerDesc(ctypes.Structure):
     _fields_ = [(n, _int) for n in ("type", "heads", "dim", "rot_dim", "rot_dims", "vdim", "kv_rank")] + \
                [("scale", ctypes.c_float), ("rot_base", ctypes.c_double)] + \
                [(n, _int) for n in ("channels", "taps", "state", "dt_rank", "blocks")] + \
-               [("decay", ctypes.c_float)] + [(n, _int) for n in ("gate_act", "ff", "ff_act")] + \
-               [("t", _vp * TENSORS_PER_LAYER)]
+               [("decay", ctypes.c_float)] + \
+               [(n, _int) for n in ("gate_act", "ff", "ff_act", "experts", "top", "kv_heads", "chunk", "in_act")] + \
+               [("out_scale", ctypes.c_float), ("head_decay", ctypes.POINTER(ctypes.c_float)), ("beside", _vp),
+                ("t", _vp * TENSORS_PER_LAYER)]
 
 
 class MixedDesc(ctypes.Structure):
     """tllm_b200_mixed_desc."""
     _fields_ = [(n, _int) for n in ("vocab_size", "width", "n_layers", "max_seq_len")] + [("norm_eps", ctypes.c_float)] + \
                [(n, _int) for n in ("loop_start", "loop_stop", "loop_times", "loop_inject")] + \
-               [("embedding", _vp), ("final_norm", _vp), ("layers", ctypes.POINTER(MixedLayerDesc))]
+               [("norm_after_sum", _int), ("residual_scale", ctypes.c_float), ("logit_softcap", ctypes.c_float)] + \
+               [("embedding", _vp), ("head", _vp), ("final_norm", _vp), ("layers", ctypes.POINTER(MixedLayerDesc))]
 
 
 class TllmError(RuntimeError):

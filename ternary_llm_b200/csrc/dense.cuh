@@ -2,6 +2,8 @@
 // activations, FP32 accumulation.  Every matrix is packed at load time so that rows start on
 // 16-byte boundaries: `ld` elements per row, a multiple of 8, padding columns zero.
 #pragma once
+#include <climits>
+
 #include <cuda_bf16.h>
 
 #include "common.cuh"
@@ -11,7 +13,7 @@ namespace tllm {
 using bf16 = __nv_bfloat16;
 
 // element-wise function applied to (product + bias)
-enum Act { kActNone = 0, kActGeluTanh = 1, kActSilu = 2, kActSoftplus = 3, kActSigmoid = 4 };
+enum Act { kActNone = 0, kActGeluTanh = 1, kActSilu = 2, kActSoftplus = 3, kActSigmoid = 4, kActSoftcap = 5 };
 
 // y[m, z, n] = post(sum_k W[z, n, k] x[m, z, k]),  z = 0..batch-1
 template <typename T>
@@ -26,6 +28,16 @@ struct LinearArgs {
     int M = 0, N = 0, K = 0, batch = 1;   // K: a multiple of 8 (padded)
     const float* bias = nullptr; // [batch * N], null = none
     int act = kActNone;
+    float act_param = 0.f;       // softcap: the cap
+    // features [act_lo, act_hi) take the activation; features from f32_from on go to y2 as FP32
+    // (row stride ldy2, feature f32_from first); all three multiples of 64
+    int act_lo = 0, act_hi = INT_MAX, f32_from = INT_MAX;
+    float* y2 = nullptr;
+    int ldy2 = 0;
+    // rows in groups with a matrix each (entries of w, w_rows apart): 128 rows from 128 i on use
+    // entry group[i], i < *groups (both on the device); entries: matrices in w
+    const int *group = nullptr, *groups = nullptr;
+    int entries = 0;
     // glu: w holds N gate rows followed by N up rows; y = act(gate) * up
     bool glu = false;
     const T* gate = nullptr;     // y *= sigmoid(gate[m * gate_ld + z])
@@ -33,16 +45,19 @@ struct LinearArgs {
 };
 
 // ---- what a GEMV of a decode step takes over from its neighbours --------------------------
-// Staging: x = norm(x_in + post-normed y (+ extra)) computed by every CTA instead of a launch of
-// its own (the step of the residual chain in mixers.cuh); the sum goes to x_out, a different
-// buffer than x_in, because every CTA reads the old one while the first writes.
+// Staging: the step of the residual chain in mixers.cuh computed by every CTA instead of a launch
+// of its own; the new residual goes to x_out, a different buffer than x_in, because every CTA
+// reads the old one while the first writes.
 struct GemvNorm {
     const float* y = nullptr;       // [M, K]; null: no norm staging, the vectors come from x
+    float alpha = 1.f;
     const float* w_post = nullptr;  // null: plain add
+    const float* w_sum = nullptr;   // null: the sum is not normed
     const float* x_in = nullptr;
     float* x_out = nullptr;
     const float* extra = nullptr;
-    const float* w_next = nullptr;
+    const float* w_next = nullptr;  // null: the vectors are the residual itself
+    void* h_out = nullptr;          // the vectors, T [M, K], or null
     int width = 0;                  // true width (K is padded)
     float eps = 0.f;
 };
@@ -71,6 +86,8 @@ struct GemvTail {
     int ld_out = 0;
 };
 
+constexpr int kGroupRows = 128;     // rows that share an entry of a grouped product
+
 // vectors one after the other against streamed weights; at most 8 vectors per pass
 template <typename T>
 int launch_dense_gemv(const LinearArgs<T>& a, cudaStream_t stream);
@@ -80,7 +97,7 @@ int launch_dense_gemv_fused(const LinearArgs<T>& a, const GemvNorm& norm, const 
 // the tails need this many lanes per row
 template <typename T>
 bool gemv_tail_fits(int k, int taps);
-// norm staging of up to 8 rows of this width
+// norm staging of up to 8 rows of this width, with two norm weights
 template <typename T>
 bool gemv_norm_fits(int k);
 int launch_dense_gemm_tcgen05(const LinearArgs<bf16>& a, cudaStream_t stream);
@@ -95,7 +112,7 @@ int linear(const LinearArgs<float>& a, cudaStream_t stream);
 // (i * rp + a), column (j * cp + b) = fn(src row (i * rs + a), column (j * c + b)); everything
 // else of dst stays as it is (zero).  transpose: each row group is transposed (gc must be 1):
 // dst row (i * rp + b), column a.
-enum PackFn { kPackCopy = 0, kPackNegExpLog2e = 1, kPackSoftplus = 2 };   // applied once at load, in double
+enum PackFn { kPackCopy = 0, kPackNegExpLog2e = 1, kPackSoftplus = 2, kPackNegExp = 3 };   // applied once at load, in double
 struct PackSpec {
     int gr = 1, r = 1, rs = 1, rp = 1;
     int gc = 1, c = 1, cp = 1;
@@ -154,7 +171,7 @@ template <> __device__ __forceinline__ float decay_exp2<float>(float x) { return
 
 // the switch stays outside the loop over the elements
 template <int N>
-__device__ __forceinline__ void apply_act_n(int act, float (&v)[N])
+__device__ __forceinline__ void apply_act_n(int act, float (&v)[N], float param = 0.f)
 {
     switch (act) {
         case kActGeluTanh:
@@ -173,13 +190,17 @@ __device__ __forceinline__ void apply_act_n(int act, float (&v)[N])
 #pragma unroll
             for (int i = 0; i < N; i++) v[i] = sigmoid_f(v[i]);
             break;
+        case kActSoftcap:
+#pragma unroll
+            for (int i = 0; i < N; i++) v[i] = param * tanhf(v[i] / param);
+            break;
         default: break;
     }
 }
-__device__ __forceinline__ float apply_act(int act, float z)
+__device__ __forceinline__ float apply_act(int act, float z, float param = 0.f)
 {
     float v[1] = {z};
-    apply_act_n<1>(act, v);
+    apply_act_n<1>(act, v, param);
     return v[0];
 }
 

@@ -50,6 +50,10 @@ struct DenseEpi {
     int M, N, K, x_batch, w_rows;
     int mt, nt, tiles;             // tiles along the tokens, along the features, in all
     int act, glu, y_f32, vec, bias_vec;
+    float act_param;
+    int act_lo, act_hi, f32_from, ldy2, vec2;
+    float* y2;
+    const int *group, *groups;
     int* err;
 };
 
@@ -86,13 +90,6 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
     auto empty = [&](int s) { return bar0 + 8u * (kStages + s); };
     auto acc_full = [&](int i) { return bar0 + 8u * (2 * kStages + i); };
     auto acc_empty = [&](int i) { return bar0 + 8u * (2 * kStages + 2 + i); };
-    // tile -> first token, first feature, batch entry; tokens vary fastest (neighbours share W)
-    auto where = [&](int tile, int& m0, int& n0, int& z) {
-        m0 = (tile % a.mt) * kTok;
-        tile /= a.mt;
-        n0 = (tile % a.nt) * outs;
-        z = tile / a.nt;
-    };
 
     if (tid == 0) {
         for (int s = 0; s < kStages; s++) {
@@ -119,16 +116,24 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
     volatile int* abortp = &abort_flag;
     int never = 0;
     pdl_wait();
+    // tile -> first token, first feature, batch entry; tokens vary fastest (neighbours share W)
+    const int mt = a.group ? min(*a.groups, a.mt) : a.mt, tiles = a.group ? mt * a.nt : a.tiles;
+    auto where = [&](int tile, int& m0, int& n0, int& z) {
+        m0 = (tile % mt) * kTok;
+        tile /= mt;
+        n0 = (tile % a.nt) * outs;
+        z = tile / a.nt;
+    };
 
     if (warp == 0) {
         // ---------------- TMA producer ----------------
         if (lane == 0) {
             int it = 0;                                  // stages filled so far, over all tiles
             bool ok = true;
-            for (int tile = blockIdx.x; ok && tile < a.tiles; tile += gridDim.x) {
+            for (int tile = blockIdx.x; ok && tile < tiles; tile += gridDim.x) {
                 int m0, n0, z;
                 where(tile, m0, n0, z);
-                const int wr0 = z * a.w_rows + n0, wr1 = a.glu ? wr0 + a.N : wr0 + TN / 2;
+                const int wr0 = (a.group ? a.group[m0 / kTok] : z) * a.w_rows + n0, wr1 = a.glu ? wr0 + a.N : wr0 + TN / 2;
                 for (int k = 0; k < nk; k++, it++) {
                     const int s = it % kStages;
                     if (!mbar_wait(empty(s), ((it / kStages) & 1) ^ 1, abortp)) {
@@ -154,7 +159,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
             const uint32_t idesc = idesc_bf16<TN>();
             int it = 0, i = 0;                           // i: tiles of this CTA so far
             bool ok = true;
-            for (int tile = blockIdx.x; ok && tile < a.tiles; tile += gridDim.x, i++) {
+            for (int tile = blockIdx.x; ok && tile < tiles; tile += gridDim.x, i++) {
                 const int buf = i & 1;
                 if (!mbar_wait(acc_empty(buf), ((i >> 1) & 1) ^ 1, abortp)) {
                     abort_flag = 1;
@@ -189,9 +194,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
         const uint32_t lane_base = tmem + ((uint32_t)row0 << 16);
         uint32_t* st = reinterpret_cast<uint32_t*>(smem + (size_t)kStages * kStage) + ew * 32 * kStageLd;
         const int sr = lane >> 2, sw = (lane & 3) * 4;   // row (of eight) and words this lane stores
-        const int wcols = a.y_f32 ? 1 : 2;               // columns per staged word
         int i = 0;
-        for (int tile = blockIdx.x; tile < a.tiles; tile += gridDim.x, i++) {
+        for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x, i++) {
             const int buf = i & 1;
             if (!__all_sync(0xffffffffu, mbar_wait(acc_full(buf), (i >> 1) & 1, abortp))) {
                 abort_flag = 1;
@@ -207,6 +211,10 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
             if (mrow < a.M)
 #pragma unroll 1
             for (int c = half * 32; c < ncols; c += 64) {
+                // 32 columns go one way: the limits of the activation and of y2 are multiples of 64
+                const bool second = n0 + c >= a.f32_from, y_f32 = a.y_f32 || second;
+                const int act = n0 + c >= a.act_lo && n0 + c < a.act_hi && !second ? a.act : kActNone;
+                const int wcols = y_f32 ? 1 : 2;         // columns per staged word
                 uint32_t v[32];
                 __syncwarp();
                 tmem_ld32(acc + c, v);
@@ -217,7 +225,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
                     for (int j = 0; j < 32; j++) f[j] = __uint_as_float(v[j]);
-                    apply_act_n<32>(a.act, f);
+                    apply_act_n<32>(act, f);
 #pragma unroll
                     for (int j = 0; j < 32; j++) f[j] *= __uint_as_float(u[j]);
                 } else {
@@ -241,7 +249,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
                                 if (c + j < ncols) f[j] += __ldg(bp + j);
                         }
                     }
-                    apply_act_n<32>(a.act, f);
+                    apply_act_n<32>(act, f, a.act_param);
                     if (a.gate) {
 #pragma unroll
                         for (int j = 0; j < 32; j++) f[j] *= hg;
@@ -250,7 +258,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
                 // through shared memory, 16 words of a row at a time: FP32 in two halves, BF16 at once
 #pragma unroll
                 for (int part = 0; part < 2; part++) {
-                    if (part == 1 && !a.y_f32) break;
+                    if (part == 1 && !y_f32) break;
                     __syncwarp();
 #pragma unroll
                     for (int j = 0; j < 4; j++) {
@@ -258,7 +266,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
 #pragma unroll
                         for (int q = 0; q < 4; q++) {
                             const int e = 4 * j + q;
-                            if (a.y_f32) {
+                            if (y_f32) {
                                 w[q] = __float_as_uint(f[part * 16 + e]);
                             } else {
                                 const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * e], f[2 * e + 1]);
@@ -270,20 +278,21 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
                     __syncwarp();
                     const int col = c + part * 16 + sw * wcols;      // first of this lane's columns inside the tile
                     if (col < ncols) {
-                        const bool vec = a.vec && col + 4 * wcols <= ncols;
+                        const bool vec = (second ? a.vec2 : a.vec) && col + 4 * wcols <= ncols;
 #pragma unroll
                         for (int r = 0; r < 4; r++) {
                             const int rr = r * 8 + sr, m = mrow + rr;
                             if (m >= a.M) break;
                             const uint4 t = *reinterpret_cast<const uint4*>(st + rr * kStageLd + sw);
-                            const size_t o = (size_t)m * a.ldy + (size_t)z * a.y_batch + n0 + col;
+                            const size_t o = second ? (size_t)m * a.ldy2 + n0 + col - a.f32_from
+                                                    : (size_t)m * a.ldy + (size_t)z * a.y_batch + n0 + col;
                             if (vec) {
-                                if (a.y_f32) *reinterpret_cast<uint4*>(static_cast<float*>(a.y) + o) = t;
+                                if (y_f32) *reinterpret_cast<uint4*>((second ? a.y2 : static_cast<float*>(a.y)) + o) = t;
                                 else *reinterpret_cast<uint4*>(static_cast<bf16*>(a.y) + o) = t;
                             } else {
                                 const uint32_t w[4] = {t.x, t.y, t.z, t.w};
                                 for (int q = 0; q < 4 * wcols && col + q < ncols; q++) {
-                                    if (a.y_f32) static_cast<uint32_t*>(a.y)[o + q] = w[q];
+                                    if (y_f32) (second ? a.y2 : static_cast<float*>(a.y))[o + q] = __uint_as_float(w[q]);
                                     else static_cast<uint16_t*>(a.y)[o + q] = (uint16_t)(w[q >> 1] >> ((q & 1) * 16));
                                 }
                             }
@@ -323,7 +332,7 @@ int launch_tn(EncodeTiledFn enc, const LinearArgs<bf16>& l, DenseEpi e, int sms,
     CUtensorMap mx, mw;
     int st;
     if ((st = encode(enc, &mx, l.x, (l.batch - 1) * l.x_batch + l.K, l.M, l.ldx, kTok))) return st;
-    if ((st = encode(enc, &mw, l.w, l.K, l.batch * l.w_rows, l.ldw, TN / 2))) return st;
+    if ((st = encode(enc, &mw, l.w, l.K, (l.group ? l.entries : l.batch) * l.w_rows, l.ldw, TN / 2))) return st;
     static bool attr[64] = {};
     int dev = 0;
     cudaGetDevice(&dev);
@@ -348,6 +357,10 @@ int launch_dense_gemm_tcgen05(const LinearArgs<bf16>& l, cudaStream_t stream)
         return fail(TLLM_ERR_SHAPE, "dense_gemm: K=%d ldw=%d ldx=%d x_batch=%d must be multiples of 8", l.K, l.ldw, l.ldx, l.x_batch);
     if ((reinterpret_cast<uintptr_t>(l.x) | reinterpret_cast<uintptr_t>(l.w)) & 15)
         return fail(TLLM_ERR_ALIGN, "dense_gemm: operands must be 16-byte aligned");
+    if (l.group && (l.batch != 1 || !l.groups)) return fail(TLLM_ERR_SHAPE, "dense_gemm: grouped rows with %d batch entries", l.batch);
+    if ((l.act_lo | (l.act_hi == INT_MAX ? 0 : l.act_hi) | (l.f32_from == INT_MAX ? 0 : l.f32_from)) % 64 ||
+        ((l.act_lo || l.act_hi != INT_MAX || l.f32_from != INT_MAX) && (l.glu || l.batch != 1)))
+        return fail(TLLM_ERR_SHAPE, "dense_gemm: column ranges %d..%d and %d", l.act_lo, l.act_hi, l.f32_from);
     if (l.w_rows < (l.glu ? 2 : 1) * l.N) return fail(TLLM_ERR_SHAPE, "dense_gemm: %d rows of W for N=%d", l.w_rows, l.N);
     EncodeTiledFn enc = encode_fn();
     if (!enc) return fail(TLLM_ERR_LAUNCH, "cuTensorMapEncodeTiled is not available from this driver");
@@ -369,6 +382,15 @@ int launch_dense_gemm_tcgen05(const LinearArgs<bf16>& l, cudaStream_t stream)
     const size_t es = l.y_f32 ? 4 : 2;
     e.vec = ((l.ldy * es) % 16 == 0 && (l.y_batch * es) % 16 == 0 && (reinterpret_cast<uintptr_t>(l.y) & 15) == 0);
     e.bias_vec = l.N % 4 == 0 && (reinterpret_cast<uintptr_t>(l.bias) & 15) == 0;
+    e.act_param = l.act_param;
+    e.act_lo = l.act_lo;
+    e.act_hi = l.act_hi;
+    e.f32_from = l.f32_from;
+    e.y2 = l.y2;
+    e.ldy2 = l.ldy2;
+    e.vec2 = l.ldy2 % 4 == 0 && (reinterpret_cast<uintptr_t>(l.y2) & 15) == 0;
+    e.group = l.group;
+    e.groups = l.groups;
     e.err = device_error_flag();
     if (!e.err) return fail(TLLM_ERR_LAUNCH, "device scratch unavailable");
     static int sms[64] = {};

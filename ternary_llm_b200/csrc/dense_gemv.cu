@@ -41,10 +41,10 @@ __device__ __forceinline__ float gemv_cta_sum(float v, float* sh)
 
 __device__ __forceinline__ float4 gemv_ld4(const float* p, int i) { return *(reinterpret_cast<const float4*>(p) + i); }
 
-// One vector of the residual chain into shared memory; wp, wn: the norm weights, staged before
-// the wait on the previous kernel.  sh: 2 * kWarps words.
+// One vector of the residual chain into shared memory; wp, ws, wn: the norm weights, staged before
+// the wait on the previous kernel.  sh: 3 * kWarps words.
 template <typename T>
-__device__ __forceinline__ void stage_norm(const GemvNorm& f, int m, int K, T* xs, const float* wp, const float* wn, float* sh)
+__device__ __forceinline__ void stage_norm(const GemvNorm& f, int m, int K, T* xs, const float* wp, const float* ws, const float* wn, float* sh)
 {
     const size_t row = (size_t)m * K;
     const int n4 = K >> 2;
@@ -76,24 +76,46 @@ __device__ __forceinline__ void stage_norm(const GemvNorm& f, int m, int K, T* x
         if (i >= n4) continue;
         float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
         if (f.w_post) w = reinterpret_cast<const float4*>(wp)[i];
-        x[j].x += y[j].x * rinv * w.x;
-        x[j].y += y[j].y * rinv * w.y;
-        x[j].z += y[j].z * rinv * w.z;
-        x[j].w += y[j].w * rinv * w.w;
-        if (blockIdx.x == 0 && blockIdx.y == 0) reinterpret_cast<float4*>(f.x_out + row)[i] = x[j];
+        x[j].x = f.alpha * x[j].x + y[j].x * rinv * w.x;
+        x[j].y = f.alpha * x[j].y + y[j].y * rinv * w.y;
+        x[j].z = f.alpha * x[j].z + y[j].z * rinv * w.z;
+        x[j].w = f.alpha * x[j].w + y[j].w * rinv * w.w;
         ss += (x[j].x * x[j].x + x[j].y * x[j].y) + (x[j].z * x[j].z + x[j].w * x[j].w);
     }
-    rinv = 1.0f / sqrtf(gemv_cta_sum(ss, sh + kWarps) / (float)f.width + f.eps);
+    const bool first = blockIdx.x == 0 && blockIdx.y == 0;
+    auto scale = [&](float r, const float* w) {          // x *= r * w; the new sum of squares
+        ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < kNormVecs; j++) {
+            const int i = threadIdx.x + j * kWarps * 32;
+            if (i >= n4) continue;
+            const float4 v = reinterpret_cast<const float4*>(w)[i];
+            x[j].x = x[j].x * r * v.x;
+            x[j].y = x[j].y * r * v.y;
+            x[j].z = x[j].z * r * v.z;
+            x[j].w = x[j].w * r * v.w;
+            ss += (x[j].x * x[j].x + x[j].y * x[j].y) + (x[j].z * x[j].z + x[j].w * x[j].w);
+        }
+    };
+    if (f.w_sum) scale(1.0f / sqrtf(gemv_cta_sum(ss, sh + kWarps) / (float)f.width + f.eps), ws);
+    if (first) {
+#pragma unroll
+        for (int j = 0; j < kNormVecs; j++) {
+            const int i = threadIdx.x + j * kWarps * 32;
+            if (i < n4) reinterpret_cast<float4*>(f.x_out + row)[i] = x[j];
+        }
+    }
+    if (f.w_next) scale(1.0f / sqrtf(gemv_cta_sum(ss, sh + 2 * kWarps) / (float)f.width + f.eps), wn);
 #pragma unroll
     for (int j = 0; j < kNormVecs; j++) {
         const int i = threadIdx.x + j * kWarps * 32;
         if (i >= n4) continue;
-        const float4 w = reinterpret_cast<const float4*>(wn)[i];
-        T* d = xs + 4 * i;
-        d[0] = from_f<T>(x[j].x * rinv * w.x);
-        d[1] = from_f<T>(x[j].y * rinv * w.y);
-        d[2] = from_f<T>(x[j].z * rinv * w.z);
-        d[3] = from_f<T>(x[j].w * rinv * w.w);
+        T d[4] = {from_f<T>(x[j].x), from_f<T>(x[j].y), from_f<T>(x[j].z), from_f<T>(x[j].w)};
+#pragma unroll
+        for (int e = 0; e < 4; e++) xs[4 * i + e] = d[e];
+        if (first && f.h_out)
+#pragma unroll
+            for (int e = 0; e < 4; e++) static_cast<T*>(f.h_out)[row + 4 * i + e] = d[e];
     }
     __syncthreads();             // the next vector's sums reuse sh
 }
@@ -104,8 +126,8 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
 {
     constexpr int V = Vec16<T>::n;
     extern __shared__ __align__(16) uint8_t smem_raw[];
-    __shared__ float sh[2 * kWarps];
-    // ring, then the vectors [MB][K], then with NORM the two norm weights [K] each
+    __shared__ float sh[3 * kWarps];
+    // ring, then the vectors [MB][K], then with NORM the norm weights [K] each
     T* xs = reinterpret_cast<T*>(smem_raw + kRingBytes);
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -147,9 +169,12 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
     for (int g = 0; g < kGroups; g++) request();
     if (NORM) {
         float* wn = reinterpret_cast<float*>(xs + (size_t)MB * a.K);
-        for (int i = threadIdx.x; i < a.K / 4; i += kWarps * 32) {
-            reinterpret_cast<float4*>(wn)[i] = gemv_ld4(f.w_next, i);
-            if (f.w_post) reinterpret_cast<float4*>(wn + a.K)[i] = gemv_ld4(f.w_post, i);
+        const float* w[3] = {f.w_next, f.w_post, f.w_sum};
+#pragma unroll
+        for (int p = 0; p < 3; p++) {
+            if (!w[p]) continue;
+            for (int i = threadIdx.x; i < a.K / 4; i += kWarps * 32) reinterpret_cast<float4*>(wn)[i] = gemv_ld4(w[p], i);
+            wn += a.K;
         }
     }
 
@@ -157,7 +182,9 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
     const int mb = min(MB, a.M - m0);
     if (NORM) {
         const float* wn = reinterpret_cast<const float*>(xs + (size_t)MB * a.K);
-        for (int m = 0; m < mb; m++) stage_norm<T>(f, m, a.K, xs + (size_t)m * a.K, wn + a.K, wn, sh);
+        const float* wp = wn + (f.w_next ? a.K : 0);
+        const float* ws = wp + (f.w_post ? a.K : 0);
+        for (int m = 0; m < mb; m++) stage_norm<T>(f, m, a.K, xs + (size_t)m * a.K, wp, ws, wn, sh);
     } else {
         for (int i = threadIdx.x; i < mb * nv; i += kWarps * 32) {
             const int m = i / nv, c = i - m * nv;
@@ -256,7 +283,11 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
             }
             float v = res[0][m];
             if (a.bias) v += a.bias[(size_t)z * a.N + n];
-            v = apply_act(a.act, v);
+            if (n >= a.f32_from) {
+                a.y2[(size_t)(m0 + m) * a.ldy2 + n - a.f32_from] = v;
+                continue;
+            }
+            if (n >= a.act_lo && n < a.act_hi) v = apply_act(a.act, v, a.act_param);
             if (a.glu) v *= res[1][m];
             if (a.gate) v *= sigmoid_f(to_f<T>(a.gate[(size_t)(m0 + m) * a.gate_ld + z]));
             const size_t o = (size_t)(m0 + m) * a.ldy + (size_t)z * a.y_batch + n;
@@ -295,7 +326,8 @@ int launch_mb(const LinearArgs<T>& a, const GemvNorm& f, const GemvTail<T>& t, i
     // two CTAs per SM: the next launch finds room and requests its weights early
     const int cap = (2 * sms[dev] + a.batch - 1) / a.batch;
     if (grid > cap) grid = cap;
-    const size_t smem = kRingBytes + (size_t)MB * a.K * sizeof(T) + (NORM ? (size_t)2 * a.K * sizeof(float) : 0);
+    const int norms = NORM ? (f.w_next != nullptr) + (f.w_post != nullptr) + (f.w_sum != nullptr) : 0;
+    const size_t smem = kRingBytes + (size_t)MB * a.K * sizeof(T) + (size_t)norms * a.K * sizeof(float);
     if (smem > kSmemLimit || (NORM && a.K > kNormMaxK)) return fail(TLLM_ERR_SHAPE, "dense_gemv: %d vectors of %d", MB, a.K);
     return launch_pdl("dense_gemv", dense_gemv_kernel<T, MB, NORM, TAIL>, dim3(grid, a.batch), dim3(kWarps * 32), smem, stream, a, f, t, lpr, m0);
 }
@@ -396,11 +428,12 @@ dense_gemm_f32_kernel(const LinearArgs<float> a)
     pdl_launch_dependents();
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;      // outputs n = 4 tx.., m = 4 ty..
     const int n0 = blockIdx.x * kTile, m0 = blockIdx.y * kTile, z = blockIdx.z;
-    const float* wz = a.w + (size_t)z * a.w_rows * a.ldw;
-    const float* xz = a.x + (size_t)z * a.x_batch;
     const int parts = a.glu ? 2 : 1;
     float acc[2][4][4] = {};
     pdl_wait();
+    if (a.group && m0 / kGroupRows >= *a.groups) return;
+    const float* wz = a.w + (size_t)(a.group ? a.group[m0 / kGroupRows] : z) * a.w_rows * a.ldw;
+    const float* xz = a.x + (size_t)z * a.x_batch;
     const int lr = threadIdx.x >> 2, lc = (threadIdx.x & 3) * 4;  // loader: row of the tile, 4 columns
     for (int k0 = 0; k0 < a.K; k0 += kSlice) {
         __syncthreads();
@@ -443,7 +476,11 @@ dense_gemm_f32_kernel(const LinearArgs<float> a)
             if (m >= a.M || n >= a.N) continue;
             float v = acc[0][i][j];
             if (a.bias) v += a.bias[(size_t)z * a.N + n];
-            v = apply_act(a.act, v);
+            if (n >= a.f32_from) {
+                a.y2[(size_t)m * a.ldy2 + n - a.f32_from] = v;
+                continue;
+            }
+            if (n >= a.act_lo && n < a.act_hi) v = apply_act(a.act, v, a.act_param);
             if (a.glu) v *= acc[1][i][j];
             if (a.gate) v *= sigmoid_f(a.gate[(size_t)m * a.gate_ld + z]);
             y[(size_t)m * a.ldy + (size_t)z * a.y_batch + n] = v;
@@ -468,6 +505,7 @@ __device__ __forceinline__ float pack_fn(float v, int fn)
 {
     const double d = (double)v;
     if (fn == kPackNegExpLog2e) return (float)(-exp(d) * 1.4426950408889634074);
+    if (fn == kPackNegExp) return (float)-exp(d);
     if (fn == kPackSoftplus) return (float)(fmax(d, 0.0) + log1p(exp(-fabs(d))));
     return v;
 }

@@ -1,6 +1,8 @@
 // Decoder of a list of mixer layers (include/tllm_b200_mixed.h): latent attention, selective
-// scan, real-gated linear recurrence, each with an optional gated feed-forward, a norm before
-// and after every sublayer, layers that run several times.
+// scan, real-gated linear recurrence, and the mixers made of heads (grouped-query attention,
+// linear attention, gated delta rule; alone or two side by side), each with an optional dense or
+// routed feed-forward, norms around every sublayer or behind the sum, layers that run several
+// times.
 //
 // The residual stream, the norms, the recurrent states and what feeds them are FP32; weights and
 // activations are BF16 (or FP32 in the exact mode, the same code instantiated for float).  All
@@ -35,9 +37,34 @@ struct Mat {
     int rows = 0, ld = 0;
 };
 
+// A mixer made of heads; a layer has one, or two that share the projection in front and the one
+// behind.  Columns: of the layer's projection, of its FP32 part (a, b), of the input of the output
+// projection.  Padded sizes unless marked.
+struct HeadPart {
+    int type = 0, heads = 0, kv_heads = 0, dim = 0, dim_true = 0, vdim = 0, vdim_true = 0;
+    int q = 0, k = 0, v = 0, gate = 0, a = 0, b = 0, out = 0;
+    float out_scale = 1.f;
+    // attention
+    float scale = 0.f;
+    int rot_dims = 0, chunk = 0;
+    const float2* rope = nullptr;
+    float *q_norm = nullptr, *k_norm = nullptr;
+    // linear attention, delta rule
+    float *norm = nullptr, *decay = nullptr, *neg_a = nullptr, *dt_bias = nullptr, *conv = nullptr;
+    int taps = 0, in_act = 0, gate_act = 0;
+    int conv_channels() const { return 2 * kv_heads * dim + heads * vdim; }
+};
+
 template <typename T>
 struct MixLayer {
     int type = 0;
+    std::vector<HeadPart> parts;
+    int in_ld = 0;                             // projected columns kept in T
+    int act_lo = 0, act_hi = INT_MAX, in_act = kActNone, f32_from = INT_MAX, n_f32 = 0;
+    int experts = 0, top = 0;
+    Mat<T> router;
+    bool few = false;                          // the experts' rows may be streamed token by token
+    bool has_ff() const { return ff > 0; }
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
     Mat<T> gate_up, down, in, out;
     int ff = 0, ff_act = 0;
@@ -56,9 +83,18 @@ struct MixLayer {
     float *gate_bias = nullptr, *soft_lam = nullptr;
 };
 
+template <typename T>
+struct PartState {
+    T *k = nullptr, *v = nullptr, *conv = nullptr;
+    float* rec = nullptr;
+    size_t k_slot = 0, v_slot = 0, conv_slot = 0, rec_slot = 0;
+    int cache_rows = 0;
+};
+
 // cache or state of one run of a layer, all slots
 template <typename T>
 struct RunState {
+    PartState<T> part[2];
     T* cache = nullptr;        // latent attention
     T* conv = nullptr;
     float* rec = nullptr;
@@ -72,8 +108,10 @@ struct MixedDecoder : Decoder {
     std::vector<MixLayer<T>> layers;
     std::vector<std::pair<int, bool>> order;   // (layer, add the embedding output first)
     std::vector<RunState<T>> runs;
-    Mat<T> embed;
+    Mat<T> embed, out_head;
     float* final_norm = nullptr;
+    bool norm_after = false;
+    float alpha = 1.f, softcap = 0.f;
     bool recurrent = false, inject = false, fused_ok = true;
     int rows_cap = 0;
     std::vector<int> len;                  // tokens each slot's sequence has consumed
@@ -82,6 +120,10 @@ struct MixedDecoder : Decoder {
     float *x = nullptr, *x2 = nullptr, *emb = nullptr, *y = nullptr, *f32buf = nullptr, *ws = nullptr, *rec = nullptr, *logits = nullptr;
     T *h = nullptr, *proj = nullptr, *mixed = nullptr, *conv_out = nullptr, *xdbc = nullptr, *q_abs = nullptr, *o_lat = nullptr;
     T *kx = nullptr, *vx = nullptr;
+    float *heads_o = nullptr, *router_z = nullptr, *part_w = nullptr;
+    uint8_t* scan_ws = nullptr;
+    T *gathered = nullptr, *hidden = nullptr, *expert_out = nullptr;
+    int *counts = nullptr, *chosen = nullptr, *part_row = nullptr, *group = nullptr, *groups = nullptr;
     int* want_dev = nullptr;
     uint8_t* backup = nullptr;
     size_t backup_bytes = 0;
@@ -111,6 +153,20 @@ private:
     }
     int vec(float** out, const void* src, int gr, int r, int rp, int fn = kPackCopy);
     int load_layer(const tllm_b200_mixed_layer& s, MixLayer<T>& L);
+    int load_heads(const tllm_b200_mixed_layer& s, MixLayer<T>& L);
+    int load_part(const tllm_b200_mixed_layer& s, MixLayer<T>& L, HeadPart& p);
+    int pack_rows(const void* src, int gr, int r, int rs, int rp, int gc, int c, int cp, T* dst, int ld)
+    {
+        PackSpec p;
+        p.gr = gr; p.r = r; p.rs = rs; p.rp = rp; p.gc = gc; p.c = c; p.cp = cp;
+        return launch_pack<T>(src, p, dst, ld, nullptr);
+    }
+    int part_state(const HeadPart& p, PartState<T>* s);
+    int heads_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, bool conv_done, cudaStream_t s);
+    LinearArgs<T> in_product(const MixLayer<T>& L, int n_rows) const;
+    LinearArgs<T> head_product(int n, float* out) const;
+    int experts(const MixLayer<T>& L, int n_rows, const GemvNorm* norm, cudaStream_t s);
+    bool gathers(const MixLayer<T>& L, int n_rows) const { return L.experts && (n_rows > kFewRows || !L.few); }
     int rope_table(double base, int dims, const float2** out);
     int layers_pass(const int* tokens, const StepGeo& g, float* taps, size_t tap_stride, cudaStream_t s);
     int embed_rows(const int* tokens, int rows, cudaStream_t s);
@@ -203,14 +259,20 @@ int MixedDecoder<T>::load_layer(const tllm_b200_mixed_layer& s, MixLayer<T>& L)
         return TLLM_OK;
     };
     auto rows_to = [&](const void* src, int gr, int r, int rs, int rp, int gc, int c, int cp, T* dst, int ld) -> int {
-        PackSpec p;
-        p.gr = gr; p.r = r; p.rs = rs; p.rp = rp; p.gc = gc; p.c = c; p.cp = cp;
-        return launch_pack<T>(src, p, dst, ld, nullptr);
+        return pack_rows(src, gr, r, rs, rp, gc, c, cp, dst, ld);
     };
     const void* const* t = s.t;
     L.type = s.type;
     TRY(need({TLLM_T_NORM1, TLLM_T_OUT}));
     TRY(vec(&L.norm1, t[TLLM_T_NORM1], 1, width, w));
+    if (s.ff > 0 && s.experts > 0) {
+        TRY(need({TLLM_T_ROUTER}));
+        if (s.top < 1 || s.top > s.experts) return fail(TLLM_ERR_SHAPE, "mixed decoder: %d of %d experts", s.top, s.experts);
+        L.experts = s.experts;
+        L.top = s.top;
+        TRY(mat(&L.router, pad8(s.experts), w));
+        TRY(rows_to(t[TLLM_T_ROUTER], 1, s.experts, s.experts, L.router.rows, 1, width, w, L.router.p, w));
+    }
     if (t[TLLM_T_NORM1B]) TRY(vec(&L.norm1b, t[TLLM_T_NORM1B], 1, width, w));
     if (s.ff > 0) {
         TRY(need({TLLM_T_NORM2, TLLM_T_GATE, TLLM_T_UP, TLLM_T_DOWN}));
@@ -218,12 +280,15 @@ int MixedDecoder<T>::load_layer(const tllm_b200_mixed_layer& s, MixLayer<T>& L)
         L.ff_act = s.ff_act;
         TRY(vec(&L.norm2, t[TLLM_T_NORM2], 1, width, w));
         if (t[TLLM_T_NORM2B]) TRY(vec(&L.norm2b, t[TLLM_T_NORM2B], 1, width, w));
-        TRY(mat(&L.gate_up, 2 * L.ff, w));
-        TRY(rows_to(t[TLLM_T_GATE], 1, s.ff, s.ff, L.ff, 1, width, w, L.gate_up.p, w));
-        TRY(rows_to(t[TLLM_T_UP], 1, s.ff, s.ff, L.ff, 1, width, w, L.gate_up.p + (size_t)L.ff * w, w));
-        TRY(mat(&L.down, w, L.ff));
-        TRY(rows_to(t[TLLM_T_DOWN], 1, width, width, w, 1, s.ff, L.ff, L.down.p, L.ff));
+        const int n = L.experts ? L.experts : 1;             // matrices one behind the other
+        L.few = L.experts && experts_few_fits(L.top, L.ff, w, sizeof(T));
+        TRY(mat(&L.gate_up, n * 2 * L.ff, w));
+        TRY(rows_to(t[TLLM_T_GATE], n, s.ff, s.ff, 2 * L.ff, 1, width, w, L.gate_up.p, w));
+        TRY(rows_to(t[TLLM_T_UP], n, s.ff, s.ff, 2 * L.ff, 1, width, w, L.gate_up.p + (size_t)L.ff * w, w));
+        TRY(mat(&L.down, n * w, L.ff));
+        TRY(rows_to(t[TLLM_T_DOWN], n, width, width, w, 1, s.ff, L.ff, L.down.p, L.ff));
     }
+    if (s.type == TLLM_MIXER_ATTENTION || s.type == TLLM_MIXER_LINEAR_ATTENTION || s.type == TLLM_MIXER_DELTA_RULE) return load_heads(s, L);
     if (s.type == TLLM_MIXER_LATENT_ATTENTION) {
         TRY(need({TLLM_T_Q, TLLM_T_KV_DOWN, TLLM_T_KV_NORM, TLLM_T_K_UP, TLLM_T_V_UP}));
         if (s.heads < 1 || s.dim < 1 || s.rot_dim < 0 || s.rot_dims < 0 || s.rot_dims > s.rot_dim || s.rot_dims % 2 || s.vdim < 1 || s.kv_rank < 1)
@@ -333,6 +398,148 @@ int MixedDecoder<T>::load_layer(const tllm_b200_mixed_layer& s, MixLayer<T>& L)
     return TLLM_OK;
 }
 
+// Sizes and columns are set; matrices into L.in and L.out, vectors of the mixer alone.
+template <typename T>
+int MixedDecoder<T>::load_part(const tllm_b200_mixed_layer& s, MixLayer<T>& L, HeadPart& p)
+{
+    int st;
+    const void* const* t = s.t;
+    auto need = [&](std::initializer_list<int> ids) -> int {
+        for (int i : ids)
+            if (!t[i]) return fail(TLLM_ERR_NULL, "mixed decoder: tensor %d of a mixer of type %d is missing", i, s.type);
+        return TLLM_OK;
+    };
+    TRY(need({TLLM_T_Q, TLLM_T_K, TLLM_T_V, TLLM_T_OUT}));
+    const int H = s.heads, G = s.type == TLLM_MIXER_LINEAR_ATTENTION ? H : s.kv_heads;
+    auto project = [&](int slot, int heads, int n, int np, int col) -> int {
+        return pack_rows(t[slot], heads, n, n, np, 1, width, w, L.in.p + (size_t)col * w, w);
+    };
+    const bool att = s.type == TLLM_MIXER_ATTENTION, delta = s.type == TLLM_MIXER_DELTA_RULE;
+    TRY(project(TLLM_T_Q, delta ? G : H, s.dim, p.dim, p.q));
+    TRY(project(TLLM_T_K, G, s.dim, p.dim, p.k));
+    TRY(project(TLLM_T_V, att ? G : H, s.vdim, p.vdim, p.v));
+    TRY(pack_rows(t[TLLM_T_OUT], 1, width, width, w, H, s.vdim, p.vdim, L.out.p + p.out, L.out.ld));
+    if (att) {
+        if (t[TLLM_T_Q_NORM]) TRY(vec(&p.q_norm, t[TLLM_T_Q_NORM], 1, s.dim, p.dim));
+        if (t[TLLM_T_K_NORM]) TRY(vec(&p.k_norm, t[TLLM_T_K_NORM], 1, s.dim, p.dim));
+        return rope_table(s.rot_base, s.rot_dims, &p.rope);
+    }
+    recurrent = true;
+    TRY(need({TLLM_T_MIX_NORM, TLLM_T_MIX_GATE}));
+    TRY(project(TLLM_T_MIX_GATE, H, s.vdim, p.vdim, p.gate));
+    if (!delta) {
+        if (!s.head_decay) return fail(TLLM_ERR_NULL, "mixed decoder: linear attention without decays");
+        TRY(dev_alloc(&p.decay, (size_t)H, false));
+        if (cudaMemcpy(p.decay, s.head_decay, H * sizeof(float), cudaMemcpyHostToDevice) != cudaSuccess)
+            return fail(TLLM_ERR_LAUNCH, "mixed decoder: %s", cudaGetErrorString(cudaGetLastError()));
+        return vec(&p.norm, t[TLLM_T_MIX_NORM], H, s.vdim, p.vdim);
+    }
+    TRY(need({TLLM_T_Q_CONV, TLLM_T_K_CONV, TLLM_T_V_CONV, TLLM_T_STEP, TLLM_T_DECAY, TLLM_T_DT_BIAS, TLLM_T_A_LOG}));
+    TRY(project(TLLM_T_STEP, 1, H, H, L.f32_from + p.b));
+    TRY(project(TLLM_T_DECAY, 1, H, H, L.f32_from + p.a));
+    TRY(vec(&p.neg_a, t[TLLM_T_A_LOG], 1, H, H, kPackNegExp));
+    TRY(vec(&p.dt_bias, t[TLLM_T_DT_BIAS], 1, H, H));
+    TRY(vec(&p.norm, t[TLLM_T_MIX_NORM], 1, s.vdim, p.vdim));
+    TRY(dev_alloc(&p.conv, (size_t)p.conv_channels() * p.taps, true));
+    const int slots[3] = {TLLM_T_Q_CONV, TLLM_T_K_CONV, TLLM_T_V_CONV};
+    for (int i = 0; i < 3; i++) {
+        PackSpec c;
+        c.gr = i < 2 ? G : H;
+        c.r = c.rs = i < 2 ? s.dim : s.vdim;
+        c.rp = i < 2 ? p.dim : p.vdim;
+        c.c = c.cp = p.taps;
+        TRY(launch_pack<float>(t[slots[i]], c, p.conv + (size_t)i * G * p.dim * p.taps, p.taps, nullptr));
+    }
+    return TLLM_OK;
+}
+
+// One or two mixers of heads.  Columns of the common projection: every mixer's q, k, v (and
+// gate) in order, ranges that take an activation and the FP32 part on multiples of 64.
+template <typename T>
+int MixedDecoder<T>::load_heads(const tllm_b200_mixed_layer& s, MixLayer<T>& L)
+{
+    int st;
+    const tllm_b200_mixed_layer* mixers[2] = {&s, s.beside};
+    const int n = s.beside ? 2 : 1;
+    auto pad64 = [](int v) { return (v + 63) / 64 * 64; };
+    int col = 0, out = 0;
+    L.parts.resize(n);
+    for (int i = 0; i < n; i++) {
+        const tllm_b200_mixed_layer& m = *mixers[i];
+        HeadPart& p = L.parts[i];
+        const bool att = m.type == TLLM_MIXER_ATTENTION, lin = m.type == TLLM_MIXER_LINEAR_ATTENTION, delta = m.type == TLLM_MIXER_DELTA_RULE;
+        const int G = lin ? m.heads : m.kv_heads;
+        if ((!att && !lin && !delta) || m.heads < 1 || G < 1 || m.heads % G || m.dim < 1 || m.vdim < 1 || (delta && m.taps < 1) ||
+            (att && (m.rot_dims < 0 || m.rot_dims % 2 || m.rot_dims > m.dim || m.chunk < 0)))
+            return fail(TLLM_ERR_SHAPE, "mixed decoder: mixer of type %d with heads=%d/%d dim=%d vdim=%d rot=%d taps=%d chunk=%d", m.type, m.heads, G,
+                        m.dim, m.vdim, m.rot_dims, m.taps, m.chunk);
+        if (i == 1 && !att && m.type == s.type) return fail(TLLM_ERR_SHAPE, "mixed decoder: two mixers of type %d side by side", m.type);
+        p.type = m.type;
+        p.heads = m.heads;
+        p.kv_heads = G;
+        p.dim_true = m.dim;
+        p.dim = pad8(m.dim);
+        p.vdim_true = m.vdim;
+        p.vdim = pad8(m.vdim);
+        if (att ? !grouped_supported(p.heads, G, p.dim, p.vdim) : p.dim > 512)
+            return fail(TLLM_ERR_SHAPE, "mixed decoder: mixer of type %d with dim=%d vdim=%d", m.type, m.dim, m.vdim);
+        p.out_scale = m.out_scale;
+        p.scale = m.scale;
+        p.rot_dims = m.rot_dims;
+        p.chunk = m.chunk;
+        p.taps = m.taps;
+        p.in_act = m.in_act;
+        p.gate_act = m.gate_act;
+        if (lin) {
+            L.act_lo = col = pad64(col);
+            L.in_act = m.in_act;
+        }
+        p.q = col;
+        p.k = p.q + (delta ? G : p.heads) * p.dim;
+        p.v = p.k + G * p.dim;
+        col = p.v + (att ? G : p.heads) * p.vdim;
+        if (lin) L.act_hi = col = pad64(col);
+        p.gate = col;
+        if (!att) col += p.heads * p.vdim;
+        if (delta) {
+            p.b = L.n_f32;
+            p.a = L.n_f32 + pad8(p.heads);
+            L.n_f32 += 2 * pad8(p.heads);
+        }
+        p.out = out;
+        out += p.heads * p.vdim;
+    }
+    if (L.n_f32) L.f32_from = col = pad64(col);
+    L.in_ld = col;
+    TRY(mat(&L.in, col + L.n_f32, w));
+    TRY(mat(&L.out, w, out));
+    for (int i = 0; i < n; i++) TRY(load_part(*mixers[i], L, L.parts[i]));
+    return TLLM_OK;
+}
+
+// cache and state of one mixer, all slots
+template <typename T>
+int MixedDecoder<T>::part_state(const HeadPart& p, PartState<T>* s)
+{
+    int st;
+    if (p.type == TLLM_MIXER_ATTENTION) {
+        s->cache_rows = grouped_cache_rows(max_seq, p.chunk, rows_cap);
+        if (s->cache_rows < max_seq) recurrent = true;
+        s->k_slot = (size_t)s->cache_rows * p.kv_heads * p.dim;
+        s->v_slot = (size_t)s->cache_rows * p.kv_heads * p.vdim;
+        TRY(dev_alloc(&s->k, s->k_slot * max_batch, true));
+        return dev_alloc(&s->v, s->v_slot * max_batch, true);
+    }
+    s->rec_slot = (size_t)p.heads * p.dim * p.vdim;
+    TRY(dev_alloc(&s->rec, s->rec_slot * max_batch, true));
+    if (p.type == TLLM_MIXER_DELTA_RULE && p.taps > 1) {
+        s->conv_slot = (size_t)(p.taps - 1) * p.conv_channels();
+        TRY(dev_alloc(&s->conv, s->conv_slot * max_batch, true));
+    }
+    backup_bytes += s->conv_slot * sizeof(T) + s->rec_slot * sizeof(float);
+    return TLLM_OK;
+}
+
 template <typename T>
 int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_batch_)
 {
@@ -351,13 +558,25 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
         p.cp = w;
         TRY(launch_pack<T>(c.embedding, p, embed.p, w, nullptr));
     }
+    out_head = embed;
+    if (c.head) {
+        TRY(mat(&out_head, vocab, w));
+        TRY(pack_rows(c.head, 1, vocab, vocab, vocab, 1, width, w, out_head.p, w));
+    }
+    norm_after = c.norm_after_sum != 0;
+    if (norm_after) alpha = c.residual_scale;
+    softcap = c.logit_softcap;
     TRY(vec(&final_norm, c.final_norm, 1, width, w));
     layers.resize(c.n_layers);
     for (int i = 0; i < c.n_layers; i++) TRY(load_layer(c.layers[i], layers[i]));
 
     // a convolution in the tail of a GEMV needs a lane per tap; norm staging rows in shared memory
-    for (const MixLayer<T>& L : layers)
+    for (const MixLayer<T>& L : layers) {
         if (L.ch && !gemv_tail_fits<T>(w, L.taps)) fused_ok = false;
+        for (const HeadPart& p : L.parts)
+            if (p.taps && !gemv_tail_fits<T>(w, p.taps)) fused_ok = false;
+        if (L.experts && !L.few) fused_ok = false;
+    }
     if (!gemv_norm_fits<T>(w)) fused_ok = false;
 
     const bool loop = c.loop_times != 1 && c.loop_stop > c.loop_start;
@@ -378,10 +597,31 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
     const int ar = rows_cap < kAbsorbRows ? rows_cap : kAbsorbRows;
     size_t n_proj = 0, n_mixed = 0, n_ch = 0, n_x = 0, n_f32 = 0, n_q = 0, n_o = 0, n_ws = 0, n_k = 0, n_v = 0, n_rec = 0;
     auto up = [](size_t& a, size_t b) { if (b > a) a = b; };
+    size_t n_heads_o = 0, n_scan = 0, n_z = 0, n_top = 0, n_gather = 0, n_hidden = 0, n_experts = 0;
     for (const MixLayer<T>& L : layers) {
-        up(n_mixed, L.ff);
+        if (!L.experts) up(n_mixed, L.ff);
         up(n_mixed, L.out.ld);
-        up(n_proj, L.in.rows);
+        up(n_proj, L.parts.empty() ? L.in.rows : L.in_ld);
+        for (const HeadPart& p : L.parts) {
+            if (p.type == TLLM_MIXER_ATTENTION) {
+                up(n_ws, grouped_workspace_floats(p.heads, p.vdim));
+            } else {
+                const bool delta = p.type == TLLM_MIXER_DELTA_RULE;
+                up(n_heads_o, (size_t)p.heads * p.vdim);
+                up(n_scan, matrix_scan_workspace(sizeof(T) == 2, delta, rows_cap, p.heads, p.dim));
+                if (delta) up(n_ch, p.conv_channels());
+            }
+            up(n_f32, L.n_f32);
+        }
+        if (L.experts) {
+            const size_t few = (size_t)(rows_cap < kFewRows ? rows_cap : kFewRows) * L.top, many = expert_rows(rows_cap, L.top, L.experts);
+            up(n_z, L.router.rows);
+            up(n_top, L.top);
+            up(n_gather, many);
+            up(n_hidden, (few > many ? few : many) * L.ff);
+            up(n_experts, L.experts);
+        }
+        if (!L.parts.empty()) continue;
         if (L.type == TLLM_MIXER_LATENT_ATTENTION) {
             up(n_q, (size_t)L.heads * (L.rank + L.rot));
             up(n_o, (size_t)L.heads * L.rank);
@@ -410,6 +650,18 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
     TRY(dev_alloc(&o_lat, some(ar * n_o), true));
     TRY(dev_alloc(&ws, some(n_ws), true));
     TRY(dev_alloc(&rec, some(n_rec), true));
+    TRY(dev_alloc(&heads_o, some(R * n_heads_o), true));
+    TRY(dev_alloc(&scan_ws, some(n_scan), true));
+    TRY(dev_alloc(&router_z, some(R * n_z), true));
+    TRY(dev_alloc(&part_w, some(R * n_top), true));
+    TRY(dev_alloc(&chosen, some(R * n_top), true));
+    TRY(dev_alloc(&part_row, some(R * n_top), true));
+    TRY(dev_alloc(&gathered, some(n_gather * w), true));
+    TRY(dev_alloc(&expert_out, some(n_gather * w), true));
+    TRY(dev_alloc(&hidden, some(n_hidden), true));
+    TRY(dev_alloc(&counts, some(2 * n_experts), true));
+    TRY(dev_alloc(&group, some(n_gather / kGroupRows), true));
+    TRY(dev_alloc(&groups, 1, true));
     if (sizeof(T) == 2) {
         TRY(dev_alloc(&kx, some(max_seq * n_k), true));
         TRY(dev_alloc(&vx, some(max_seq * n_v), true));
@@ -419,6 +671,11 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
     for (const auto& o : order) {
         const MixLayer<T>& L = layers[o.first];
         RunState<T> rs;
+        for (size_t i = 0; i < L.parts.size(); i++) TRY(part_state(L.parts[i], &rs.part[i]));
+        if (!L.parts.empty()) {
+            runs.push_back(rs);
+            continue;
+        }
         if (L.type == TLLM_MIXER_LATENT_ATTENTION) {
             rs.cache_slot = (size_t)max_seq * (L.rank + L.rot);
             TRY(dev_alloc(&rs.cache, rs.cache_slot * max_batch, true));
@@ -460,6 +717,11 @@ int MixedDecoder<T>::copy_sequence(int seq, bool save, cudaStream_t s)
         p += bytes;
     };
     for (RunState<T>& r : runs) {
+        for (PartState<T>& p : r.part) {
+            if (!p.rec) continue;
+            one(p.rec + (size_t)seq * p.rec_slot, p.rec_slot * sizeof(float));
+            one(p.conv + (size_t)seq * p.conv_slot, p.conv_slot * sizeof(T));
+        }
         if (!r.rec) continue;
         one(r.rec + (size_t)seq * r.rec_slot, r.rec_slot * sizeof(float));
         one(r.conv + (size_t)seq * r.conv_slot, r.conv_slot * sizeof(T));
@@ -634,12 +896,130 @@ LinearArgs<T> MixedDecoder<T>::gates_args(const MixLayer<T>& L, int n_rows) cons
     return l;
 }
 
+template <typename T>
+LinearArgs<T> MixedDecoder<T>::in_product(const MixLayer<T>& L, int n_rows) const
+{
+    LinearArgs<T> l = product(L.in, h, w, w, proj, L.parts.empty() ? L.in.rows : L.in_ld, false, n_rows, L.in_bias, L.in_act);
+    l.act_lo = L.act_lo;
+    l.act_hi = L.act_hi;
+    l.f32_from = L.f32_from;
+    l.y2 = f32buf;
+    l.ldy2 = L.n_f32;
+    return l;
+}
+
+// Mixers of heads: proj (and f32buf) -> mixed.  conv_done: conv_out is there already.
+template <typename T>
+int MixedDecoder<T>::heads_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, bool conv_done, cudaStream_t s)
+{
+    int st;
+    for (size_t i = 0; i < L.parts.size(); i++) {
+        const HeadPart& p = L.parts[i];
+        const PartState<T>& S = R.part[i];
+        if (p.type == TLLM_MIXER_ATTENTION) {
+            GroupedArgs<T> a;
+            a.proj = proj;
+            a.ld = L.in_ld;
+            a.q_off = p.q;
+            a.k_off = p.k;
+            a.v_off = p.v;
+            a.heads = p.heads;
+            a.kv_heads = p.kv_heads;
+            a.dim = p.dim;
+            a.vdim = p.vdim;
+            a.dim_true = p.dim_true;
+            a.q_norm = p.q_norm;
+            a.k_norm = p.k_norm;
+            a.eps = eps;
+            a.rope = p.rope;
+            a.rot_dims = p.rot_dims;
+            a.kc = S.k;
+            a.vc = S.v;
+            a.k_slot = S.k_slot;
+            a.v_slot = S.v_slot;
+            a.cache_rows = S.cache_rows;
+            a.max_seq = max_seq;
+            a.chunk = p.chunk;
+            a.scale = p.scale;
+            a.out_scale = p.out_scale;
+            a.out = mixed + p.out;
+            a.ld_out = L.out.ld;
+            a.g = g;
+            TRY(launch_grouped_attention<T>(a, ws, s));
+            continue;
+        }
+        MatrixScanArgs<T> a;
+        a.delta = p.type == TLLM_MIXER_DELTA_RULE;
+        const T* x = proj + p.q;
+        a.ld = L.in_ld;
+        if (a.delta) {
+            if (!conv_done) {
+                ConvArgs<T> c;
+                c.x = proj + p.q;
+                c.ldx = L.in_ld;
+                c.w = p.conv;
+                c.state = S.conv;
+                c.slot_stride = S.conv_slot;
+                c.y = conv_out;
+                c.channels = p.conv_channels();
+                c.taps = p.taps;
+                c.act = p.in_act;
+                c.g = g;
+                TRY(launch_causal_conv<T>(c, s));
+            }
+            x = conv_out;
+            a.ld = p.conv_channels();
+            a.a = f32buf + p.a;
+            a.b = f32buf + p.b;
+            a.ld_ab = L.n_f32;
+            a.neg_a = p.neg_a;
+            a.dt_bias = p.dt_bias;
+            a.q_scale = 1.f / std::sqrt((float)p.dim_true);
+        } else {
+            a.decay = p.decay;
+        }
+        a.q = x;
+        a.k = x + (p.k - p.q);
+        a.v = x + (p.v - p.q);
+        a.heads = p.heads;
+        a.kv_heads = p.kv_heads;
+        a.dim = p.dim;
+        a.vdim = p.vdim;
+        a.state = S.rec;
+        a.slot_stride = S.rec_slot;
+        a.o = heads_o;
+        a.ws = scan_ws;
+        a.g = g;
+        TRY(launch_matrix_scan<T>(a, s));
+        GatedNormArgs<T> n;
+        n.o = heads_o;
+        n.w = p.norm;
+        n.gate = proj + p.gate;
+        n.ld_gate = L.in_ld;
+        n.act = p.gate_act;
+        n.eps = eps;
+        n.out_scale = p.out_scale;
+        n.out = mixed + p.out;
+        n.ld_out = L.out.ld;
+        n.rows = g.rows();
+        n.groups = a.delta ? p.heads : 1;
+        n.n = a.delta ? p.vdim : p.heads * p.vdim;
+        n.n_true = a.delta ? p.vdim_true : p.heads * p.vdim_true;
+        TRY(launch_gated_norm<T>(n, s));
+    }
+    return TLLM_OK;
+}
+
 // h -> mixed, the input of the output projection
 template <typename T>
 int MixedDecoder<T>::mixer_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, cudaStream_t s)
 {
     int st;
     const int rows = g.rows(), ch = L.ch;
+    if (!L.parts.empty()) {
+        TRY(linear(in_product(L, rows), s));
+        return heads_inner(L, R, g, false, s);
+    }
     if (L.type == TLLM_MIXER_LATENT_ATTENTION) {
         TRY(project(L.in, h, w, w, proj, L.in.rows, false, rows, s));
         return attention_inner(L, R, g, s);
@@ -693,11 +1073,66 @@ int MixedDecoder<T>::mixer(const MixLayer<T>& L, const RunState<T>& R, const Ste
     return project(L.out, mixed, L.out.ld, L.out.ld, y, w, true, g.rows(), s);
 }
 
+// Mixture of experts: h (or the residual chain staged in the router's product, which leaves h) -> y
+// for few rows, expert_out with part_row and part_w for many
+template <typename T>
+int MixedDecoder<T>::experts(const MixLayer<T>& L, int n_rows, const GemvNorm* norm, cudaStream_t s)
+{
+    int st;
+    const LinearArgs<T> r = product(L.router, h, w, w, router_z, L.router.rows, true, n_rows);
+    if (norm) {
+        GemvNorm f = *norm;
+        f.h_out = h;
+        TRY(launch_dense_gemv_fused<T>(r, f, GemvTail<T>(), s));
+    } else {
+        TRY(linear(r, s));
+    }
+    ExpertArgs<T> a;
+    a.z = router_z;
+    a.ld_z = L.router.rows;
+    a.experts = L.experts;
+    a.top = L.top;
+    a.h = h;
+    a.rows = n_rows;
+    a.w = w;
+    a.ff = L.ff;
+    a.gate_up = L.gate_up.p;
+    a.down = L.down.p;
+    a.act = L.ff_act;
+    a.hidden = hidden;
+    a.y = y;
+    if (!gathers(L, n_rows)) return launch_experts_few<T>(a, s);
+    a.counts = counts;
+    a.chosen = chosen;
+    a.part_row = part_row;
+    a.part_w = part_w;
+    a.gathered = gathered;
+    a.group = group;
+    a.groups = groups;
+    TRY(launch_experts_gather<T>(a, s));
+    const int m = expert_rows(n_rows, L.top, L.experts);
+    LinearArgs<T> l = product(L.gate_up, gathered, w, w, hidden, L.ff, false, m, nullptr, L.ff_act);
+    l.w_rows = 2 * L.ff;
+    l.N = L.ff;
+    l.glu = true;
+    l.group = group;
+    l.groups = groups;
+    l.entries = L.experts;
+    TRY(linear(l, s));
+    LinearArgs<T> d = product(L.down, hidden, L.ff, L.ff, expert_out, w, false, m);
+    d.w_rows = d.N = w;
+    d.group = group;
+    d.groups = groups;
+    d.entries = L.experts;
+    return linear(d, s);
+}
+
 // h (or the residual chain staged in the first product) -> y
 template <typename T>
 int MixedDecoder<T>::feed_forward(const MixLayer<T>& L, int n_rows, const GemvNorm* norm, cudaStream_t s)
 {
     int st;
+    if (L.experts) return experts(L, n_rows, norm, s);
     LinearArgs<T> l;
     l.w = L.gate_up.p;
     l.ldw = w;
@@ -729,14 +1164,14 @@ int MixedDecoder<T>::embed_rows(const int* tokens, int rows, cudaStream_t s)
     a.table = embed.p;
     a.tokens = tokens;
     a.emb = inject ? emb : nullptr;
-    a.w_next = layers[order[0].first].norm1;
+    a.w_next = norm_after ? nullptr : layers[order[0].first].norm1;
     return launch_norm_chain<T>(a, s);
 }
 
 // One new token of each of a few sequences, logits of all of them: the residual chain is staged
 // in the products behind it, the convolution step and the gated recurrence step are tails of
-// the products in front of them.  Launches per layer without / with feed-forward: attention
-// 7 / 9, scan 4 / 6, recurrence 3 / 5.
+// the products in front of them.  Launches per layer without / with feed-forward: latent attention
+// 7 / 9, scan 4 / 6, recurrence 3 / 5; a routed feed-forward is one more.
 template <typename T>
 int MixedDecoder<T>::decode_step(const int* tokens, const StepGeo& g, float* out, cudaStream_t s)
 {
@@ -744,11 +1179,13 @@ int MixedDecoder<T>::decode_step(const int* tokens, const StepGeo& g, float* out
     const int rows = g.rows();
     TRY(embed_rows(tokens, rows, s));
     float *cur = x, *next = x2;
-    const float* post = nullptr;
+    const float *post = nullptr, *sum = nullptr;
     auto chain = [&](const float* w_next, const float* extra) {
         GemvNorm f;
         f.y = y;
+        f.alpha = alpha;
         f.w_post = post;
+        f.w_sum = sum;
         f.x_in = cur;
         f.x_out = next;
         f.extra = extra;
@@ -761,10 +1198,27 @@ int MixedDecoder<T>::decode_step(const int* tokens, const StepGeo& g, float* out
     for (size_t r = 0; r < order.size(); r++) {
         const MixLayer<T>& L = layers[order[r].first];
         const RunState<T>& R = runs[r];
-        const GemvNorm f = r == 0 ? GemvNorm() : chain(L.norm1, order[r].second ? emb : nullptr);
-        const LinearArgs<T> in = product(L.in, h, w, w, proj, L.in.rows, false, rows, L.in_bias);
+        const GemvNorm f = r == 0 ? GemvNorm() : chain(norm_after ? nullptr : L.norm1, order[r].second ? emb : nullptr);
+        const LinearArgs<T> in = in_product(L, rows);
         GemvTail<T> t;
-        if (L.type != TLLM_MIXER_LATENT_ATTENTION) {
+        for (size_t i = 0; i < L.parts.size(); i++) {
+            const HeadPart& p = L.parts[i];
+            if (p.type != TLLM_MIXER_DELTA_RULE) continue;
+            t.kind = kTailConv;
+            t.lo = p.q;
+            t.hi = p.q + p.conv_channels();
+            t.taps = p.taps;
+            t.act = p.in_act;
+            t.w = p.conv;
+            t.carried = R.part[i].conv;
+            t.slot_stride = R.part[i].conv_slot;
+            t.first_slot = g.first_slot;
+            t.start_pos = g.start_pos;
+            t.pos_dev = g.pos_dev;
+            t.out = conv_out;
+            t.ld_out = p.conv_channels();
+        }
+        if (L.parts.empty() && L.type != TLLM_MIXER_LATENT_ATTENTION) {
             const bool scan = L.type == TLLM_MIXER_SELECTIVE_SCAN;
             t.kind = kTailConv;
             t.lo = scan ? 0 : L.ch;
@@ -782,7 +1236,9 @@ int MixedDecoder<T>::decode_step(const int* tokens, const StepGeo& g, float* out
             t.ld_out = L.ch;
         }
         TRY(launch_dense_gemv_fused<T>(in, f, t, s));
-        if (L.type == TLLM_MIXER_LATENT_ATTENTION) {
+        if (!L.parts.empty()) {
+            TRY(heads_inner(L, R, g, t.kind == kTailConv, s));
+        } else if (L.type == TLLM_MIXER_LATENT_ATTENTION) {
             TRY(attention_inner(L, R, g, s));
         } else if (L.type == TLLM_MIXER_SELECTIVE_SCAN) {
             TRY(project(L.x, conv_out, L.ch, L.ch, xdbc, L.x.rows, false, rows, s));
@@ -805,13 +1261,15 @@ int MixedDecoder<T>::decode_step(const int* tokens, const StepGeo& g, float* out
         }
         TRY(project(L.out, mixed, L.out.ld, L.out.ld, y, w, true, rows, s));
         post = L.norm1b;
-        if (L.ff) {
-            const GemvNorm n2 = chain(L.norm2, nullptr);
+        sum = norm_after ? L.norm1 : nullptr;
+        if (L.has_ff()) {
+            const GemvNorm n2 = chain(norm_after ? nullptr : L.norm2, nullptr);
             TRY(feed_forward(L, rows, &n2, s));
             post = L.norm2b;
+            sum = norm_after ? L.norm2 : nullptr;
         }
     }
-    return launch_dense_gemv_fused<T>(product(embed, h, w, w, out, vocab, true, rows), chain(final_norm, nullptr), GemvTail<T>(), s);
+    return launch_dense_gemv_fused<T>(head_product(rows, out), chain(final_norm, nullptr), GemvTail<T>(), s);
 }
 
 template <typename T>
@@ -828,29 +1286,47 @@ int MixedDecoder<T>::layers_pass(const int* tokens, const StepGeo& g, float* tap
     base.eps = eps;
     TRY(embed_rows(tokens, rows, s));
     base.y = y;
+    base.alpha = alpha;
     for (size_t r = 0; r < order.size(); r++) {
         const MixLayer<T>& L = layers[order[r].first];
         TRY(mixer(L, runs[r], g, s));
-        const float* post = L.norm1b;
-        if (L.ff) {
-            NormArgs<T> a = base;
-            a.w_post = post;
-            a.w_next = L.norm2;
+        NormArgs<T> a = base;
+        a.w_post = L.norm1b;
+        a.w_sum = norm_after ? L.norm1 : nullptr;
+        if (L.has_ff()) {
+            a.w_next = norm_after ? nullptr : L.norm2;
             TRY(launch_norm_chain<T>(a, s));
             TRY(feed_forward(L, rows, nullptr, s));
-            post = L.norm2b;
+            a = base;
+            a.w_post = L.norm2b;
+            a.w_sum = norm_after ? L.norm2 : nullptr;
+            if (gathers(L, rows)) {
+                a.y = nullptr;
+                a.parts = expert_out;
+                a.part_row = part_row;
+                a.part_w = part_w;
+                a.top = L.top;
+            }
         }
-        NormArgs<T> a = base;
-        a.w_post = post;
         a.tap = taps ? taps + r * tap_stride : nullptr;
         a.tap_width = width;
         if (r + 1 < order.size()) {
             a.extra = order[r + 1].second ? emb : nullptr;
-            a.w_next = layers[order[r + 1].first].norm1;
+            a.w_next = norm_after ? nullptr : layers[order[r + 1].first].norm1;
+        } else {
+            a.h = nullptr;
         }
         TRY(launch_norm_chain<T>(a, s));
     }
     return TLLM_OK;
+}
+
+template <typename T>
+LinearArgs<T> MixedDecoder<T>::head_product(int n, float* out) const
+{
+    LinearArgs<T> l = product(out_head, h, w, w, out, vocab, true, n, nullptr, softcap > 0.f ? kActSoftcap : kActNone);
+    l.act_param = softcap;
+    return l;
 }
 
 // final norm and output head of n rows of the residual stream
@@ -868,7 +1344,7 @@ int MixedDecoder<T>::head(const float* rows_x, const int* row_map, int n, float*
     a.w = w;
     a.eps = eps;
     TRY(launch_norm_chain<T>(a, s));
-    return project(embed, h, w, w, out, vocab, true, n, s);
+    return linear(head_product(n, out), s);
 }
 
 template <typename T>

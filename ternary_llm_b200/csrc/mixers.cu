@@ -53,40 +53,32 @@ norm_chain_kernel(const NormArgs<T> a)
     const int n4 = a.w >> 2;
     float* x = a.x + (size_t)src * a.w;
     float rinv = 1.f;
-    if (a.y && a.w_post) {
-        const float* y = a.y + (size_t)row * a.w;
+    auto branch = [&](int i) -> float4 {                // this row's y
+        if (!a.parts) return load4(a.y + (size_t)row * a.w + 4 * i);
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int k = 0; k < a.top; k++) {
+            const float4 v = load4(a.parts + (size_t)a.part_row[(size_t)row * a.top + k] * a.w + 4 * i);
+            const float p = a.part_w[(size_t)row * a.top + k];
+            s.x = fmaf(p, v.x, s.x);
+            s.y = fmaf(p, v.y, s.y);
+            s.z = fmaf(p, v.z, s.z);
+            s.w = fmaf(p, v.w, s.w);
+        }
+        return s;
+    };
+    const bool any = a.y || a.parts;
+    if (any && a.w_post) {
         float ss = 0.f;
         for (int i = threadIdx.x; i < n4; i += kNormThreads) {
-            const float4 v = load4(y + 4 * i);
+            const float4 v = branch(i);
             store4(vals + 4 * i, v);
             ss += sq4(v);
         }
         rinv = 1.0f / sqrtf(cta_sum(ss, sh) / (float)a.width + a.eps);
     }
     float ss = 0.f;
-    for (int i = threadIdx.x; i < n4; i += kNormThreads) {
-        float4 v;
-        if (a.table) {
-            v = load4(a.table + (size_t)a.tokens[row] * a.w + 4 * i);
-            if (a.emb) store4(a.emb + (size_t)row * a.w + 4 * i, v);
-        } else {
-            v = load4(x + 4 * i);
-        }
-        if (a.y) {
-            if (a.w_post) {
-                const float4 y = load4(vals + 4 * i), w = load4(a.w_post + 4 * i);
-                v.x += y.x * rinv * w.x;
-                v.y += y.y * rinv * w.y;
-                v.z += y.z * rinv * w.z;
-                v.w += y.w * rinv * w.w;
-            } else {
-                const float4 y = load4(a.y + (size_t)row * a.w + 4 * i);
-                v.x += y.x;
-                v.y += y.y;
-                v.z += y.z;
-                v.w += y.w;
-            }
-        }
+    auto finish = [&](int i, float4 v) {                // the new residual
         if (a.tap) {
             const float t[4] = {v.x, v.y, v.z, v.w};
             for (int j = 0; j < 4; j++)
@@ -102,8 +94,48 @@ norm_chain_kernel(const NormArgs<T> a)
         if (!a.row_map) store4(x + 4 * i, v);
         store4(vals + 4 * i, v);
         ss += sq4(v);
+    };
+    for (int i = threadIdx.x; i < n4; i += kNormThreads) {
+        float4 v;
+        if (a.table) {
+            v = load4(a.table + (size_t)a.tokens[row] * a.w + 4 * i);
+            if (a.emb) store4(a.emb + (size_t)row * a.w + 4 * i, v);
+        } else {
+            v = load4(x + 4 * i);
+        }
+        if (any) {
+            float4 y, w = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (a.w_post) {
+                y = load4(vals + 4 * i);
+                w = load4(a.w_post + 4 * i);
+            } else {
+                y = branch(i);
+            }
+            v.x = a.alpha * v.x + y.x * rinv * w.x;
+            v.y = a.alpha * v.y + y.y * rinv * w.y;
+            v.z = a.alpha * v.z + y.z * rinv * w.z;
+            v.w = a.alpha * v.w + y.w * rinv * w.w;
+        }
+        if (a.w_sum) {
+            store4(vals + 4 * i, v);
+            ss += sq4(v);
+        } else {
+            finish(i, v);
+        }
     }
-    if (!a.w_next) return;
+    if (a.w_sum) {
+        rinv = 1.0f / sqrtf(cta_sum(ss, sh) / (float)a.width + a.eps);
+        ss = 0.f;
+        for (int i = threadIdx.x; i < n4; i += kNormThreads) {
+            const float4 v = load4(vals + 4 * i), w = load4(a.w_sum + 4 * i);
+            finish(i, make_float4(v.x * rinv * w.x, v.y * rinv * w.y, v.z * rinv * w.z, v.w * rinv * w.w));
+        }
+    }
+    if (!a.h) return;
+    if (!a.w_next) {
+        for (int i = threadIdx.x; i < n4; i += kNormThreads) store4(a.h + (size_t)row * a.w + 4 * i, load4(vals + 4 * i));
+        return;
+    }
     rinv = 1.0f / sqrtf(cta_sum(ss, sh) / (float)a.width + a.eps);
     for (int i = threadIdx.x; i < n4; i += kNormThreads) {
         const float4 v = load4(vals + 4 * i), w = load4(a.w_next + 4 * i);

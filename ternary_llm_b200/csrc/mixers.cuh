@@ -16,17 +16,25 @@ struct StepGeo {
 };
 
 // One step of the residual chain, one CTA per row:
-//   x += y / rms(y) * w_post        (x += y when w_post is null; skipped when y is null)
+//   y = sum_s part_w[s] * parts[part_row[s]]   (when parts is not null: outputs of a token's experts)
+//   x = alpha x + y / rms(y) * w_post  (alpha x + y when w_post is null; skipped when there is no y)
+//   x = x / rms(x) * w_sum          (when w_sum is not null)
 //   tap = x                         (when tap is not null)
 //   x += extra                      (when extra is not null)
-//   h = x / rms(x) * w_next         (when w_next is not null)
+//   h = x / rms(x) * w_next         (when h is not null; h = x when w_next is null)
 // table / tokens not null: x = table[token] first (and emb = x when emb is not null).
 // row_map not null: row i of h comes from row row_map[i] of x (x is only read).
 // Widths are padded to `w` (a multiple of 8, padding zero everywhere); `width` divides the sums.
 template <typename T>
 struct NormArgs {
     const float* y = nullptr;
+    const T* parts = nullptr;          // [.., w]
+    const int* part_row = nullptr;     // [rows, top]
+    const float* part_w = nullptr;     // [rows, top]
+    int top = 0;
+    float alpha = 1.f;
     const float* w_post = nullptr;
+    const float* w_sum = nullptr;
     float* x = nullptr;
     float* tap = nullptr;
     int tap_width = 0;
@@ -144,5 +152,107 @@ int launch_latent_absorbed(const LatentArgs<T>& a, const T* q_abs, T* o_lat, flo
 // [heads][dim], vx [context][heads][vdim], out [rows][heads][vdim] times the output gate.
 bool latent_expanded_supported(const LatentArgs<bf16>& a);
 int launch_latent_expanded(const LatentArgs<bf16>& a, const bf16* kx, const bf16* vx, bf16* out, cudaStream_t stream);
+
+// ---- grouped-query attention --------------------------------------------------------------
+// Query head h reads key/value head h / (heads / kv_heads); per-head RMS norm of queries and keys
+// (optional), then rotation of the first rot_dims entries (i paired with i + rot_dims / 2).  With
+// `chunk` > 0 position i sees only the positions of its own chunk (i / chunk), counted from the
+// start of the sequence.  Cache row of a position: position % cache_rows, keys [kv_heads][dim]
+// and values [kv_heads][vdim] apart.  out = out_scale * softmax(scale q.k) v.
+template <typename T>
+struct GroupedArgs {
+    T* proj = nullptr;                 // rows of the step; queries, keys and values at these columns
+    int ld = 0, q_off = 0, k_off = 0, v_off = 0;
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0, dim_true = 0;   // dim, vdim: padded sizes
+    const float *q_norm = nullptr, *k_norm = nullptr;               // [dim] or null
+    float eps = 0.f;
+    const float2* rope = nullptr;      // [position][rot_dims / 2] (cos, sin)
+    int rot_dims = 0;
+    T *kc = nullptr, *vc = nullptr;    // [slot][cache_rows][kv_heads * dim], [..][kv_heads * vdim]
+    size_t k_slot = 0, v_slot = 0;     // elements
+    int cache_rows = 0, max_seq = 0, chunk = 0;
+    float scale = 0.f, out_scale = 1.f;
+    T* out = nullptr;                  // [rows, ld_out], heads * vdim entries
+    int ld_out = 0;
+    StepGeo g;
+};
+// cache rows that passes of up to `rows` tokens need
+int grouped_cache_rows(int max_seq, int chunk, int rows);
+bool grouped_supported(int heads, int kv_heads, int dim, int vdim);
+size_t grouped_workspace_floats(int heads, int vdim);
+// norms, rotations, cache append and attention of a step; ws: grouped_workspace_floats
+template <typename T>
+int launch_grouped_attention(const GroupedArgs<T>& a, float* ws, cudaStream_t stream);
+
+// ---- recurrences on a matrix per head ------------------------------------------------------
+// delta: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, with unit-length q (times
+//   q_scale) and k, g = exp(neg_a softplus(a + dt_bias)), beta = sigmoid(b);
+// else:  S <- decay S + k v^T; o = S^T q.
+// Head h reads query/key head h / (heads / kv_heads).  State [slot][heads][vdim][dim].
+template <typename T>
+struct MatrixScanArgs {
+    bool delta = false;
+    const T *q = nullptr, *k = nullptr, *v = nullptr;   // [rows, ld]
+    int ld = 0;
+    int heads = 0, kv_heads = 0, dim = 0, vdim = 0;     // padded sizes
+    const float* decay = nullptr;                        // [heads] (not delta)
+    const float *a = nullptr, *b = nullptr;              // [rows, ld_ab] (delta)
+    int ld_ab = 0;
+    const float *neg_a = nullptr, *dt_bias = nullptr;    // [heads]
+    float q_scale = 1.f;
+    float* state = nullptr;
+    size_t slot_stride = 0;
+    float* o = nullptr;                                  // [rows, heads * vdim]
+    void* ws = nullptr;                                  // matrix_scan_workspace bytes
+    StepGeo g;
+};
+// bytes for a step of `rows` tokens in all
+size_t matrix_scan_workspace(bool bf16_path, bool delta, int rows, int heads, int dim);
+template <typename T>
+int launch_matrix_scan(const MatrixScanArgs<T>& a, cudaStream_t stream);
+
+// out = out_scale * (o / rms(o) * w) * act(gate), the norm over groups of n entries (n_true of
+// them count), `groups` per row
+template <typename T>
+struct GatedNormArgs {
+    const float* o = nullptr;          // [rows, groups * n]
+    const float* w = nullptr;          // per_group ? [n] : [groups * n]
+    const T* gate = nullptr;           // [rows, ld_gate]
+    int ld_gate = 0, act = kActSilu;
+    float eps = 0.f, out_scale = 1.f;
+    T* out = nullptr;                  // [rows, ld_out]
+    int ld_out = 0;
+    int rows = 0, groups = 1, n = 0, n_true = 0;
+};
+template <typename T>
+int launch_gated_norm(const GatedNormArgs<T>& a, cudaStream_t stream);
+
+// ---- mixture of experts ----------------------------------------------------------------------
+// Router logits [rows, ld_z]; the `top` largest are chosen (the lower index on a tie) and weighed
+// by the softmax over them.  Few rows: the experts' rows are streamed for each token.  Many: the
+// tokens are gathered by expert, every expert's group padded to kGroupRows.
+template <typename T>
+struct ExpertArgs {
+    const float* z = nullptr;
+    int ld_z = 0, experts = 0, top = 0;
+    const T* h = nullptr;              // [rows, w]
+    int rows = 0, w = 0, ff = 0;       // padded sizes
+    const T *gate_up = nullptr, *down = nullptr;   // [experts * 2 ff, w], [experts * w, ff]
+    int act = kActSilu;
+    T* hidden = nullptr;               // few: [rows * top, ff]
+    float* y = nullptr;                // few: [rows, w]
+    // many
+    int* counts = nullptr;             // [2 * experts], zeroed by the launch
+    int *chosen = nullptr, *part_row = nullptr;    // [rows, top]
+    float* part_w = nullptr;                       // [rows, top]
+    T* gathered = nullptr;             // [expert_rows, w]
+    int *group = nullptr, *groups = nullptr;       // expert of every 128 rows; number of groups
+};
+int expert_rows(int rows, int top, int experts);   // capacity of the gathered rows
+bool experts_few_fits(int top, int ff, int w, size_t element);
+template <typename T>
+int launch_experts_few(const ExpertArgs<T>& a, cudaStream_t stream);
+template <typename T>
+int launch_experts_gather(const ExpertArgs<T>& a, cudaStream_t stream);
 
 }  // namespace tllm

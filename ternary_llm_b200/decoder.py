@@ -52,16 +52,24 @@ class Decoder:
             raise ValueError(f"dtype {dtype!r}: bfloat16 or float32")
         staging = []             # source tensors, needed only until create() has packed them
 
-        def up(a):
+        def on_device(a):
             if isinstance(a, torch.Tensor):
                 t = a.to(self.device).contiguous()
                 if t.dtype != torch.bfloat16:
                     raise TypeError(f"weights must be bfloat16, got {t.dtype}")
+                return t
+            a = np.array(a)
+            if a.dtype != np.uint16:
+                raise TypeError(f"weights must be BF16 bit patterns (uint16), got {a.dtype}")
+            return torch.from_numpy(a.view(np.int16)).to(self.device).view(torch.bfloat16)
+
+        def up(a):
+            if isinstance(a, list):                   # one behind the other
+                t = torch.empty((len(a),) + tuple(a[0].shape), dtype=torch.bfloat16, device=self.device)
+                for i, one in enumerate(a):
+                    t[i].copy_(on_device(one))
             else:
-                a = np.array(a)
-                if a.dtype != np.uint16:
-                    raise TypeError(f"weights must be BF16 bit patterns (uint16), got {a.dtype}")
-                t = torch.from_numpy(a.view(np.int16)).to(self.device)
+                t = on_device(a)
             staging.append(t)
             return t.data_ptr()
 

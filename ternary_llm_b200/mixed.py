@@ -5,9 +5,14 @@ Petulix: latent attention with a softmax sink and an output gate, Mamba, and Gri
 block in any order, a norm before and after every sublayer, an optional gated feed-forward per
 layer, a run of layers repeated with the embedding output added before each further pass, and
 the embedding table as output head.
+
+Femolix: gated delta rule, or chunk-local grouped-query attention beside linear attention of
+constant decay, in any order; a norm behind every sum of scaled residual and sublayer; a dense
+feed-forward, a mixture of experts or none per layer; a head of its own with a soft cap.
 """
 from __future__ import annotations
 
+import ctypes
 from dataclasses import dataclass, field
 
 import numpy as np
@@ -15,24 +20,27 @@ import numpy as np
 from . import _lib
 from .models import register
 
-LATENT_ATTENTION, SELECTIVE_SCAN, GATED_RECURRENCE = 1, 2, 3
-ACTIVATIONS = {None: 0, "gelu_tanh": 1, "silu": 2}
+LATENT_ATTENTION, SELECTIVE_SCAN, GATED_RECURRENCE, ATTENTION, LINEAR_ATTENTION, DELTA_RULE = range(1, 7)
+ACTIVATIONS = {None: 0, "gelu_tanh": 1, "silu": 2, "sigmoid": 4}
 
 # order of the TLLM_T_... enumeration
 TENSOR_SLOTS = ("norm1", "norm1b", "norm2", "norm2b", "gate", "up", "down", "out",
                 "q", "kv_down", "kv_norm", "k_up", "v_up", "sink", "head_gate",
                 "in", "in_bias", "conv", "conv_bias", "x", "dt", "dt_bias", "a_log", "d",
-                "y", "y_bias", "ra", "ra_bias", "ri", "ri_bias", "lam")
+                "y", "y_bias", "ra", "ra_bias", "ri", "ri_bias", "lam",
+                "k", "v", "q_norm", "k_norm", "q_conv", "k_conv", "v_conv", "step", "decay_in", "mix_norm", "mix_gate", "router")
 
 
 @dataclass
 class MixedLayer:
     """Sizes of one layer and its tensors (slot of TENSOR_SLOTS -> array of BF16 bit patterns or
-    a torch BF16 tensor)."""
+    a torch BF16 tensor; a list of equal ones is laid out one behind the other)."""
     type: int
     sizes: dict                                   # fields of tllm_b200_mixed_layer
     tensors: dict
-    shapes: dict = field(default_factory=dict)    # slot -> shape the sizes imply
+    shapes: dict = field(default_factory=dict)    # slot -> shape the sizes imply (of each in a list)
+    head_decay: object = None                     # floats, one per head
+    beside: "MixedLayer | None" = None            # a second mixer added to this layer's
 
 
 @dataclass
@@ -44,6 +52,9 @@ class MixedModel:
     embedding: object
     final_norm: object
     loop: tuple = (0, 0, 1, False)                # start, stop, times, add the embedding output before further passes
+    head: object = None                           # None: the embedding
+    residual_scale: float | None = None           # not None: norm(scale * x + sublayer(x)) instead of x + sublayer(norm(x))
+    logit_softcap: float = 0.0
     architecture = "mixed"
 
     def check(self) -> None:
@@ -51,29 +62,72 @@ class MixedModel:
         def shape(name, t, want):
             if tuple(t.shape) != tuple(want):
                 raise ValueError(f"tensor {name} is {tuple(t.shape)}, the configuration implies {tuple(want)}")
+
+        def mixer(layer, i):
+            for slot, t in layer.tensors.items():
+                for one in t if isinstance(t, list) else [t]:
+                    shape(f"{slot} of layer {i}", one, layer.shapes[slot])
+            if layer.head_decay is not None and len(layer.head_decay) != layer.sizes["heads"]:
+                raise ValueError(f"layer {i}: {len(layer.head_decay)} decays for {layer.sizes['heads']} heads")
+            if layer.beside is not None:
+                mixer(layer.beside, i)
+
         shape("embedding", self.embedding, (self.vocab_size, self.width))
         shape("final norm", self.final_norm, (self.width,))
+        if self.head is not None:
+            shape("head", self.head, (self.vocab_size, self.width))
         for i, layer in enumerate(self.layers):
-            for slot, t in layer.tensors.items():
-                shape(f"{slot} of layer {i}", t, layer.shapes[slot])
+            mixer(layer, i)
 
     def fill_desc(self, up, max_seq_len: int):
-        """tllm_b200_mixed_desc for this model; up(array) -> device pointer."""
+        """tllm_b200_mixed_desc for this model; up(array or list of arrays) -> device pointer."""
         self.check()
-        layers = (_lib.MixedLayerDesc * len(self.layers))()
-        for dst, layer in zip(layers, self.layers):
+        keep = []                                 # what the structures point to
+
+        def fill(dst, layer):
             dst.type = layer.type
             for k, v in layer.sizes.items():
                 setattr(dst, k, v)
             for slot, t in layer.tensors.items():
                 dst.t[TENSOR_SLOTS.index(slot)] = up(t)
+            if layer.head_decay is not None:
+                dst.head_decay = (ctypes.c_float * len(layer.head_decay))(*layer.head_decay)
+            if layer.beside is not None:
+                other = _lib.MixedLayerDesc()
+                fill(other, layer.beside)
+                keep.append(other)
+                dst.beside = ctypes.addressof(other)
+
+        layers = (_lib.MixedLayerDesc * len(self.layers))()
+        for dst, layer in zip(layers, self.layers):
+            fill(dst, layer)
         d = _lib.MixedDesc()
         d.vocab_size, d.width, d.n_layers, d.max_seq_len = self.vocab_size, self.width, len(self.layers), max_seq_len
         d.norm_eps = self.norm_eps
         d.loop_start, d.loop_stop, d.loop_times, d.loop_inject = self.loop
+        d.norm_after_sum, d.residual_scale = self.residual_scale is not None, self.residual_scale or 0.0
+        d.logit_softcap = self.logit_softcap
         d.embedding, d.final_norm = up(self.embedding), up(self.final_norm)
+        d.head = up(self.head) if self.head is not None else None
         d.layers = layers
+        d.keep = keep
         return d
+
+
+def _taker(tensors):
+    """name -> BF16 tensor of a model file, with the refusals."""
+    dtypes = getattr(tensors, "dtypes", {})
+
+    def take(name):
+        if isinstance(name, list):
+            return [take(n) for n in name]
+        if name not in tensors:
+            raise ValueError(f"tensor {name} is missing")
+        if dtypes.get(name, "BF16") != "BF16":
+            raise ValueError(f"tensor {name} is {dtypes[name]}, expected BF16")
+        return tensors[name]
+
+    return take
 
 
 def _latent_attention(m, width):
@@ -144,15 +198,7 @@ class Petulix(MixedModel):
 
     @classmethod
     def from_config(cls, cfg: dict, tensors) -> "Petulix":
-        dtypes = getattr(tensors, "dtypes", {})
-
-        def take(name):
-            if name not in tensors:
-                raise ValueError(f"tensor {name} is missing")
-            if dtypes.get(name, "BF16") != "BF16":
-                raise ValueError(f"tensor {name} is {dtypes[name]}, expected BF16")
-            return tensors[name]
-
+        take = _taker(tensors)
         layers = []
         for i, entry in enumerate(cfg["layers"]):
             kind, sizes, names = cls._layer(cfg, i, entry)
@@ -161,6 +207,98 @@ class Petulix(MixedModel):
         lp = cfg.get("loop")
         loop = (lp["start"], lp["stop"], lp["times"], True) if lp else (0, 0, 1, False)
         m = cls(cfg["vocab"], cfg["width"], cfg["norm"]["eps"], layers, take("embed"), take("final.norm"), loop)
+        m.check()
+        return m
+
+
+# ---- Femolix -------------------------------------------------------------------------------
+def _delta(m, width, prefix):
+    H, G, d, e, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+    sizes = dict(heads=H, kv_heads=G, dim=d, vdim=e, taps=taps, in_act=ACTIVATIONS["silu"], gate_act=ACTIVATIONS["silu"], out_scale=1.0)
+    names = {"q": ("q", (G * d, width)), "k": ("k", (G * d, width)), "v": ("v", (H * e, width)), "q_conv": ("q.conv", (G * d, taps)),
+             "k_conv": ("k.conv", (G * d, taps)), "v_conv": ("v.conv", (H * e, taps)), "step": ("b", (H, width)), "decay_in": ("a", (H, width)),
+             "a_log": ("A_log", (H,)), "dt_bias": ("dt_bias", (H,)), "mix_norm": ("norm", (e,)), "mix_gate": ("g", (H * e, width)),
+             "out": ("o", (width, H * e))}
+    return DELTA_RULE, sizes, {slot: (prefix + n, shape) for slot, (n, shape) in names.items()}
+
+
+def _chunked_attention(m, width, prefix, out_scale):
+    H, G, d, e, rot = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["rot"]
+    sizes = dict(heads=H, kv_heads=G, dim=d, vdim=e, rot_dims=rot["dims"], rot_base=rot["base"], scale=m["scale"], chunk=m["mask"]["size"],
+                 out_scale=out_scale)
+    names = {"q": ("q", (H * d, width)), "k": ("k", (G * d, width)), "v": ("v", (G * e, width)), "q_norm": ("q.norm", (d,)),
+             "k_norm": ("k.norm", (d,)), "out": ("o", (width, H * e))}
+    return ATTENTION, sizes, {slot: (prefix + n, shape) for slot, (n, shape) in names.items()}
+
+
+def _lightning(m, width, prefix, out_scale):
+    H, d, e = m["heads"], m["dim"], m["vdim"]
+    sizes = dict(heads=H, kv_heads=H, dim=d, vdim=e, in_act=ACTIVATIONS["silu"], gate_act=ACTIVATIONS["sigmoid"], out_scale=out_scale)
+    names = {"q": ("q", (H * d, width)), "k": ("k", (H * d, width)), "v": ("v", (H * e, width)), "mix_norm": ("norm", (H * e,)),
+             "mix_gate": ("g", (H * e, width)), "out": ("o", (width, H * e))}
+    return LINEAR_ATTENTION, sizes, {slot: (prefix + n, shape) for slot, (n, shape) in names.items()}
+
+
+@register("Femolix")
+class Femolix(MixedModel):
+    @staticmethod
+    def tensor_shapes(cfg: dict) -> dict:
+        """File name -> shape of every tensor of a model with this configuration."""
+        out = {"embed": (cfg["vocab"], cfg["width"])}
+        for i, entry in enumerate(cfg["layers"]):
+            for _, _, names in Femolix._mixers(cfg, i, entry):
+                for name, shape in names.values():
+                    out.update({n: shape for n in (name if isinstance(name, list) else [name])})
+        out["final.norm"] = (cfg["width"],)
+        out["head"] = (cfg["vocab"], cfg["width"])
+        return out
+
+    @staticmethod
+    def _mixers(cfg, i, entry):
+        """(type, sizes, slot -> (file name or names, shape)) of the layer, then of the mixer beside it."""
+        w, p, m = cfg["width"], f"l{i}.", entry["mixer"]
+        if entry["type"] == "delta":
+            mixers = [_delta(m, w, p + "mix.")]
+        elif entry["type"] == "parallel":
+            mixers = [_chunked_attention(m["left"], w, p + "mix.left.", m["left_scale"]),
+                      _lightning(m["right"], w, p + "mix.right.", m["right_scale"])]
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {entry['type']!r} (known: delta, parallel)")
+        _, sizes, names = mixers[0]
+        names["norm1"] = (p + "norm1", (w,))
+        mlp = entry.get("mlp")
+        if mlp is None:
+            return mixers
+        if mlp["kind"] not in ("dense", "moe"):
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        names["norm2"] = (p + "norm2", (w,))
+        sizes["ff_act"] = ACTIVATIONS["silu"]
+        if mlp["kind"] == "dense":
+            ff = sizes["ff"] = mlp["ff"]
+            names.update({"gate": (p + "mlp.gate", (ff, w)), "up": (p + "mlp.up", (ff, w)), "down": (p + "mlp.down", (w, ff))})
+            return mixers
+        ff, n, top = mlp["expert"]["ff"], mlp["router"]["experts"], mlp["router"]["top"]
+        if not 1 <= top <= n:
+            raise ValueError(f"layer {i}: {top} of {n} experts")
+        sizes.update(ff=ff, experts=n, top=top)
+        names["router"] = (p + "mlp.router", (n, w))
+        for slot, shape in (("gate", (ff, w)), ("up", (ff, w)), ("down", (w, ff))):
+            names[slot] = ([f"{p}mlp.e{e}.{slot}" for e in range(n)], shape)
+        return mixers
+
+    @classmethod
+    def from_config(cls, cfg: dict, tensors) -> "Femolix":
+        take = _taker(tensors)
+        layers = []
+        for i, entry in enumerate(cfg["layers"]):
+            made = [MixedLayer(kind, sizes, {slot: take(name) for slot, (name, _) in names.items()},
+                               {slot: shape for slot, (_, shape) in names.items()}) for kind, sizes, names in cls._mixers(cfg, i, entry)]
+            if len(made) == 2:
+                made[0].beside = made[1]
+                made[1].head_decay = list(entry["mixer"]["right"]["decay"])
+            layers.append(made[0])
+        m = cls(cfg["vocab"], cfg["width"], cfg["norm"]["eps"], layers, take("embed"), take("final.norm"), head=take("head"),
+                residual_scale=cfg["postln_alpha"], logit_softcap=cfg["logit_softcap"])
         m.check()
         return m
 
@@ -178,10 +316,10 @@ def random_tensors(shapes: dict, seed: int, device=None) -> dict:
         if last in ("norm1", "norm2", "norm1b", "norm2b", "norm"):
             t = torch.ones_like(t)
         elif last == "A_log":
-            t = torch.log(torch.arange(1, shape[1] + 1, device=t.device, dtype=torch.float32)).expand(shape) + 0.1 * t
+            t = torch.log(torch.arange(1, shape[-1] + 1, device=t.device, dtype=torch.float32)).expand(shape) + 0.1 * t
         elif last == "D":
             t = 1.0 + 0.1 * t
-        elif name.endswith("dt.b"):
+        elif name.endswith("dt.b") or last == "dt_bias":
             t = t - 4.0
         elif last == "lam":
             t = 0.5 * t - 2.0
