@@ -1038,16 +1038,45 @@ def mixed_config(size):
             "loop": {"start": 0, "stop": 0, "times": 1}}
 
 
-def mixed_case(torch, tl, dev, size, n_prompt, n_steps, eager):
-    """mixed:SIZE[:prompt[:steps[:eager]]] -- prefill and greedy decode of a model of mixer layers
-    with seeded random BF16 weights (1b, 8b; 1b-3l with `eager` for profilers)."""
+# Femolix at the same sizes: delta-rule and parallel layers in turn, a dense feed-forward in the first
+# and third of four layers, in the others a mixture whose chosen experts are as wide together
+FEMOLIX_SIZES = {
+    "1b": dict(heads=16, kv=4, r_heads=8, d_heads=16, experts=32, top=4),
+    "8b": dict(heads=32, kv=8, r_heads=16, d_heads=32, experts=16, top=4),
+}
+FEMOLIX_SIZES["1b-4l"] = FEMOLIX_SIZES["1b"]
+MIXED_SIZES["1b-4l"] = dict(MIXED_SIZES["1b"], n_layers=4, vocab=32000)      # every kind of layer, for profilers
+
+
+def femolix_config(size):
+    z, f = MIXED_SIZES[size], FEMOLIX_SIZES[size]
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "router": {"experts": f["experts"], "top": f["top"]}, "expert": {"ff": z["ff"] // f["top"]}}
+    delta = {"type": "delta", "mixer": {"heads": f["d_heads"], "kv_heads": f["d_heads"] // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    both = {"type": "parallel", "mixer": {
+        "left": {"heads": f["heads"], "kv_heads": f["kv"], "dim": 128, "vdim": 128, "mask": {"size": 1024},
+                 "rot": {"base": 10000.0, "dims": 128}, "scale": 128 ** -0.5}, "left_scale": 0.5, "right_scale": 0.5,
+        "right": {"heads": f["r_heads"], "dim": 128, "vdim": 128, "decay": (1 - 2.0 ** -np.linspace(3, 9, f["r_heads"])).tolist()}}}
+    kinds = [dict(delta, mlp=dense), dict(both, mlp=moe), dict(both, mlp=dense), dict(delta, mlp=moe)]
+    return {"architecture": "Femolix", "vocab": z["vocab"], "width": z["width"], "layers": [kinds[i % 4] for i in range(z["n_layers"])],
+            "norm": {"eps": 1e-5}, "postln_alpha": 2.0, "logit_softcap": 30.0}
+
+
+def mixed_case(torch, tl, dev, design, size, n_prompt, n_steps, eager):
+    """mixed:SIZE or femolix:SIZE[:prompt[:steps[:eager]]] -- prefill and greedy decode of a model of
+    mixer layers with seeded random BF16 weights (1b, 8b; mixed:1b-3l and femolix:1b-4l with `eager`
+    for profilers)."""
     from ternary_llm_b200 import mixed
-    cfg = mixed_config(size)
-    shapes = mixed.Petulix.tensor_shapes(cfg)
+    cls = mixed.Femolix if design == "femolix" else mixed.Petulix
+    cfg = femolix_config(size) if design == "femolix" else mixed_config(size)
+    shapes = cls.tensor_shapes(cfg)
     tensors = mixed.random_tensors(shapes, 2026, dev)
-    # every matrix is read once per token (the embedding table as output head)
-    weight_bytes = 2 * sum(int(np.prod(s)) for s in shapes.values())
-    dec = tl.Decoder(mixed.Petulix.from_config(cfg, tensors), max_seq_len=n_prompt + n_steps + 8)
+    # what a token uses: every matrix once (an untied embedding: one row), of the experts the chosen ones
+    weight_bytes = 2 * sum(int(np.prod(s)) for n, s in shapes.items() if not (n == "embed" and "head" in shapes) and ".mlp.e" not in n)
+    for layer in cfg["layers"]:
+        if layer["mlp"]["kind"] == "moe":
+            weight_bytes += 2 * 3 * cfg["width"] * layer["mlp"]["expert"]["ff"] * layer["mlp"]["router"]["top"]
+    dec = tl.Decoder(cls.from_config(cfg, tensors), max_seq_len=n_prompt + n_steps + 8)
     del tensors
     prompt = torch.from_numpy(np.random.default_rng(0).integers(0, cfg["vocab"], n_prompt).astype(np.int32)).to(dev)
     first = int(dec.forward(prompt, 0).argmax().item())
@@ -1086,7 +1115,7 @@ def mixed_case(torch, tl, dev, size, n_prompt, n_steps, eager):
 def run_case(args):
     """A small single-kernel case for profilers: `gemv:NxK[:copies]`, `gemv_int8:NxK[:copies]`
     `gemm:MxNxK`, or `decode:ARCH[:prompt[:steps[:eager]]]` (the decoder on a random model), or
-    `mixed:SIZE[:prompt[:steps[:eager]]]` (mixed_case).
+    `mixed:SIZE[:prompt[:steps[:eager]]]`, `femolix:...` alike (mixed_case).
     Distinct matrices are cycled so that the weights come from HBM."""
     import torch
 
@@ -1136,8 +1165,8 @@ def run_case(args):
         c = torch.zeros(m, n, device=dev, dtype=torch.float16)
         for _ in range(4):
             tl.ternary_gemm_packed(a, w, c, m)
-    elif kind == "mixed":
-        info = mixed_case(torch, tl, dev, dims, int(rest[0]) if rest else 2048, int(rest[1]) if len(rest) > 1 else 64,
+    elif kind in ("mixed", "femolix"):
+        info = mixed_case(torch, tl, dev, kind, dims, int(rest[0]) if rest else 2048, int(rest[1]) if len(rest) > 1 else 64,
                           len(rest) > 2 and rest[2] == "eager")
         print(json.dumps({"case": args.case, "status": "ok", **info}))
         return

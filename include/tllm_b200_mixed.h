@@ -173,6 +173,31 @@ int tllm_b200_latent_attention_expanded(const void* q, const void* kx, const voi
                                         const void* gate, void* o, int heads, int dim, int rot, int vdim, int rank, float scale,
                                         int max_seq, int seq_len, int start_pos, void* stream);
 
+/* Norms, rotation, cache append and attention of a step (TLLM_MIXER_ATTENTION): proj [rows,
+ * heads * dim + kv_heads * (dim + vdim)] = q, k, v (q is overwritten); norms float [dim] or NULL;
+ * rope float [positions][rot_dims / 2][2] = cos, sin; kc [n_seq][cache_rows][kv_heads * dim], vc
+ * alike; position p is cache row p % cache_rows, so cache_rows is at least chunk + seq_len, or all
+ * positions; o [rows, heads * vdim]. */
+int tllm_b200_grouped_attention(int bf16, void* proj, const float* q_norm, const float* k_norm, float eps, const float* rope, int rot_dims,
+                                void* kc, void* vc, void* o, int heads, int kv_heads, int dim, int vdim, int chunk, int cache_rows, int max_seq,
+                                float scale, float out_scale, int n_seq, int seq_len, int start_pos, void* stream);
+/* Linear attention (delta = 0: decay float [heads], kv_heads = heads) or the gated delta rule
+ * (delta = 1: a, b float [rows, heads], neg_a = -exp(A_log) and dt_bias float [heads]): q, k [rows,
+ * kv_heads * dim], v [rows, heads * vdim] as one row q, k, v each; state float
+ * [n_seq][heads][vdim][dim]; o float [rows, heads * vdim]. */
+int tllm_b200_matrix_scan(int bf16, int delta, const void* qkv, const float* decay, const float* a, const float* b, const float* neg_a,
+                          const float* dt_bias, float q_scale, float* state, float* o, int heads, int kv_heads, int dim, int vdim, int n_seq,
+                          int seq_len, int start_pos, void* stream);
+/* out = out_scale * o / rms(o) * w * act(gate): o float, gate and out [rows, groups * n], the norm
+ * over each group of n; w float [n]. */
+int tllm_b200_gated_norm(int bf16, const float* o, const float* w, const void* gate, void* out, int rows, int groups, int n, float eps,
+                         float out_scale, int act, void* stream);
+/* y float [rows, width] = sum over the `top` experts with the largest z (softmax over them) of
+ * down (act(gate h) * up h); z float [rows, experts]; gate_up [experts][2 * ff, width], down
+ * [experts][width, ff]. */
+int tllm_b200_experts(int bf16, const void* h, const float* z, const void* gate_up, const void* down, float* y, int rows, int width, int ff,
+                      int experts, int top, int act, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

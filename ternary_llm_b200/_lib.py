@@ -71,6 +71,11 @@ SIGNATURES = {
     "tllm_b200_gated_scan": (_int, [_int] + [_vp] * 6 + [_int, _int, ctypes.c_float] + [_int] * 4 + [_vp]),
     "tllm_b200_latent_attention": (_int, [_int] + [_vp] * 4 + [_int] * 3 + [ctypes.c_float] + [_int] * 4 + [_vp]),
     "tllm_b200_latent_attention_expanded": (_int, [_vp] * 7 + [_int] * 5 + [ctypes.c_float] + [_int] * 3 + [_vp]),
+    "tllm_b200_grouped_attention": (_int, [_int] + [_vp] * 3 + [ctypes.c_float, _vp, _int] + [_vp] * 3 + [_int] * 7 + [ctypes.c_float] * 2 +
+                                    [_int] * 3 + [_vp]),
+    "tllm_b200_matrix_scan": (_int, [_int, _int] + [_vp] * 6 + [ctypes.c_float, _vp, _vp] + [_int] * 7 + [_vp]),
+    "tllm_b200_gated_norm": (_int, [_int] + [_vp] * 4 + [_int] * 3 + [ctypes.c_float] * 2 + [_int, _vp]),
+    "tllm_b200_experts": (_int, [_int] + [_vp] * 5 + [_int] * 6 + [_vp]),
 }
 
 TENSORS_PER_LAYER = 43      # TLLM_T_COUNT

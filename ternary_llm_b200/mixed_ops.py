@@ -83,3 +83,54 @@ def latent_attention_expanded(q, kx, vx, cache, sink, gate, o, heads: int, dim: 
         _chk(q, t, "q", seq_len * heads * (dim + rot)), _chk(kx, t, "kx", ctx * heads * dim), _chk(vx, t, "vx", ctx * heads * vdim),
         _chk(cache, t, "cache", max_seq * (rank + rot)), _opt(sink, _F, "sink", heads), _opt(gate, t, "gate", seq_len * heads),
         _chk(o, t, "o", seq_len * heads * vdim), heads, dim, rot, vdim, rank, scale, max_seq, seq_len, start_pos, _stream()))
+
+
+def grouped_attention(proj, q_norm, k_norm, eps: float, rope, rot_dims: int, kc, vc, o, heads: int, kv_heads: int, dim: int, vdim: int,
+                      chunk: int, cache_rows: int, max_seq: int, scale: float, n_seq: int, seq_len: int, start_pos: int,
+                      out_scale: float = 1.0) -> None:
+    """Per-head norms, rotation, cache append and attention of a step; proj [rows, q | k | v]
+    (q is overwritten), rope [max_seq, rot_dims / 2, 2] = cos, sin, caches [n_seq, cache_rows, ..]."""
+    t, rows = proj.dtype, n_seq * seq_len
+    _lib.check(_lib.lib().tllm_b200_grouped_attention(
+        _kind(proj), _chk(proj, t, "proj", rows * (heads * dim + kv_heads * (dim + vdim))), _opt(q_norm, _F, "q_norm", dim),
+        _opt(k_norm, _F, "k_norm", dim), eps, _opt(rope, _F, "rope", max_seq * rot_dims), rot_dims,
+        _chk(kc, t, "kc", n_seq * cache_rows * kv_heads * dim), _chk(vc, t, "vc", n_seq * cache_rows * kv_heads * vdim),
+        _chk(o, t, "o", rows * heads * vdim), heads, kv_heads, dim, vdim, chunk, cache_rows, max_seq, scale, out_scale, n_seq, seq_len,
+        start_pos, _stream()))
+
+
+def linear_attention(qkv, decay, state, o, heads: int, dim: int, vdim: int, n_seq: int, seq_len: int, start_pos: int) -> None:
+    """S = decay S + k v^T, o = S^T q; qkv [rows, q | k | v], state [n_seq, heads, vdim, dim]."""
+    rows = n_seq * seq_len
+    _lib.check(_lib.lib().tllm_b200_matrix_scan(
+        _kind(qkv), 0, _chk(qkv, qkv.dtype, "qkv", rows * heads * (2 * dim + vdim)), _chk(decay, _F, "decay", heads), None, None, None, None, 1.0,
+        _chk(state, _F, "state", n_seq * heads * dim * vdim), _chk(o, _F, "o", rows * heads * vdim), heads, heads, dim, vdim, n_seq, seq_len,
+        start_pos, _stream()))
+
+
+def delta_rule(qkv, a, b, neg_a, dt_bias, q_scale: float, state, o, heads: int, kv_heads: int, dim: int, vdim: int, n_seq: int, seq_len: int,
+               start_pos: int) -> None:
+    """S = g S, u = beta (v - S^T k), S = S + k u^T, o = S^T q with unit-length q (times q_scale)
+    and k, g = exp(neg_a softplus(a + dt_bias)), beta = sigmoid(b)."""
+    rows = n_seq * seq_len
+    _lib.check(_lib.lib().tllm_b200_matrix_scan(
+        _kind(qkv), 1, _chk(qkv, qkv.dtype, "qkv", rows * (2 * kv_heads * dim + heads * vdim)), None, _chk(a, _F, "a", rows * heads),
+        _chk(b, _F, "b", rows * heads), _chk(neg_a, _F, "neg_a", heads), _chk(dt_bias, _F, "dt_bias", heads), q_scale,
+        _chk(state, _F, "state", n_seq * heads * dim * vdim), _chk(o, _F, "o", rows * heads * vdim), heads, kv_heads, dim, vdim, n_seq, seq_len,
+        start_pos, _stream()))
+
+
+def gated_norm(o, w, gate, out, rows: int, groups: int, n: int, eps: float, act="silu", out_scale: float = 1.0) -> None:
+    """out = out_scale * o / rms(o) * w * act(gate), the norm over each group of n entries."""
+    t = gate.dtype
+    _lib.check(_lib.lib().tllm_b200_gated_norm(
+        _kind(gate), _chk(o, _F, "o", rows * groups * n), _chk(w, _F, "w", n), _chk(gate, t, "gate", rows * groups * n),
+        _chk(out, t, "out", rows * groups * n), rows, groups, n, eps, out_scale, ACTIVATIONS[act], _stream()))
+
+
+def experts(h, z, gate_up, down, y, rows: int, width: int, ff: int, n: int, top: int, act="silu") -> None:
+    """Weighted sum of the outputs of the `top` experts with the largest z, softmax over them."""
+    t = h.dtype
+    _lib.check(_lib.lib().tllm_b200_experts(
+        _kind(h), _chk(h, t, "h", rows * width), _chk(z, _F, "z", rows * n), _chk(gate_up, t, "gate_up", n * 2 * ff * width),
+        _chk(down, t, "down", n * width * ff), _chk(y, _F, "y", rows * width), rows, width, ff, n, top, ACTIVATIONS[act], _stream()))
