@@ -171,7 +171,7 @@ int matrix_op(int delta, const void* qkv, const float* decay, const float* a, co
     m.o = o;
     m.g = g;
     float* ws = nullptr;
-    return with_records((matrix_scan_workspace(sizeof(T) == 2, m.delta, g.rows(), heads, dim) + 3) / 4, &ws, s, [&] {
+    return with_records((matrix_scan_workspace(sizeof(T) == 2, m.delta, g.rows(), heads, kv_heads, dim, vdim) + 3) / 4, &ws, s, [&] {
         m.ws = ws;
         return launch_matrix_scan<T>(m, s);
     });
@@ -193,12 +193,12 @@ int experts_op(const void* h, const float* z, const void* gate_up, const void* d
     a.down = static_cast<const T*>(down);
     a.act = act;
     a.y = y;
-    const bool few = rows <= 8 && experts_few_fits(top, ff, w, sizeof(T));
+    const bool few = rows <= 8 && gemv_routed_fits(top, ff, sizeof(T));
     const int m = expert_rows(rows, top, n), k = rows * top;
     // hidden, gathered rows, outputs; counts, choices, places, weights, groups
     const size_t es = sizeof(T), n_hidden = (size_t)(few ? k : m) * ff, n_rows = few ? 0 : (size_t)m * w;
     float* ws = nullptr;
-    return with_records((n_hidden + 2 * n_rows) * es / 4 + 2 * (size_t)n + 3 * (size_t)k + m / kGroupRows + 64, &ws, s, [&]() -> int {
+    return with_records((n_hidden + 2 * n_rows) * es / 4 + 2 * (size_t)n + 3 * (size_t)k + 3 * (m / kGroupRows) + 64, &ws, s, [&]() -> int {
         a.hidden = reinterpret_cast<T*>(ws);
         if (few) return launch_experts_few<T>(a, s);
         a.gathered = a.hidden + n_hidden;

@@ -35,11 +35,17 @@ struct LinearArgs {
     float* y2 = nullptr;
     int ldy2 = 0;
     // rows in groups with a matrix each (entries of w, w_rows apart): 128 rows from 128 i on use
-    // entry group[i], i < *groups (both on the device); entries: matrices in w
+    // entry group[3 i], i < *groups (both on the device); group[3 i + 1], [3 i + 2]: first of the
+    // groups with this entry and their number; entries: matrices in w
     const int *group = nullptr, *groups = nullptr;
     int entries = 0;
     // glu: w holds N gate rows followed by N up rows; y = act(gate) * up
     bool glu = false;
+    // rows with chosen entries (launch_dense_gemv_routed)
+    struct {
+        const float* z = nullptr;    // logits [M, ld_z]
+        int ld_z = 0, experts = 0, top = 0;
+    } route;
     const T* gate = nullptr;     // y *= sigmoid(gate[m * gate_ld + z])
     int gate_ld = 0;
 };
@@ -94,6 +100,12 @@ int launch_dense_gemv(const LinearArgs<T>& a, cudaStream_t stream);
 // at most 8 vectors
 template <typename T>
 int launch_dense_gemv_fused(const LinearArgs<T>& a, const GemvNorm& norm, const GemvTail<T>& tail, cudaStream_t stream);
+// A row's chosen entries.  sum = false: row (m * top + s) of y is the (gated) product of row m of x
+// with its s-th entry; sum = true: row m of y is the weighted sum over s of the products of entry s
+// with columns s * K .. of row m of x.
+template <typename T>
+int launch_dense_gemv_routed(const LinearArgs<T>& a, bool sum, cudaStream_t stream);
+bool gemv_routed_fits(int top, int k, size_t element);
 // the tails need this many lanes per row
 template <typename T>
 bool gemv_tail_fits(int k, int taps);

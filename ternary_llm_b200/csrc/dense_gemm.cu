@@ -116,13 +116,23 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
     volatile int* abortp = &abort_flag;
     int never = 0;
     pdl_wait();
-    // tile -> first token, first feature, batch entry; tokens vary fastest (neighbours share W)
-    const int mt = a.group ? min(*a.groups, a.mt) : a.mt, tiles = a.group ? mt * a.nt : a.tiles;
-    auto where = [&](int tile, int& m0, int& n0, int& z) {
-        m0 = (tile % mt) * kTok;
-        tile /= mt;
+    // tile -> first token, first feature, batch entry, entry of W; tokens vary fastest (neighbours
+    // share W), with grouped rows those of one entry
+    const int tiles = a.group ? min(*a.groups, a.mt) * a.nt : a.tiles;
+    auto where = [&](int tile, int& m0, int& n0, int& z, int& entry) {
+        if (a.group) {
+            const int* g = a.group + 3 * (tile / a.nt);
+            const int first = g[1], count = g[2], r = tile - first * a.nt, n = r / count;
+            m0 = (first + r - n * count) * kTok;
+            n0 = n * outs;
+            z = 0;
+            entry = g[0];
+            return;
+        }
+        m0 = (tile % a.mt) * kTok;
+        tile /= a.mt;
         n0 = (tile % a.nt) * outs;
-        z = tile / a.nt;
+        entry = z = tile / a.nt;
     };
 
     if (warp == 0) {
@@ -131,9 +141,9 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
             int it = 0;                                  // stages filled so far, over all tiles
             bool ok = true;
             for (int tile = blockIdx.x; ok && tile < tiles; tile += gridDim.x) {
-                int m0, n0, z;
-                where(tile, m0, n0, z);
-                const int wr0 = (a.group ? a.group[m0 / kTok] : z) * a.w_rows + n0, wr1 = a.glu ? wr0 + a.N : wr0 + TN / 2;
+                int m0, n0, z, entry;
+                where(tile, m0, n0, z, entry);
+                const int wr0 = entry * a.w_rows + n0, wr1 = a.glu ? wr0 + a.N : wr0 + TN / 2;
                 for (int k = 0; k < nk; k++, it++) {
                     const int s = it % kStages;
                     if (!mbar_wait(empty(s), ((it / kStages) & 1) ^ 1, abortp)) {
@@ -202,8 +212,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_consta
                 break;
             }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            int m0, n0, z;
-            where(tile, m0, n0, z);
+            int m0, n0, z, entry;
+            where(tile, m0, n0, z, entry);
             const int mrow = m0 + row0;
             const float hg = (a.gate && mrow + lane < a.M) ? sigmoid_f(__bfloat162float(a.gate[(size_t)(mrow + lane) * a.gate_ld + z])) : 1.f;
             const int ncols = min(outs, a.N - n0);

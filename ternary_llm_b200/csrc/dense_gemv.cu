@@ -11,6 +11,7 @@
 // launch leaves room on the SM for the next one to do the same.
 #include "dense.cuh"
 #include "launch.cuh"
+#include "route.cuh"
 
 namespace tllm {
 
@@ -120,7 +121,11 @@ __device__ __forceinline__ void stage_norm(const GemvNorm& f, int m, int K, T* x
     __syncthreads();             // the next vector's sums reuse sh
 }
 
-template <typename T, int MB, bool NORM, int TAIL>
+enum Route { kRouteNone = 0, kRouteEach = 1, kRouteSum = 2 };
+
+// ROUTE (one vector per CTA, blockIdx.y = place in y): the entries of w are chosen from the row's
+// logits, so nothing is requested before the wait.
+template <typename T, int MB, bool NORM, int TAIL, int ROUTE = kRouteNone>
 __global__ void __launch_bounds__(kWarps * 32)
 dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, int lanes_per_row, int m0)
 {
@@ -132,12 +137,16 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int sub = lane / lanes_per_row, l = lane - sub * lanes_per_row, rpw = 32 / lanes_per_row;
-    const int z = blockIdx.y;
+    const int z = ROUTE ? 0 : blockIdx.y;
+    const int xr = ROUTE == kRouteEach ? blockIdx.y / a.route.top : blockIdx.y;      // row of x (ROUTE)
     const int nv = a.K / V;                                  // 16-byte pieces per row
     const int stride = gridDim.x * kWarps * rpw;
     const int nb0 = (blockIdx.x * kWarps + warp) * rpw;
-    const int parts = (TAIL == kTailGate || a.glu) ? 2 : 1;
+    const int parts = ROUTE == kRouteSum ? a.route.top : (TAIL == kTailGate || a.glu) ? 2 : 1;
     const T* wz = a.w + (size_t)z * a.w_rows * a.ldw;
+    // ROUTE: weights and entries of the choice behind the vectors
+    float* wgt = reinterpret_cast<float*>(xs + (size_t)(ROUTE == kRouteSum ? parts : MB) * a.K);
+    int* idx = reinterpret_cast<int*>(wgt + a.route.top);
 
     // ring of this lane: piece u of slot s at ring[(s * kPieces + u) * threads]
     const uint4* ring = reinterpret_cast<const uint4*>(smem_raw) + threadIdx.x;
@@ -146,7 +155,8 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
     auto request = [&]() {
         if (f_nb < a.N) {
             const int n = f_nb + sub;
-            const T* row = wz + (size_t)(n < a.N ? n + f_part * a.N : 0) * a.ldw;
+            const size_t r = n < a.N ? (ROUTE == kRouteSum ? (size_t)idx[f_part] * a.w_rows + n : (size_t)n + f_part * a.N) : 0;
+            const T* row = wz + r * a.ldw;
 #pragma unroll
             for (int u = 0; u < kPieces; u++) {
                 const int c = f_c + u * lanes_per_row + l;
@@ -165,8 +175,10 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
         asm volatile("cp.async.commit_group;" ::: "memory");
         f_slot = f_slot == kGroups - 1 ? 0 : f_slot + 1;
     };
+    if (!ROUTE) {
 #pragma unroll
-    for (int g = 0; g < kGroups; g++) request();
+        for (int g = 0; g < kGroups; g++) request();
+    }
     if (NORM) {
         float* wn = reinterpret_cast<float*>(xs + (size_t)MB * a.K);
         const float* w[3] = {f.w_next, f.w_post, f.w_sum};
@@ -179,8 +191,17 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
     }
 
     pdl_wait();
-    const int mb = min(MB, a.M - m0);
-    if (NORM) {
+    const int mb = ROUTE ? 1 : min(MB, a.M - m0);
+    if (ROUTE) {
+        if (warp == 0) choose_experts(a.route.z + (size_t)xr * a.route.ld_z, a.route.experts, a.route.top, idx, wgt);
+        const int n16 = ROUTE == kRouteSum ? parts * nv : nv;
+        for (int i = (int)threadIdx.x - 32; i < n16; i += (kWarps - 1) * 32)
+            if (i >= 0) reinterpret_cast<uint4*>(xs)[i] = *(reinterpret_cast<const uint4*>(a.x + (size_t)xr * a.ldx) + i);
+        __syncthreads();
+        if (ROUTE == kRouteEach) wz += (size_t)idx[blockIdx.y - xr * a.route.top] * a.w_rows * a.ldw;
+#pragma unroll
+        for (int g = 0; g < kGroups; g++) request();
+    } else if (NORM) {
         const float* wn = reinterpret_cast<const float*>(xs + (size_t)MB * a.K);
         const float* wp = wn + (f.w_next ? a.K : 0);
         const float* ws = wp + (f.w_post ? a.K : 0);
@@ -192,7 +213,7 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
                 *(reinterpret_cast<const uint4*>(a.x + (size_t)(m0 + m) * a.ldx + (size_t)z * a.x_batch) + c);
         }
     }
-    for (int i = threadIdx.x + mb * nv; i < MB * nv; i += kWarps * 32) reinterpret_cast<uint4*>(xs)[i] = make_uint4(0, 0, 0, 0);
+    for (int i = threadIdx.x + mb * nv; i < (ROUTE ? 0 : MB * nv); i += kWarps * 32) reinterpret_cast<uint4*>(xs)[i] = make_uint4(0, 0, 0, 0);
     const bool fresh = TAIL != kTailNone && (t.pos_dev ? *t.pos_dev : t.start_pos) == 0;
     __syncthreads();
 
@@ -235,7 +256,7 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
 #pragma unroll
                     for (int m = 0; m < MB; m++) {
                         float xf[V];
-                        Vec16<T>::unpack(*(reinterpret_cast<const uint4*>(xs + (size_t)m * a.K) + c), xf);
+                        Vec16<T>::unpack(*(reinterpret_cast<const uint4*>(xs + (size_t)(ROUTE == kRouteSum ? part : m) * a.K) + c), xf);
 #pragma unroll
                         for (int j = 0; j < V; j++) acc[m] = fmaf(wf[j], xf[j], acc[m]);
                     }
@@ -246,7 +267,8 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
 #pragma unroll
             for (int m = 0; m < MB; m++) {
                 for (int o = lanes_per_row >> 1; o > 0; o >>= 1) acc[m] += __shfl_xor_sync(0xffffffffu, acc[m], o);
-                if (part == 0) res[0][m] = acc[m];
+                if (ROUTE == kRouteSum) res[0][m] = part == 0 ? wgt[0] * acc[m] : fmaf(wgt[part], acc[m], res[0][m]);
+                else if (part == 0) res[0][m] = acc[m];
                 else res[1][m] = acc[m];
             }
         }
@@ -290,7 +312,7 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
             if (n >= a.act_lo && n < a.act_hi) v = apply_act(a.act, v, a.act_param);
             if (a.glu) v *= res[1][m];
             if (a.gate) v *= sigmoid_f(to_f<T>(a.gate[(size_t)(m0 + m) * a.gate_ld + z]));
-            const size_t o = (size_t)(m0 + m) * a.ldy + (size_t)z * a.y_batch + n;
+            const size_t o = (size_t)(ROUTE ? (int)blockIdx.y : m0 + m) * a.ldy + (size_t)z * a.y_batch + n;
             if (a.y_f32) static_cast<float*>(a.y)[o] = v;
             else static_cast<T*>(a.y)[o] = from_f<T>(v);
         }
@@ -330,6 +352,30 @@ int launch_mb(const LinearArgs<T>& a, const GemvNorm& f, const GemvTail<T>& t, i
     const size_t smem = kRingBytes + (size_t)MB * a.K * sizeof(T) + (size_t)norms * a.K * sizeof(float);
     if (smem > kSmemLimit || (NORM && a.K > kNormMaxK)) return fail(TLLM_ERR_SHAPE, "dense_gemv: %d vectors of %d", MB, a.K);
     return launch_pdl("dense_gemv", dense_gemv_kernel<T, MB, NORM, TAIL>, dim3(grid, a.batch), dim3(kWarps * 32), smem, stream, a, f, t, lpr, m0);
+}
+
+size_t routed_smem(int top, int k, size_t element, bool sum) { return kRingBytes + (size_t)(sum ? top : 1) * k * element + (size_t)top * 8; }
+
+template <typename T, int ROUTE>
+int launch_routed(const LinearArgs<T>& a, cudaStream_t stream)
+{
+    static bool attr[64] = {};
+    static int sms[64] = {};
+    int dev = 0;
+    cudaGetDevice(&dev);
+    const auto kernel = dense_gemv_kernel<T, 1, false, kTailNone, ROUTE>;
+    if (!attr[dev]) {
+        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemLimit);
+        cudaDeviceGetAttribute(&sms[dev], cudaDevAttrMultiProcessorCount, dev);
+        attr[dev] = true;
+    }
+    const size_t smem = routed_smem(a.route.top, a.K, sizeof(T), ROUTE == kRouteSum);
+    if (smem > kSmemLimit) return fail(TLLM_ERR_SHAPE, "dense_gemv: %d entries of K=%d do not fit shared memory", a.route.top, a.K);
+    const int lpr = row_lanes<T>(a.K), rows_per_cta = kWarps * (32 / lpr), ny = ROUTE == kRouteSum ? a.M : a.M * a.route.top;
+    int grid = (a.N + rows_per_cta - 1) / rows_per_cta;
+    const int cap = (2 * sms[dev] + ny - 1) / ny;
+    if (grid > cap) grid = cap;
+    return launch_pdl("dense_gemv_routed", kernel, dim3(grid, ny), dim3(kWarps * 32), smem, stream, a, GemvNorm(), GemvTail<T>(), lpr, 0);
 }
 
 template <typename T, bool NORM, int TAIL>
@@ -388,6 +434,19 @@ int launch_dense_gemv_fused(const LinearArgs<T>& a, const GemvNorm& f, const Gem
 template int launch_dense_gemv_fused<bf16>(const LinearArgs<bf16>&, const GemvNorm&, const GemvTail<bf16>&, cudaStream_t);
 template int launch_dense_gemv_fused<float>(const LinearArgs<float>&, const GemvNorm&, const GemvTail<float>&, cudaStream_t);
 
+bool gemv_routed_fits(int top, int k, size_t element) { return routed_smem(top, k, element, true) <= kSmemLimit; }
+
+template <typename T>
+int launch_dense_gemv_routed(const LinearArgs<T>& a, bool sum, cudaStream_t stream)
+{
+    if (a.M == 0 || a.N == 0) return TLLM_OK;
+    const int st = check_gemv(a);
+    if (st) return st;
+    return sum ? launch_routed<T, kRouteSum>(a, stream) : launch_routed<T, kRouteEach>(a, stream);
+}
+template int launch_dense_gemv_routed<bf16>(const LinearArgs<bf16>&, bool, cudaStream_t);
+template int launch_dense_gemv_routed<float>(const LinearArgs<float>&, bool, cudaStream_t);
+
 template <typename T>
 int launch_dense_gemv(const LinearArgs<T>& a, cudaStream_t stream)
 {
@@ -432,7 +491,7 @@ dense_gemm_f32_kernel(const LinearArgs<float> a)
     float acc[2][4][4] = {};
     pdl_wait();
     if (a.group && m0 / kGroupRows >= *a.groups) return;
-    const float* wz = a.w + (size_t)(a.group ? a.group[m0 / kGroupRows] : z) * a.w_rows * a.ldw;
+    const float* wz = a.w + (size_t)(a.group ? a.group[3 * (m0 / kGroupRows)] : z) * a.w_rows * a.ldw;
     const float* xz = a.x + (size_t)z * a.x_batch;
     const int lr = threadIdx.x >> 2, lc = (threadIdx.x & 3) * 4;  // loader: row of the tile, 4 columns
     for (int k0 = 0; k0 < a.K; k0 += kSlice) {

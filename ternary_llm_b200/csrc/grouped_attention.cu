@@ -49,6 +49,67 @@ __device__ __forceinline__ void norm_rotate(const T* x, const GroupedArgs<T>& a,
     for (int i = a.rot_dims + lane; i < a.dim; i += 32) put(i, at(i));
 }
 
+// The same with eight neighbouring entries per lane, `lanes` lanes per vector (a power of two, lane
+// l of them): put(first entry, values).  Needs rot_dims in steps of 16 and dim <= 8 * lanes.
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) { Vec16<bf16>::unpack(*reinterpret_cast<const uint4*>(p), v); }
+__device__ __forceinline__ void load8(const float* p, float (&v)[8])
+{
+    Vec16<float>::unpack(*reinterpret_cast<const uint4*>(p), v);
+    Vec16<float>::unpack(*reinterpret_cast<const uint4*>(p + 4), v + 4);
+}
+__device__ __forceinline__ void store8(bf16* p, const float (&v)[8])
+{
+    __nv_bfloat162 t[4];
+#pragma unroll
+    for (int i = 0; i < 4; i++) t[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(t);
+}
+__device__ __forceinline__ void store8(float* p, const float (&v)[8])
+{
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <typename T> __host__ __device__ __forceinline__ bool rotates8(const GroupedArgs<T>& a) { return a.rot_dims % 16 == 0 && a.dim <= 256; }
+
+template <typename T, typename F>
+__device__ __forceinline__ void norm_rotate8(const T* x, const GroupedArgs<T>& a, const float* w, int pos, int lanes, int l, F&& put)
+{
+    const int half = a.rot_dims >> 1, half8 = half >> 3;
+    const bool in = l * 8 < a.dim, turns = l < 2 * half8;
+    float v[8], g[8], c[16];
+#pragma unroll
+    for (int j = 0; j < 8; j++) v[j] = g[j] = 0.f;
+    if (in) load8(x + l * 8, v);
+    if (in && w) load8(w + l * 8, g);
+    if (turns) {
+        const float* cs = reinterpret_cast<const float*>(a.rope + (size_t)pos * half + (l < half8 ? l : l - half8) * 8);
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const float4 t = *reinterpret_cast<const float4*>(cs + 4 * j);
+            c[4 * j] = t.x;
+            c[4 * j + 1] = t.y;
+            c[4 * j + 2] = t.z;
+            c[4 * j + 3] = t.w;
+        }
+    }
+    if (w) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; j++) ss += v[j] * v[j];
+        for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float f = 1.0f / sqrtf(ss / (float)a.dim_true + a.eps);
+#pragma unroll
+        for (int j = 0; j < 8; j++) v[j] = v[j] * (f * g[j]);
+    }
+    const int partner = (int)(threadIdx.x & 31) + (!turns ? 0 : l < half8 ? half8 : -half8);
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+        const float o = __shfl_sync(0xffffffffu, v[j], partner);
+        if (turns) v[j] = l < half8 ? v[j] * c[2 * j] - o * c[2 * j + 1] : v[j] * c[2 * j] + o * c[2 * j + 1];
+    }
+    if (in) put(l * 8, v);
+}
+
 // ---------------------------------------------------------------------------
 // Norms, rotations, cache append
 // ---------------------------------------------------------------------------
@@ -68,6 +129,16 @@ grouped_prep_kernel(const GroupedArgs<T> a)
     T* proj = a.proj + (size_t)row * a.ld;
     T* kc = a.kc + (size_t)(a.g.first_slot + b) * a.k_slot + (size_t)r * a.kv_heads * a.dim;
     T* vc = a.vc + (size_t)(a.g.first_slot + b) * a.v_slot + (size_t)r * a.kv_heads * a.vdim;
+    if (rotates8(a)) {
+        const int lanes = a.dim <= 64 ? 8 : a.dim <= 128 ? 16 : 32, l = threadIdx.x & (lanes - 1), per = kPrepThreads / lanes;
+        for (int h0 = 0; h0 < a.heads + a.kv_heads; h0 += per) {          // all lanes take part in every round
+            const int hh = h0 + threadIdx.x / lanes, h = min(hh, a.heads + a.kv_heads - 1);
+            const bool q = h < a.heads;
+            const T* src = q ? proj + a.q_off + (size_t)h * a.dim : proj + a.k_off + (size_t)(h - a.heads) * a.dim;
+            T* dst = q ? const_cast<T*>(src) : kc + (size_t)(h - a.heads) * a.dim;
+            norm_rotate8<T>(src, a, q ? a.q_norm : a.k_norm, pos, lanes, l, [&](int i, const float (&v)[8]) { if (hh == h) store8(dst + i, v); });
+        }
+    } else
     for (int h = warp; h < a.heads + a.kv_heads; h += kPrepWarps) {
         const bool q = h < a.heads;
         const T* src = q ? proj + a.q_off + (size_t)h * a.dim : proj + a.k_off + (size_t)(h - a.heads) * a.dim;
@@ -83,8 +154,8 @@ grouped_prep_kernel(const GroupedArgs<T> a)
 // ---------------------------------------------------------------------------
 // One query row against a range of positions
 // ---------------------------------------------------------------------------
-constexpr int kSpanThreads = 128, kSpanWarps = kSpanThreads / 32, kSpanHeads = 8;
-constexpr int kSpanAcc = 8;                          // pairs of output entries per thread
+constexpr int kSpanThreads = 256, kSpanWarps = kSpanThreads / 32, kSpanHeads = 8;
+constexpr int kSpanAcc = 4;                          // pairs of output entries per thread
 constexpr int kSpanMaxSplit = 32, kSpanTargetCtas = 2 * 148;
 
 __device__ __forceinline__ int range_len(int span, int nsplit, int tile) { return ((span + tile - 1) / tile + nsplit - 1) / nsplit * tile; }
@@ -133,19 +204,49 @@ grouped_span_kernel(const GroupedArgs<T> a, float* __restrict__ ws, int hb, int 
         for (int i = tid; i < TK * nk; i += kSpanThreads) {
             const int r = i / nk, c = i - r * nk, p = k0 + r;
             const bool v = p < p1 && p < stored;
+            if (ONE && p == pos) continue;                            // written below
             copy16(kt + r * ldk + c * V, v ? kc + (size_t)(p % a.cache_rows) * krow + c * V : kc, v);
         }
         for (int i = tid; i < TK * nv; i += kSpanThreads) {
             const int r = i / nv, c = i - r * nv, p = k0 + r;
             const bool v = p < p1 && p < stored;
+            if (ONE && p == pos) continue;
             copy16(vt + r * E + c * V, v ? vc + (size_t)(p % a.cache_rows) * vrow + c * V : vc, v);
         }
         cp_commit();
+        if (ONE && pos >= k0 && pos < k0 + TK && pos < p1) {          // the new token's key and value, here and into the cache
+            const int r = pos - k0, ring = pos % a.cache_rows;
+            T *krow_s = kt + r * ldk, *krow_g = kc + (size_t)ring * krow;
+            if (warp == kSpanWarps - 1) {
+                const T* src = proj + a.k_off + (size_t)g * D;
+                if (rotates8(a))
+                    norm_rotate8<T>(src, a, a.k_norm, pos, 32, lane, [&](int i, const float (&v)[8]) {
+                        store8(krow_s + i, v);
+                        if (h0 == 0) store8(krow_g + i, v);
+                    });
+                else
+                    norm_rotate<T>(src, a, a.k_norm, pos, [&](int i, float v) {
+                        krow_s[i] = from_f<T>(v);
+                        if (h0 == 0) krow_g[i] = from_f<T>(v);
+                    });
+            } else {
+                for (int i = tid; i < E; i += kSpanThreads - 32) {
+                    const T v = proj[a.v_off + (size_t)g * E + i];
+                    vt[r * E + i] = v;
+                    if (h0 == 0) vc[(size_t)ring * vrow + i] = v;
+                }
+            }
+        }
     };
     load(p0);
     for (int h = warp; h < nh; h += kSpanWarps) {
         const T* q = proj + a.q_off + (size_t)(g * per + h0 + h) * D;
-        if (ONE) norm_rotate<T>(q, a, a.q_norm, pos, [&](int i, float v) { qs[h * D + i] = to_f<T>(from_f<T>(v)) * a.scale; });
+        if (ONE && rotates8(a))
+            norm_rotate8<T>(q, a, a.q_norm, pos, 32, lane, [&](int i, const float (&v)[8]) {
+#pragma unroll
+                for (int j = 0; j < 8; j++) qs[h * D + i + j] = to_f<T>(from_f<T>(v[j])) * a.scale;
+            });
+        else if (ONE) norm_rotate<T>(q, a, a.q_norm, pos, [&](int i, float v) { qs[h * D + i] = to_f<T>(from_f<T>(v)) * a.scale; });
         else
             for (int i = lane; i < D; i += 32) qs[h * D + i] = to_f<T>(q[i]) * a.scale;
     }
@@ -160,21 +261,6 @@ grouped_span_kernel(const GroupedArgs<T> a, float* __restrict__ ws, int hb, int 
     for (int k0 = p0; k0 < p1; k0 += TK) {
         cp_wait<0>();
         __syncthreads();
-        if (ONE && pos >= k0 && pos < k0 + TK) {                      // the new token's key and value
-            const int r = pos - k0, ring = pos % a.cache_rows;
-            if (warp == 0)
-                norm_rotate<T>(proj + a.k_off + (size_t)g * D, a, a.k_norm, pos, [&](int i, float v) {
-                    kt[r * ldk + i] = from_f<T>(v);
-                    if (h0 == 0) kc[(size_t)ring * krow + i] = from_f<T>(v);
-                });
-            else
-                for (int i = tid - 32; i < E; i += kSpanThreads - 32) {
-                    const T v = proj[a.v_off + (size_t)g * E + i];
-                    vt[r * E + i] = v;
-                    if (h0 == 0) vc[(size_t)ring * vrow + i] = v;
-                }
-            __syncthreads();
-        }
         {
             const int r = tid & (TK - 1), set = tid / TK;             // one position, every SETS-th head
             float s[MAXH];

@@ -17,6 +17,7 @@
 #include "launch.cuh"
 #include "mixers.cuh"
 #include "mma_sync.cuh"
+#include "tcgen05.cuh"
 
 namespace tllm {
 
@@ -144,17 +145,30 @@ matrix_seq_kernel(const MatrixScanArgs<T> a, int lpc)
 // ---------------------------------------------------------------------------
 // Chunks
 // ---------------------------------------------------------------------------
-constexpr int kC = 64, kChunkThreads = 128;
+constexpr int kC = 64, kChunkThreads = 128, kScanThreads = 256;
 constexpr int kLdC = kC + 8;                       // row stride of a [64][64] tile in shared memory
+constexpr int kLdA = kC + 4;                       // of an FP32 one
 
-// per (sequence, chunk, head): matrices [64][64], BF16 high and low parts -- P, then with the delta
+// floats of the region that holds the queries, then the inverse
+__host__ __device__ inline int inverse_floats(int ld) { return kC * (ld / 2 > kLdA ? ld / 2 : kLdA); }
+
+// What the first launch leaves for the second, laid out as it lies in shared memory there, so that a
+// tile is one bulk copy.  Per (sequence, chunk, key head): keys, then queries, [64][ld], zero behind
+// the sequence; per (sequence, chunk, head): slices of `nv` value columns [64][nv + 8]; matrices [64][kLdC] as they lie in shared memory, BF16 high and low parts -- P, then with the delta
 // rule the inverse -- and four vectors of 64 floats (log of the running decay, step size, 1/|k|,
 // q_scale/|q|)
 struct ChunkWs {
-    bf16* mats;
-    float* vecs;
-    int n_mats;
+    bf16 *kq, *v, *mats;
+    float *vecs, *rec;
+    int n_mats, nv;
+    int* err;
 };
+__device__ __forceinline__ void bulk_copy(void* dst, const void* src, uint32_t bytes, uint32_t bar)
+{
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                 ::"r"(sm32(dst)), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
+__device__ __forceinline__ void carriers_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 __host__ __device__ inline size_t chunk_mats(bool delta) { return delta ? 4 : 2; }
 inline int chunks_of(int n) { return (n + kC - 1) / kC; }
 
@@ -164,9 +178,13 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
 {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     const int D = a.dim, ld = ((D + 15) & ~15) + 8, ksteps = (D + 15) / 16;
-    bf16* ks = reinterpret_cast<bf16*>(smem_raw);          // [64][ld]
+    // keys [64][ld], queries [64][ld]; delta: A [64][kLdA], a block column of sums, and the inverse
+    // [64][kLdA] over the queries
+    bf16* ks = reinterpret_cast<bf16*>(smem_raw);
     bf16* qs = ks + kC * ld;
-    float* A = reinterpret_cast<float*>(qs + kC * ld);     // [64][64] (delta)
+    float* inv = reinterpret_cast<float*>(qs);
+    float* A = inv + inverse_floats(ld);
+    float* tmp = A + kC * kLdA;
     __shared__ float logg[kC], beta[kC], rk[kC], rq[kC];
     pdl_launch_dependents();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -174,7 +192,7 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
     const int n = min(kC, a.g.seq_len - chunk * kC);
     const size_t row0 = (size_t)b * a.g.seq_len + (size_t)chunk * kC;
     const size_t unit = ((size_t)b * gridDim.x + chunk) * a.heads + h;
-    bf16* mats = ws.mats + unit * ws.n_mats * kC * kC;
+    bf16* mats = ws.mats + unit * ws.n_mats * kC * kLdC;
     pdl_wait();
     {
         const int pieces = D / 8, per = ld / 8;
@@ -204,8 +222,22 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
         logg[2 * lane] = s - lg[1];
         logg[2 * lane + 1] = s;
     }
+    {
+        const int slices = (a.vdim + ws.nv - 1) / ws.nv, per = ws.nv / 8, ldv = ws.nv + 8;
+        bf16* v = ws.v + unit * slices * kC * ldv;
+        for (int i = tid; i < kC * slices * per; i += kChunkThreads) {
+            const int r = i / (slices * per), c = i - r * slices * per, s = c / per;
+            const uint4 x = (r < n && c * 8 < a.vdim) ? *(reinterpret_cast<const uint4*>(a.v + (row0 + r) * a.ld + (size_t)h * a.vdim) + c)
+                                                      : make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint4*>(v + (s * kC + r) * ldv + (c - s * per) * 8) = x;
+        }
+    }
     cp_wait<0>();
     __syncthreads();
+    if (h % (a.heads / a.kv_heads) == 0) {
+        uint4* kq = reinterpret_cast<uint4*>(ws.kq + (((size_t)b * gridDim.x + chunk) * a.kv_heads + kh) * 2 * kC * ld);
+        for (int i = tid; i < 2 * kC * ld / 8; i += kChunkThreads) kq[i] = reinterpret_cast<const uint4*>(ks)[i];
+    }
     if (DELTA) {
         // a quarter of a warp per vector
         for (int i = tid >> 3; i < 2 * kC; i += kChunkThreads / 8) {
@@ -272,14 +304,12 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
                 for (int e = 0; e < 2; e++) p[e] = c + e <= i ? s[j][2 * half + e] * weight(i, c + e) * rq[i] * rk[c + e] : 0.f;
                 uint32_t hi, lo;
                 split2(p[0], p[1], hi, lo);
-                *reinterpret_cast<uint32_t*>(mats + i * kC + c) = hi;
-                *reinterpret_cast<uint32_t*>(mats + kC * kC + i * kC + c) = lo;
+                *reinterpret_cast<uint32_t*>(mats + i * kLdC + c) = hi;
+                *reinterpret_cast<uint32_t*>(mats + kC * kLdC + i * kLdC + c) = lo;
             }
     };
-    if (!DELTA) {
-        write_p(warp * 16);
-        return;
-    }
+    write_p(warp * 16);
+    if (!DELTA) return;
     {
         float s[8][4];
         gram(ks, warp * 16, s);
@@ -288,39 +318,90 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const int i = warp * 16 + (lane >> 2) + (e >> 1) * 8, c = j * 8 + 2 * (lane & 3) + (e & 1);
-                A[i * kC + c] = c < i ? beta[i] * weight(i, c) * rk[i] * rk[c] * s[j][e] : 0.f;
+                A[i * kLdA + c] = c < i ? beta[i] * weight(i, c) * rk[i] * rk[c] * s[j][e] : 0.f;
             }
     }
-    __syncthreads();
-    if (warp >= 2) {
-        write_p((warp - 2) * 16);
-        write_p((5 - warp) * 16);                           // warps 2, 3: rows 0, 48 and 16, 32
-        return;
-    }
-    // forward substitution, a column of the inverse per thread
-    float x[kC];
+    __syncthreads();                                        // A is there, and nobody reads the queries any more
+    // (1 + A)^-1 by blocks of 16: the diagonal ones by substitution, a column per thread
+    constexpr int kB = 16, nb = kC / kB;
+    if (tid < kC) {
+        const int d0 = tid & ~(kB - 1), col = tid & (kB - 1);
+        float x[kB];
 #pragma unroll
-    for (int i = 0; i < kC; i++) {
-        float s0 = i == tid ? 1.f : 0.f, s1 = 0.f;
+        for (int i = 0; i < kB; i++) {
+            float v = i == col ? 1.f : 0.f;
 #pragma unroll
-        for (int j = 0; j < i; j += 4) {
-            const float4 r = *reinterpret_cast<const float4*>(A + i * kC + j);   // zeros from the diagonal on
-            s0 = fmaf(-r.x, x[j], s0);
-            if (j + 1 < i) s1 = fmaf(-r.y, x[j + 1], s1);
-            if (j + 2 < i) s0 = fmaf(-r.z, x[j + 2], s0);
-            if (j + 3 < i) s1 = fmaf(-r.w, x[j + 3], s1);
+            for (int j = 0; j < i; j++) v = fmaf(-A[(d0 + i) * kLdA + d0 + j], x[j], v);
+            x[i] = v;
+            inv[(d0 + i) * kLdA + d0 + col] = v;
         }
-        x[i] = s0 + s1;
-        const bf16 hi = __float2bfloat16_rn(x[i]);
-        mats[2 * kC * kC + i * kC + tid] = hi;
-        mats[3 * kC * kC + i * kC + tid] = __float2bfloat16_rn(x[i] - __bfloat162float(hi));
+    } else {                                                // blocks above the diagonal are zero
+        for (int i = tid - kC; i < kC * kC; i += kChunkThreads - kC) {
+            const int r = i / kC, c = i % kC;
+            if (r / kB < c / kB) inv[r * kLdA + c] = 0.f;
+        }
+    }
+    __syncthreads();
+    // then block (j + d, j) = -inv_ii sum_k A_ik inv_kj, one distance after the other: 16 threads per
+    // block, 4 x 4 entries each
+    const int j = tid >> 4, tr = (tid >> 2 & 3) * 4, tc = (tid & 3) * 4;
+    auto tile_product = [&](const float* x, int ldx, const float* y, int ldy, int n, float (&v)[4][4]) {
+#pragma unroll
+        for (int r = 0; r < 4; r++)
+#pragma unroll
+            for (int c = 0; c < 4; c++) v[r][c] = 0.f;
+#pragma unroll 4
+        for (int k = 0; k < n; k++) {
+            const float4 q = *reinterpret_cast<const float4*>(y + k * ldy + tc);
+#pragma unroll
+            for (int r = 0; r < 4; r++) {
+                const float p = x[(tr + r) * ldx + k];
+                v[r][0] = fmaf(p, q.x, v[r][0]);
+                v[r][1] = fmaf(p, q.y, v[r][1]);
+                v[r][2] = fmaf(p, q.z, v[r][2]);
+                v[r][3] = fmaf(p, q.w, v[r][3]);
+            }
+        }
+    };
+    for (int d = 1; d < nb; d++) {
+        float v[4][4];
+        const int i0 = (j + d) * kB;
+        if (j + d < nb) {
+            tile_product(A + i0 * kLdA + j * kB, kLdA, inv + j * kB * kLdA + j * kB, kLdA, d * kB, v);
+#pragma unroll
+            for (int r = 0; r < 4; r++) *reinterpret_cast<float4*>(tmp + j * kB * kB + (tr + r) * kB + tc) = make_float4(v[r][0], v[r][1], v[r][2], v[r][3]);
+        }
+        __syncthreads();
+        if (j + d < nb) {
+            tile_product(inv + i0 * kLdA + i0, kLdA, tmp + j * kB * kB, kB, kB, v);
+#pragma unroll
+            for (int r = 0; r < 4; r++)
+                *reinterpret_cast<float4*>(inv + (i0 + tr + r) * kLdA + j * kB + tc) = make_float4(-v[r][0], -v[r][1], -v[r][2], -v[r][3]);
+        }
+        __syncthreads();
+    }
+    for (int i = tid; i < kC * kC / 4; i += kChunkThreads) {
+        const float4 v = *reinterpret_cast<const float4*>(inv + (i >> 4) * kLdA + (i & 15) * 4);
+        uint32_t h0, l0, h1, l1;
+        split2(v.x, v.y, h0, l0);
+        split2(v.z, v.w, h1, l1);
+        bf16* m = mats + 2 * kC * kLdC + (i >> 4) * kLdC + (i & 15) * 4;
+        *reinterpret_cast<uint2*>(m) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2*>(m + kC * kLdC) = make_uint2(l0, l1);
     }
 }
 
-// NV columns of the state per CTA, MT tiles of 16 state rows per warp; `stages` chunks in flight
-template <bool DELTA, int NV, int MT>
-__global__ void __launch_bounds__(kChunkThreads)
-chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int stages)
+// A segment of the chunks and NV columns of the state per CTA.  Four warps carry the state (U, then
+// the state behind the chunk; MT tiles of 16 rows each), four others compute the outputs beside
+// them.  `stages` chunks are in flight.
+//
+// Linear attention is cut into segments that run at the same time: RECORD runs all but the last
+// from a zero state and keeps their final states, the second launch starts each segment from the
+// carried state and the records before it.  (The record of the last segment holds a copy of the
+// carried state, which that segment overwrites while others may not have started.)
+template <bool DELTA, int NV, int MT, bool RECORD>
+__global__ void __launch_bounds__(kScanThreads)
+chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_seg, int nseg, int stages)
 {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     constexpr int ldv = NV + 8, NT = NV / 8, MATS = DELTA ? 4 : 2;
@@ -331,42 +412,43 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int stag
     bf16* rs = sh + 2 * D16 * ldv;                                             // right-hand side [64][ldv], high and low
     bf16* us = rs + (DELTA ? 2 * kC * ldv : 0);                                // U
     bf16* ups = us + (DELTA ? 2 * kC * ldv : 0);                               // U times its decay to the end
+    __shared__ __align__(8) uint64_t full[2];
+    __shared__ int abort_flag;
     pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
-    const int v0 = blockIdx.x * NV, h = blockIdx.y, b = blockIdx.z, kh = h / (a.heads / a.kv_heads);
-    const int nv = min(NV, a.vdim - v0);
+    const int tid = threadIdx.x, warp = (tid >> 5) & 3, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
+    const bool carrier = tid < 128;                                            // carries the state
+    const int slices = (a.vdim + NV - 1) / NV, seg = blockIdx.x / slices;
+    const int v0 = (blockIdx.x - seg * slices) * NV, h = blockIdx.y, b = blockIdx.z, kh = h / (a.heads / a.kv_heads);
+    const int nv = min(NV, a.vdim - v0), c0 = seg * per_seg, c1 = min(nchunk, c0 + per_seg);
     const size_t row0 = (size_t)b * a.g.seq_len;
+    int never = 0;
+    if (tid == 0) {
+        gemm::mbar_init(gemm::smem_u32(&full[0]), 1);
+        gemm::mbar_init(gemm::smem_u32(&full[1]), 1);
+        abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
     pdl_wait();
     const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
     float* st = a.state + (size_t)(a.g.first_slot + b) * a.slot_stride + ((size_t)h * a.vdim + v0) * D;
+    const size_t rec_size = (size_t)a.heads * a.vdim * D;                      // of one segment
+    float* rec = ws.rec + (size_t)b * nseg * rec_size + ((size_t)h * a.vdim + v0) * D;
 
+    // the tiles of a chunk, by bulk copies that report to the stage's barrier
     auto request = [&](int c, int stage) {
         bf16* p = reinterpret_cast<bf16*>(smem_raw + stage * stage_bytes);
-        const int n = min(kC, a.g.seq_len - c * kC), per = ld / 8, pieces = D / 8;
-        const size_t r0 = row0 + (size_t)c * kC, unit = ((size_t)b * nchunk + c) * a.heads + h;
-        for (int i = tid; i < kC * per; i += kChunkThreads) {
-            const int r = i / per, cc = i - r * per;
-            const bool v = r < n && cc < pieces;
-            const size_t o = (r0 + (v ? r : 0)) * a.ld + (size_t)kh * D + (v ? cc * 8 : 0);
-            cp16(p + r * ld + cc * 8, a.k + o, v);
-            cp16(p + kC * ld + r * ld + cc * 8, a.q + o, v);
-        }
-        p += 2 * kC * ld;
-        const bf16* m = ws.mats + unit * MATS * kC * kC;
-        for (int i = tid; i < MATS * kC * (kC / 8); i += kChunkThreads)
-            cp16(p + (i >> 3) * kLdC + (i & 7) * 8, m + (size_t)i * 8, true);
-        p += MATS * kC * kLdC;
-        for (int i = tid; i < kC * (NV / 8); i += kChunkThreads) {
-            const int r = i / (NV / 8), cc = (i - r * (NV / 8)) * 8;
-            const bool v = r < n && cc < nv;
-            cp16(p + r * ldv + cc, a.v + (r0 + (v ? r : 0)) * a.ld + (size_t)h * a.vdim + v0 + (v ? cc : 0), v);
-        }
-        p += kC * ldv;
-        const float* vec = ws.vecs + unit * 4 * kC;
-        for (int i = tid; i < kC; i += kChunkThreads) cp16(p + 8 * i, reinterpret_cast<const bf16*>(vec + 4 * i), true);
-        cp_commit();
+        const uint32_t bar = gemm::smem_u32(&full[stage]);
+        const size_t unit = ((size_t)b * nchunk + c) * a.heads + h, kunit = ((size_t)b * nchunk + c) * a.kv_heads + kh;
+        const uint32_t kq = (RECORD ? 1 : 2) * kC * ld * 2, m = RECORD ? 0 : MATS * kC * kLdC * 2, v = kC * ldv * 2, vec = 4 * kC * 4;
+        gemm::mbar_expect_tx(bar, kq + m + v + vec);
+        bulk_copy(p, ws.kq + kunit * 2 * kC * ld, kq, bar);
+        if (!RECORD) bulk_copy(p + 2 * kC * ld, ws.mats + unit * MATS * kC * kLdC, m, bar);
+        bulk_copy(p + 2 * kC * ld + MATS * kC * kLdC, ws.v + (unit * slices + v0 / NV) * kC * ldv, v, bar);
+        bulk_copy(p + tile, ws.vecs + unit * 4 * kC, vec, bar);
     };
-    request(0, 0);
+    const bool requester = tid == 128;
+    if (requester) request(c0, 0);
 
     float S[MT][NT][4];
     auto each_state = [&](auto&& f) {                       // (tile, column tile, element, row, column)
@@ -375,19 +457,13 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int stag
 #pragma unroll
             for (int j = 0; j < NT; j++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) f(i, j, e, (warp + 4 * i) * 16 + gq + (e >> 1) * 8, j * 8 + 2 * tq + (e & 1));
+                for (int e = 0; e < 4; e++) {
+                    const int r = (warp + 4 * i) * 16 + gq + (e >> 1) * 8, c = j * 8 + 2 * tq + (e & 1);
+                    const bool in = r < D && c < nv;
+                    f(S[i][j][e], in, in ? (size_t)c * D + r : 0);   // a place that may be read either way
+                }
     };
-    each_state([&](int i, int j, int e, int r, int c) { S[i][j][e] = (!fresh && r < D && c < nv) ? st[(size_t)c * D + r] : 0.f; });
-    const int lda = lane & 15, ldb = (lane >> 4) * 8;
-    const int i0 = warp * 16 + gq;                          // this lane's rows i0 and i0 + 8 of a chunk
-
-    for (int c = 0; c < nchunk; c++) {
-        const int stage = stages == 2 ? c & 1 : 0, n = min(kC, a.g.seq_len - c * kC);
-        const bf16* kt = reinterpret_cast<const bf16*>(smem_raw + stage * stage_bytes);
-        const bf16 *qt = kt + kC * ld, *pm = qt + kC * ld, *tm = pm + 2 * kC * kLdC, *vt = pm + MATS * kC * kLdC;
-        const float* logg = reinterpret_cast<const float*>(vt + kC * ldv);
-        const float *beta = logg + kC, *rk = beta + kC, *rq = rk + kC;
-        // the state as two BF16 matrices
+    auto save_state = [&]() {                               // as two BF16 matrices
 #pragma unroll
         for (int i = 0; i < MT; i++) {
             const int r = (warp + 4 * i) * 16 + gq;
@@ -403,176 +479,206 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int stag
                     *reinterpret_cast<uint32_t*>(sh + D16 * ldv + o) = lo;
                 }
         }
-        cp_wait<0>();
-        __syncthreads();
-        if (stages == 2 && c + 1 < nchunk) request(c + 1, stage ^ 1);
-        // K S0 and Q S0, 16 rows per warp
-        float ksum[NT][4], qsum[NT][4];
+    };
+    if (carrier) {
+        // loads without branches: all of them are in flight together
+        const float keep = fresh ? 0.f : 1.f;
+        if (RECORD || nseg == 1) each_state([&](float& x, bool in, size_t o) { const float v = st[o]; x = in && keep != 0.f ? v : 0.f; });
+        if (RECORD) {
+            if (seg == 0) each_state([&](float& x, bool in, size_t o) { if (in) rec[(size_t)(nseg - 1) * rec_size + o] = x; });
+            each_state([&](float& x, bool, size_t) { x = 0.f; });
+        } else if (nseg > 1) {
+            each_state([&](float& x, bool in, size_t o) { const float v = rec[(size_t)(nseg - 1) * rec_size + o]; x = in ? v : 0.f; });
+            const float d = DELTA ? 0.f : a.decay[h], f = expf((float)(per_seg * kC) * (d > 0.f ? logf(d) : -100.f));
+#pragma unroll 2
+            for (int k = 0; k < seg; k++)
+                each_state([&](float& x, bool in, size_t o) { const float v = rec[(size_t)k * rec_size + o]; x = in ? fmaf(f, x, v) : 0.f; });
+        }
+        if (!RECORD) save_state();
+    }
+    const int lda = lane & 15, ldb = (lane >> 4) * 8;
+    const int i0 = warp * 16 + gq;                          // this lane's rows i0 and i0 + 8 of a chunk
+    auto zero = [](float (&x)[NT][4]) {
 #pragma unroll
         for (int j = 0; j < NT; j++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) ksum[j][e] = qsum[j][e] = 0.f;
-#pragma unroll 2
-        for (int k = 0; k < ksteps; k++) {
-            uint32_t fk[4], fq[4];
-            if (DELTA) ldsm4(fk, kt + (warp * 16 + lda) * ld + k * 16 + ldb);
-            ldsm4(fq, qt + (warp * 16 + lda) * ld + k * 16 + ldb);
+            for (int e = 0; e < 4; e++) x[j][e] = 0.f;
+    };
+    auto join = [](float (&x)[NT][4], const float (&y)[NT][4]) {
 #pragma unroll
-            for (int part = 0; part < 2; part++)
+        for (int j = 0; j < NT; j++)
 #pragma unroll
-                for (int j = 0; j < NT; j += 2) {
-                    uint32_t fb[4];
-                    ldsm4t(fb, sh + part * D16 * ldv + (k * 16 + lda) * ldv + j * 8 + ldb);
-                    if (DELTA) {
-                        mma16816(ksum[j], fk, fb[0], fb[1]);
-                        mma16816(ksum[j + 1], fk, fb[2], fb[3]);
-                    }
-                    mma16816(qsum[j], fq, fb[0], fb[1]);
-                    mma16816(qsum[j + 1], fq, fb[2], fb[3]);
-                }
+            for (int e = 0; e < 4; e++) x[j][e] += y[j][e];
+    };
+    // x += (16 rows of the matrix m, its columns 16 k ..) times rows 16 k .. of u
+    auto times = [&](float (&x)[NT][4], const uint32_t (&f)[4], const bf16* u, int k) {
+#pragma unroll
+        for (int j = 0; j < NT; j += 2) {
+            uint32_t fb[4];
+            ldsm4t(fb, u + (k * 16 + lda) * ldv + j * 8 + ldb);
+            mma16816(x[j], f, fb[0], fb[1]);
+            mma16816(x[j + 1], f, fb[2], fb[3]);
+        }
+    };
+
+    bool ok = true;
+    for (int c = c0; c < c1; c++) {
+        const int stage = stages == 2 ? (c - c0) & 1 : 0, n = min(kC, a.g.seq_len - c * kC);
+        const bf16* kt = reinterpret_cast<const bf16*>(smem_raw + stage * stage_bytes);
+        const bf16 *qt = kt + kC * ld, *pm = qt + kC * ld, *tm = pm + 2 * kC * kLdC, *vt = pm + MATS * kC * kLdC;
+        const float* logg = reinterpret_cast<const float*>(vt + kC * ldv);
+        const float *beta = logg + kC, *rk = beta + kC, *rq = rk + kC;
+        __syncthreads();                                    // the state is there, nobody reads the other stage any more
+        if (requester && stages == 2 && c + 1 < c1) request(c + 1, stage ^ 1);
+        const int turn = stages == 2 ? (c - c0) >> 1 : c - c0;
+        if (ok && !gemm::mbar_wait(gemm::smem_u32(&full[stage]), turn & 1, &abort_flag)) {
+            ok = false;                                     // the sums are wrong from here on, the loop ends all the same
+            abort_flag = 1;
         }
         const float end = logg[n - 1];
-        float dec[2], to_end[2];
+        float acc[NT][4], low[NT][4], dec[2];               // two chains of sums: high parts, the rest
+        zero(acc);
+        zero(low);
 #pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int i = i0 + half * 8;
-            dec[half] = exp2_neg(1.4426950408889634f * logg[i]);
-            to_end[half] = i < n ? exp2_neg(1.4426950408889634f * (end - logg[i])) * rk[i] : 0.f;
-        }
-        if (DELTA) {
+        for (int half = 0; half < 2; half++) dec[half] = exp2_neg(1.4426950408889634f * logg[i0 + half * 8]);
+        if (carrier) {
+            float to_end[2];
 #pragma unroll
-            for (int j = 0; j < NT; j++)
-#pragma unroll
-                for (int half = 0; half < 2; half++) {
-                    const int i = i0 + half * 8, o = i * ldv + j * 8 + 2 * tq;
-                    const float f = dec[half] * rk[i], be = beta[i];
-                    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vt + o));
-                    uint32_t hi, lo;
-                    split2(be * (v.x - f * ksum[j][2 * half]), be * (v.y - f * ksum[j][2 * half + 1]), hi, lo);
-                    *reinterpret_cast<uint32_t*>(rs + o) = hi;
-                    *reinterpret_cast<uint32_t*>(rs + kC * ldv + o) = lo;
-                }
-            __syncthreads();
-            float u[NT][4];
-#pragma unroll
-            for (int j = 0; j < NT; j++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) u[j][e] = 0.f;
-            for (int k = 0; k <= warp; k++) {              // triangular
-                uint32_t fh[4], fl[4];
-                ldsm4(fh, tm + (warp * 16 + lda) * kLdC + k * 16 + ldb);
-                ldsm4(fl, tm + kC * kLdC + (warp * 16 + lda) * kLdC + k * 16 + ldb);
-#pragma unroll
-                for (int j = 0; j < NT; j += 2) {
-                    uint32_t fb[4], fc[4];
-                    ldsm4t(fb, rs + (k * 16 + lda) * ldv + j * 8 + ldb);
-                    ldsm4t(fc, rs + kC * ldv + (k * 16 + lda) * ldv + j * 8 + ldb);
-                    mma16816(u[j], fh, fb[0], fb[1]);
-                    mma16816(u[j + 1], fh, fb[2], fb[3]);
-                    mma16816(u[j], fl, fb[0], fb[1]);
-                    mma16816(u[j + 1], fl, fb[2], fb[3]);
-                    mma16816(u[j], fh, fc[0], fc[1]);
-                    mma16816(u[j + 1], fh, fc[2], fc[3]);
-                }
+            for (int half = 0; half < 2; half++) {
+                const int i = i0 + half * 8;
+                to_end[half] = i < n ? exp2_neg(1.4426950408889634f * (end - logg[i])) * rk[i] : 0.f;
             }
-#pragma unroll
-            for (int j = 0; j < NT; j++)
-#pragma unroll
-                for (int half = 0; half < 2; half++) {
-                    const int o = (i0 + half * 8) * ldv + j * 8 + 2 * tq;
-                    uint32_t hi, lo;
-                    split2(u[j][2 * half], u[j][2 * half + 1], hi, lo);
-                    *reinterpret_cast<uint32_t*>(us + o) = hi;
-                    *reinterpret_cast<uint32_t*>(us + kC * ldv + o) = lo;
-                    split2(u[j][2 * half] * to_end[half], u[j][2 * half + 1] * to_end[half], hi, lo);
-                    *reinterpret_cast<uint32_t*>(ups + o) = hi;
-                    *reinterpret_cast<uint32_t*>(ups + kC * ldv + o) = lo;
+            if (DELTA) {
+#pragma unroll 4
+                for (int k = 0; k < ksteps; k++) {          // K S0
+                    uint32_t f[4];
+                    ldsm4(f, kt + (warp * 16 + lda) * ld + k * 16 + ldb);
+                    times(acc, f, sh, k);
+                    times(low, f, sh + D16 * ldv, k);
                 }
-        } else {
+                join(acc, low);
 #pragma unroll
-            for (int j = 0; j < NT; j++)
+                for (int j = 0; j < NT; j++)
 #pragma unroll
-                for (int half = 0; half < 2; half++) {
-                    const int o = (i0 + half * 8) * ldv + j * 8 + 2 * tq;
-                    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vt + o));
-                    uint32_t hi, lo;
-                    split2(v.x * to_end[half], v.y * to_end[half], hi, lo);
-                    *reinterpret_cast<uint32_t*>(ups + o) = hi;
-                    *reinterpret_cast<uint32_t*>(ups + kC * ldv + o) = lo;
-                }
-        }
-        __syncthreads();
-        // outputs
-#pragma unroll
-        for (int j = 0; j < NT; j++)
-#pragma unroll
-            for (int e = 0; e < 4; e++) qsum[j][e] *= dec[e >> 1] * rq[i0 + (e >> 1) * 8];
-        const bf16* ub = DELTA ? us : vt;
-        for (int k = 0; k <= warp; k++) {
-            uint32_t fh[4], fl[4];
-            ldsm4(fh, pm + (warp * 16 + lda) * kLdC + k * 16 + ldb);
-            ldsm4(fl, pm + kC * kLdC + (warp * 16 + lda) * kLdC + k * 16 + ldb);
-#pragma unroll
-            for (int j = 0; j < NT; j += 2) {
-                uint32_t fb[4];
-                ldsm4t(fb, ub + (k * 16 + lda) * ldv + j * 8 + ldb);
-                mma16816(qsum[j], fh, fb[0], fb[1]);
-                mma16816(qsum[j + 1], fh, fb[2], fb[3]);
-                mma16816(qsum[j], fl, fb[0], fb[1]);
-                mma16816(qsum[j + 1], fl, fb[2], fb[3]);
-                if (DELTA) {
-                    ldsm4t(fb, us + kC * ldv + (k * 16 + lda) * ldv + j * 8 + ldb);
-                    mma16816(qsum[j], fh, fb[0], fb[1]);
-                    mma16816(qsum[j + 1], fh, fb[2], fb[3]);
-                }
-            }
-        }
-#pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int i = i0 + half * 8;
-            if (i >= n) continue;
-            float* op = a.o + (row0 + (size_t)c * kC + i) * ((size_t)a.heads * a.vdim) + (size_t)h * a.vdim + v0;
-#pragma unroll
-            for (int j = 0; j < NT; j++) {
-                const int cc = j * 8 + 2 * tq;
-                if (cc < nv) *reinterpret_cast<float2*>(op + cc) = make_float2(qsum[j][2 * half], qsum[j][2 * half + 1]);
-            }
-        }
-        // the state behind the chunk
-        const float g_all = exp2_neg(1.4426950408889634f * end);
-        each_state([&](int i, int j, int e, int, int) { S[i][j][e] *= g_all; });
-#pragma unroll
-        for (int i = 0; i < MT; i++) {
-            const int m0 = (warp + 4 * i) * 16;
-            if (m0 >= D16) break;
-#pragma unroll
-            for (int k = 0; k < kC / 16; k++) {
-                uint32_t fa[4];
-                ldsm4t(fa, kt + (k * 16 + (lane & 7) + ldb) * ld + m0 + ((lane >> 3) & 1) * 8);
-#pragma unroll
-                for (int part = 0; part < 2; part++)
-#pragma unroll
-                    for (int j = 0; j < NT; j += 2) {
-                        uint32_t fb[4];
-                        ldsm4t(fb, ups + part * kC * ldv + (k * 16 + lda) * ldv + j * 8 + ldb);
-                        mma16816(S[i][j], fa, fb[0], fb[1]);
-                        mma16816(S[i][j + 1], fa, fb[2], fb[3]);
+                    for (int half = 0; half < 2; half++) {
+                        const int i = i0 + half * 8, o = i * ldv + j * 8 + 2 * tq;
+                        const float f = dec[half] * rk[i], be = beta[i];
+                        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vt + o));
+                        uint32_t hi, lo;
+                        split2(be * (v.x - f * acc[j][2 * half]), be * (v.y - f * acc[j][2 * half + 1]), hi, lo);
+                        *reinterpret_cast<uint32_t*>(rs + o) = hi;
+                        *reinterpret_cast<uint32_t*>(rs + kC * ldv + o) = lo;
                     }
+                carriers_sync();
+                float mid[NT][4];
+                zero(acc);
+                zero(low);
+                zero(mid);
+                for (int k = 0; k <= warp; k++) {           // U, the inverse is triangular
+                    uint32_t fh[4], fl[4];
+                    ldsm4(fh, tm + (warp * 16 + lda) * kLdC + k * 16 + ldb);
+                    ldsm4(fl, tm + kC * kLdC + (warp * 16 + lda) * kLdC + k * 16 + ldb);
+                    times(acc, fh, rs, k);
+                    times(low, fl, rs, k);
+                    times(mid, fh, rs + kC * ldv, k);
+                }
+                join(low, mid);
+                join(acc, low);
+            }
+#pragma unroll
+            for (int j = 0; j < NT; j++)
+#pragma unroll
+                for (int half = 0; half < 2; half++) {
+                    const int o = (i0 + half * 8) * ldv + j * 8 + 2 * tq;
+                    float2 u;
+                    uint32_t hi, lo;
+                    if (DELTA) {
+                        u = make_float2(acc[j][2 * half], acc[j][2 * half + 1]);
+                        split2(u.x, u.y, hi, lo);
+                        *reinterpret_cast<uint32_t*>(us + o) = hi;
+                        *reinterpret_cast<uint32_t*>(us + kC * ldv + o) = lo;
+                    } else {
+                        u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vt + o));
+                    }
+                    split2(u.x * to_end[half], u.y * to_end[half], hi, lo);
+                    *reinterpret_cast<uint32_t*>(ups + o) = hi;
+                    *reinterpret_cast<uint32_t*>(ups + kC * ldv + o) = lo;
+                }
+            if (!DELTA) carriers_sync();
+        } else if (!RECORD) {
+#pragma unroll 4
+            for (int k = 0; k < ksteps; k++) {              // Q S0
+                uint32_t f[4];
+                ldsm4(f, qt + (warp * 16 + lda) * ld + k * 16 + ldb);
+                times(acc, f, sh, k);
+                times(low, f, sh + D16 * ldv, k);
+            }
+            join(acc, low);
+            zero(low);
+        }
+        if (DELTA) __syncthreads();                         // U is there, and nobody reads the state any more
+        if (carrier) {                                      // the state behind the chunk
+            const float g_all = exp2_neg(1.4426950408889634f * end);
+            each_state([&](float& x, bool, size_t) { x *= g_all; });
+#pragma unroll
+            for (int i = 0; i < MT; i++) {
+                const int m0 = (warp + 4 * i) * 16;
+                if (m0 >= D16) break;
+                zero(low);
+#pragma unroll
+                for (int k = 0; k < kC / 16; k++) {
+                    uint32_t f[4];
+                    ldsm4t(f, kt + (k * 16 + (lane & 7) + ldb) * ld + m0 + ((lane >> 3) & 1) * 8);
+                    times(S[i], f, ups, k);
+                    times(low, f, ups + kC * ldv, k);
+                }
+                join(S[i], low);
+            }
+        } else if (!RECORD) {                               // outputs
+#pragma unroll
+            for (int j = 0; j < NT; j++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) acc[j][e] *= dec[e >> 1] * rq[i0 + (e >> 1) * 8];
+            for (int k = 0; k <= warp; k++) {
+                uint32_t fh[4], fl[4];
+                ldsm4(fh, pm + (warp * 16 + lda) * kLdC + k * 16 + ldb);
+                ldsm4(fl, pm + kC * kLdC + (warp * 16 + lda) * kLdC + k * 16 + ldb);
+                times(acc, fh, DELTA ? us : vt, k);
+                times(low, fl, DELTA ? us : vt, k);
+                if (DELTA) times(low, fh, us + kC * ldv, k);
+            }
+            join(acc, low);
+#pragma unroll
+            for (int half = 0; half < 2; half++) {
+                const int i = i0 + half * 8;
+                if (i >= n) continue;
+                float* op = a.o + (row0 + (size_t)c * kC + i) * ((size_t)a.heads * a.vdim) + (size_t)h * a.vdim + v0;
+#pragma unroll
+                for (int j = 0; j < NT; j++) {
+                    const int cc = j * 8 + 2 * tq;
+                    if (cc < nv) *reinterpret_cast<float2*>(op + cc) = make_float2(acc[j][2 * half], acc[j][2 * half + 1]);
+                }
             }
         }
-        if (stages == 1) {
-            __syncthreads();
-            if (c + 1 < nchunk) request(c + 1, 0);
-        }
+        if ((!DELTA && !RECORD) || stages == 1) __syncthreads();   // nobody reads the state or the chunk any more
+        if (carrier && !RECORD) save_state();
+        if (requester && stages == 1 && c + 1 < c1) request(c + 1, 0);
     }
-    each_state([&](int i, int j, int e, int r, int c) {
-        if (r < D && c < nv) st[(size_t)c * D + r] = S[i][j][e];
-    });
+    if (!ok) {
+        // copies may still be under way: they land before the shared memory goes away
+        for (int s = 0; s < 2; s++) gemm::mbar_wait(gemm::smem_u32(&full[s]), 0, &never) || gemm::mbar_wait(gemm::smem_u32(&full[s]), 1, &never);
+        if (lane == 0) atomicExch(ws.err, TLLM_ERR_TIMEOUT);
+    }
+    if (!carrier) return;
+    float* last = RECORD ? rec + (size_t)seg * rec_size : st;
+    if (RECORD || seg == nseg - 1) each_state([&](float& x, bool in, size_t o) { if (in) last[o] = x; });
 }
 
 size_t prepare_smem(bool delta, int dim)
 {
-    return (size_t)2 * kC * (((dim + 15) & ~15) + 8) * 2 + (delta ? (size_t)kC * kC * 4 : 0);
+    const int ld = ((dim + 15) & ~15) + 8;
+    if (!delta) return (size_t)2 * kC * ld * 2;
+    return (size_t)kC * ld * 2 + (size_t)(inverse_floats(ld) + kC * kLdA + (kC / 16 - 1) * 256) * 4;
 }
 size_t scan_smem(bool delta, int dim, int nv, int stages)
 {
@@ -582,22 +688,63 @@ size_t scan_smem(bool delta, int dim, int nv, int stages)
 }
 
 constexpr size_t kSmemLimit = 220 * 1024;
-constexpr int kChunkNv = 32, kChunkFrom = 48;         // columns per CTA; tokens from which chunks pay
-constexpr int kChunkMaxDim = 256;
+constexpr int kChunkFrom = 48;                        // tokens from which chunks pay
+constexpr int kChunkMaxDim = 256, kMaxSegments = 8, kSms = 148;
 
 static_assert(kChunkFrom > kC / 2, "workspace bound");
 
 bool chunked(int seq_len, int dim) { return seq_len >= kChunkFrom && dim <= kChunkMaxDim; }
 
-template <bool DELTA, int MT>
+template <bool DELTA, int NV, int MT>
 int chunk_scan(const MatrixScanArgs<bf16>& a, const ChunkWs& ws, int nchunk, cudaStream_t stream)
 {
-    const int stages = scan_smem(DELTA, a.dim, kChunkNv, 2) <= kSmemLimit ? 2 : 1;
-    const size_t smem = scan_smem(DELTA, a.dim, kChunkNv, stages);
-    const auto kernel = chunk_scan_kernel<DELTA, kChunkNv, MT>;
+    const int stages = scan_smem(DELTA, a.dim, NV, 2) <= kSmemLimit ? 2 : 1;
+    const size_t smem = scan_smem(DELTA, a.dim, NV, stages);
+    if (smem > kSmemLimit) return fail(TLLM_ERR_SHAPE, "matrix_scan: dim=%d", a.dim);
+    const int slices = (a.vdim + NV - 1) / NV;
+    int nseg = 1;
+    if (!DELTA) {                                          // two chunks or more to a segment
+        nseg = kSms / (slices * a.heads * a.g.n_seq);
+        nseg = nseg > nchunk / 2 ? nchunk / 2 : nseg;
+        nseg = nseg < 1 ? 1 : nseg > kMaxSegments ? kMaxSegments : nseg;
+    }
+    const int per = (nchunk + nseg - 1) / nseg;
+    nseg = (nchunk + per - 1) / per;
+    if (nseg > 1) {
+        const auto kernel = chunk_scan_kernel<DELTA, NV, MT, !DELTA>;
+        cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const int st = launch_pdl("chunk_record", kernel, dim3(slices * (nseg - 1), a.heads, a.g.n_seq), dim3(kScanThreads), smem, stream, a, ws, nchunk,
+                                  per, nseg, stages);
+        if (st) return st;
+    }
+    const auto kernel = chunk_scan_kernel<DELTA, NV, MT, false>;
     cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return launch_pdl("chunk_scan", kernel, dim3((a.vdim + kChunkNv - 1) / kChunkNv, a.heads, a.g.n_seq), dim3(kChunkThreads), smem, stream, a, ws,
-                      nchunk, stages);
+    return launch_pdl("chunk_scan", kernel, dim3(slices * nseg, a.heads, a.g.n_seq), dim3(kScanThreads), smem, stream, a, ws, nchunk, per, nseg, stages);
+}
+
+template <bool DELTA, int NV>
+int chunk_scan_dim(const MatrixScanArgs<bf16>& a, const ChunkWs& ws, int nchunk, cudaStream_t stream)
+{
+    if (a.dim <= 64) return chunk_scan<DELTA, NV, 1>(a, ws, nchunk, stream);
+    if (a.dim <= 128) return chunk_scan<DELTA, NV, 2>(a, ws, nchunk, stream);
+    return chunk_scan<DELTA, NV, 4>(a, ws, nchunk, stream);
+}
+
+// bytes of the parts of ChunkWs, in order, for `chunks` chunks of all sequences
+struct WsLayout {
+    size_t kq, v, mats, vecs, rec;
+    size_t total() const { return kq + v + mats + vecs + rec; }
+};
+WsLayout ws_layout(bool delta, size_t chunks, size_t segs, int heads, int kv_heads, int dim, int vdim, int nv)
+{
+    const size_t ld = ((dim + 15) & ~15) + 8, slices = (vdim + nv - 1) / nv, units = chunks * heads;
+    WsLayout w;
+    w.kq = chunks * kv_heads * 2 * kC * ld * sizeof(bf16);
+    w.v = units * slices * kC * (nv + 8) * sizeof(bf16);
+    w.mats = units * chunk_mats(delta) * kC * kLdC * sizeof(bf16);
+    w.vecs = units * 4 * kC * sizeof(float);
+    w.rec = delta ? 0 : segs * heads * vdim * dim * sizeof(float);
+    return w;
 }
 
 template <bool DELTA>
@@ -605,18 +752,25 @@ int chunk_path(const MatrixScanArgs<bf16>& a, cudaStream_t stream)
 {
     if (!a.ws) return fail(TLLM_ERR_NULL, "matrix_scan: no workspace");
     const int nchunk = chunks_of(a.g.seq_len);
-    const size_t units = (size_t)a.g.n_seq * nchunk * a.heads;
+    // narrow slices of the delta rule while they give more SMs one
+    const bool narrow = DELTA && a.heads * a.g.n_seq * ((a.vdim + 31) / 32) * 2 <= kSms;
+    const WsLayout l = ws_layout(DELTA, (size_t)a.g.n_seq * nchunk, 0, a.heads, a.kv_heads, a.dim, a.vdim, narrow ? 16 : 32);
+    uint8_t* p = static_cast<uint8_t*>(a.ws);
     ChunkWs ws;
     ws.n_mats = (int)chunk_mats(DELTA);
-    ws.mats = static_cast<bf16*>(a.ws);
-    ws.vecs = reinterpret_cast<float*>(ws.mats + units * ws.n_mats * kC * kC);
+    ws.nv = narrow ? 16 : 32;
+    ws.kq = reinterpret_cast<bf16*>(p);
+    ws.v = reinterpret_cast<bf16*>(p + l.kq);
+    ws.mats = reinterpret_cast<bf16*>(p + l.kq + l.v);
+    ws.vecs = reinterpret_cast<float*>(p + l.kq + l.v + l.mats);
+    ws.rec = reinterpret_cast<float*>(p + l.total());
+    ws.err = device_error_flag();
+    if (!ws.err) return fail(TLLM_ERR_LAUNCH, "device scratch unavailable");
     const size_t smem = prepare_smem(DELTA, a.dim);
     cudaFuncSetAttribute(chunk_prepare_kernel<DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     int st = launch_pdl("chunk_prepare", chunk_prepare_kernel<DELTA>, dim3(nchunk, a.heads, a.g.n_seq), dim3(kChunkThreads), smem, stream, a, ws);
     if (st) return st;
-    if (a.dim <= 64) return chunk_scan<DELTA, 1>(a, ws, nchunk, stream);
-    if (a.dim <= 128) return chunk_scan<DELTA, 2>(a, ws, nchunk, stream);
-    return chunk_scan<DELTA, 4>(a, ws, nchunk, stream);
+    return narrow ? chunk_scan_dim<DELTA, 16>(a, ws, nchunk, stream) : chunk_scan_dim<DELTA, 32>(a, ws, nchunk, stream);
 }
 int chunk_any(const MatrixScanArgs<bf16>& a, cudaStream_t stream) { return a.delta ? chunk_path<true>(a, stream) : chunk_path<false>(a, stream); }
 int chunk_any(const MatrixScanArgs<float>&, cudaStream_t) { return TLLM_ERR_SHAPE; }
@@ -693,11 +847,15 @@ gated_norm_kernel(const GatedNormArgs<T> a)
 
 }  // namespace
 
-size_t matrix_scan_workspace(bool bf16_path, bool delta, int rows, int heads, int dim)
+size_t matrix_scan_workspace(bool bf16_path, bool delta, int rows, int heads, int kv_heads, int dim, int vdim)
 {
     if (!bf16_path || !chunked(rows, dim)) return 0;
-    const size_t units = ((size_t)rows / (kC / 2) + 1) * heads;      // a sequence of 48 tokens or more: one chunk per 32 at most
-    return units * (chunk_mats(delta) * kC * kC * sizeof(bf16) + 4 * kC * sizeof(float));
+    const size_t chunks = (size_t)rows / (kC / 2) + 1;     // a sequence of 48 tokens or more: one chunk per 32 at most
+    // records: a segment has two chunks or more
+    const size_t segs = (size_t)rows / kC < kMaxSegments ? (size_t)rows / kC + 1 : kMaxSegments * ((size_t)rows / (kMaxSegments * kC) + 1);
+    const size_t narrow = ws_layout(delta, chunks, segs, heads, kv_heads, dim, vdim, 16).total();
+    const size_t wide = ws_layout(delta, chunks, segs, heads, kv_heads, dim, vdim, 32).total();
+    return narrow > wide ? narrow : wide;
 }
 
 template <typename T>

@@ -281,7 +281,7 @@ int MixedDecoder<T>::load_layer(const tllm_b200_mixed_layer& s, MixLayer<T>& L)
         TRY(vec(&L.norm2, t[TLLM_T_NORM2], 1, width, w));
         if (t[TLLM_T_NORM2B]) TRY(vec(&L.norm2b, t[TLLM_T_NORM2B], 1, width, w));
         const int n = L.experts ? L.experts : 1;             // matrices one behind the other
-        L.few = L.experts && experts_few_fits(L.top, L.ff, w, sizeof(T));
+        L.few = L.experts && gemv_routed_fits(L.top, L.ff, sizeof(T));
         TRY(mat(&L.gate_up, n * 2 * L.ff, w));
         TRY(rows_to(t[TLLM_T_GATE], n, s.ff, s.ff, 2 * L.ff, 1, width, w, L.gate_up.p, w));
         TRY(rows_to(t[TLLM_T_UP], n, s.ff, s.ff, 2 * L.ff, 1, width, w, L.gate_up.p + (size_t)L.ff * w, w));
@@ -608,7 +608,7 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
             } else {
                 const bool delta = p.type == TLLM_MIXER_DELTA_RULE;
                 up(n_heads_o, (size_t)p.heads * p.vdim);
-                up(n_scan, matrix_scan_workspace(sizeof(T) == 2, delta, rows_cap, p.heads, p.dim));
+                up(n_scan, matrix_scan_workspace(sizeof(T) == 2, delta, rows_cap, p.heads, p.kv_heads, p.dim, p.vdim));
                 if (delta) up(n_ch, p.conv_channels());
             }
             up(n_f32, L.n_f32);
@@ -660,7 +660,7 @@ int MixedDecoder<T>::create(const tllm_b200_mixed_desc& c, int flags_, int max_b
     TRY(dev_alloc(&expert_out, some(n_gather * w), true));
     TRY(dev_alloc(&hidden, some(n_hidden), true));
     TRY(dev_alloc(&counts, some(2 * n_experts), true));
-    TRY(dev_alloc(&group, some(n_gather / kGroupRows), true));
+    TRY(dev_alloc(&group, some(3 * n_gather / kGroupRows), true));
     TRY(dev_alloc(&groups, 1, true));
     if (sizeof(T) == 2) {
         TRY(dev_alloc(&kx, some(max_seq * n_k), true));

@@ -207,7 +207,7 @@ struct MatrixScanArgs {
     StepGeo g;
 };
 // bytes for a step of `rows` tokens in all
-size_t matrix_scan_workspace(bool bf16_path, bool delta, int rows, int heads, int dim);
+size_t matrix_scan_workspace(bool bf16_path, bool delta, int rows, int heads, int kv_heads, int dim, int vdim);
 template <typename T>
 int launch_matrix_scan(const MatrixScanArgs<T>& a, cudaStream_t stream);
 
@@ -246,10 +246,9 @@ struct ExpertArgs {
     int *chosen = nullptr, *part_row = nullptr;    // [rows, top]
     float* part_w = nullptr;                       // [rows, top]
     T* gathered = nullptr;             // [expert_rows, w]
-    int *group = nullptr, *groups = nullptr;       // expert of every 128 rows; number of groups
+    int *group = nullptr, *groups = nullptr;       // LinearArgs::group: [3 * expert_rows / kGroupRows], [1]
 };
 int expert_rows(int rows, int top, int experts);   // capacity of the gathered rows
-bool experts_few_fits(int top, int ff, int w, size_t element);
 template <typename T>
 int launch_experts_few(const ExpertArgs<T>& a, cudaStream_t stream);
 template <typename T>
