@@ -8,8 +8,9 @@
 //             decode and short portions (positions split over CTAs, merged afterwards; a single
 //             token's norms, rotation and cache append happen in the same launch) and the exact
 //             32-bit mode
-//   prompt -- 64 queries of a head per CTA on mma.sync, BF16; only the tiles some query sees.
-//             Scores FP32, softmax weights enter the second product as two BF16 numbers.
+//   prompt -- BF16, only the tiles some query sees; scores FP32, softmax weights enter the second
+//             product as two BF16 numbers.  Long portions of the usual head sizes on tcgen05
+//             (grouped_prompt.cu), the rest here: 64 queries of a head per CTA on mma.sync.
 #include <cfloat>
 
 #include "launch.cuh"
@@ -113,42 +114,39 @@ __device__ __forceinline__ void norm_rotate8(const T* x, const GroupedArgs<T>& a
 // ---------------------------------------------------------------------------
 // Norms, rotations, cache append
 // ---------------------------------------------------------------------------
-constexpr int kPrepThreads = 256, kPrepWarps = kPrepThreads / 32;
+constexpr int kPrepThreads = 256;
 
+// A row is the work of `warps` warps: `hpw` heads each (queries, then keys), then the values.
 template <typename T>
 __global__ void __launch_bounds__(kPrepThreads)
-grouped_prep_kernel(const GroupedArgs<T> a)
+grouped_prep_kernel(const GroupedArgs<T> a, int warps, int hpw)
 {
     pdl_launch_dependents();
-    const int row = blockIdx.x, b = row / a.g.seq_len, t = row - b * a.g.seq_len;
-    const int warp = threadIdx.x >> 5;
+    const int unit = (blockIdx.x * kPrepThreads + threadIdx.x) >> 5, lane = threadIdx.x & 31;      // warp of all
+    const int row = unit / warps, it = unit - row * warps, b = row / a.g.seq_len, t = row - b * a.g.seq_len;
     pdl_wait();
     const int pos = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) + t;
-    if (pos >= a.max_seq) return;
+    if (row >= a.g.n_seq * a.g.seq_len || pos >= a.max_seq) return;
     const int r = pos % a.cache_rows;
     T* proj = a.proj + (size_t)row * a.ld;
     T* kc = a.kc + (size_t)(a.g.first_slot + b) * a.k_slot + (size_t)r * a.kv_heads * a.dim;
     T* vc = a.vc + (size_t)(a.g.first_slot + b) * a.v_slot + (size_t)r * a.kv_heads * a.vdim;
-    if (rotates8(a)) {
-        const int lanes = a.dim <= 64 ? 8 : a.dim <= 128 ? 16 : 32, l = threadIdx.x & (lanes - 1), per = kPrepThreads / lanes;
-        for (int h0 = 0; h0 < a.heads + a.kv_heads; h0 += per) {          // all lanes take part in every round
-            const int hh = h0 + threadIdx.x / lanes, h = min(hh, a.heads + a.kv_heads - 1);
-            const bool q = h < a.heads;
-            const T* src = q ? proj + a.q_off + (size_t)h * a.dim : proj + a.k_off + (size_t)(h - a.heads) * a.dim;
-            T* dst = q ? const_cast<T*>(src) : kc + (size_t)(h - a.heads) * a.dim;
-            norm_rotate8<T>(src, a, q ? a.q_norm : a.k_norm, pos, lanes, l, [&](int i, const float (&v)[8]) { if (hh == h) store8(dst + i, v); });
-        }
-    } else
-    for (int h = warp; h < a.heads + a.kv_heads; h += kPrepWarps) {
-        const bool q = h < a.heads;
-        const T* src = q ? proj + a.q_off + (size_t)h * a.dim : proj + a.k_off + (size_t)(h - a.heads) * a.dim;
-        T* dst = q ? const_cast<T*>(src) : kc + (size_t)(h - a.heads) * a.dim;
-        // in place: a lane writes only what it alone has read (the sum of squares comes first)
-        norm_rotate<T>(src, a, q ? a.q_norm : a.k_norm, pos, [&](int i, float v) { dst[i] = from_f<T>(v); });
-    }
     constexpr int V = Vec16<T>::n;
-    const uint4* vs = reinterpret_cast<const uint4*>(proj + a.v_off);
-    for (int i = threadIdx.x; i < a.kv_heads * a.vdim / V; i += kPrepThreads) reinterpret_cast<uint4*>(vc)[i] = vs[i];
+    const int heads = a.heads + a.kv_heads, head_warps = (heads + hpw - 1) / hpw;
+    if (it >= head_warps) {                             // values: 32 pieces of 16 bytes
+        const int i = (it - head_warps) * 32 + lane;
+        if (i < a.kv_heads * a.vdim / V) reinterpret_cast<uint4*>(vc)[i] = reinterpret_cast<const uint4*>(proj + a.v_off)[i];
+        return;
+    }
+    // in place: an entry is written only by lanes that have read it (the sum of squares comes first)
+    const int lanes = 32 / hpw, hh = it * hpw + lane / lanes, h = min(hh, heads - 1);
+    const bool q = h < a.heads;
+    const T* src = q ? proj + a.q_off + (size_t)h * a.dim : proj + a.k_off + (size_t)(h - a.heads) * a.dim;
+    T* dst = q ? const_cast<T*>(src) : kc + (size_t)(h - a.heads) * a.dim;
+    if (rotates8(a))
+        norm_rotate8<T>(src, a, q ? a.q_norm : a.k_norm, pos, lanes, lane & (lanes - 1), [&](int i, const float (&v)[8]) { if (hh == h) store8(dst + i, v); });
+    else
+        norm_rotate<T>(src, a, q ? a.q_norm : a.k_norm, pos, [&](int i, float v) { dst[i] = from_f<T>(v); });
 }
 
 // ---------------------------------------------------------------------------
@@ -603,6 +601,7 @@ bool prompt_fits(const GroupedArgs<bf16>& a) { return a.g.seq_len >= kPromptFrom
 int prompt_path(const GroupedArgs<float>&, cudaStream_t) { return TLLM_ERR_SHAPE; }
 int prompt_path(const GroupedArgs<bf16>& a, cudaStream_t stream)
 {
+    if (grouped_prompt_tcgen05_supported(a)) return launch_grouped_prompt_tcgen05(a, stream);
     const dim3 grid((a.g.seq_len + kPq - 1) / kPq, a.heads, a.g.n_seq), block(kPqThreads);
     const size_t smem = prompt_smem(a.dim, a.vdim);
     const int nv = (a.vdim + 15) / 16 * 2;
@@ -623,7 +622,7 @@ int prompt_path(const GroupedArgs<bf16>& a, cudaStream_t stream)
 
 int grouped_cache_rows(int max_seq, int chunk, int rows)
 {
-    const long long need = (long long)chunk + rows;
+    const long long need = ((long long)chunk + rows + 127) / 128 * 128;       // whole tiles of the prompt kernel
     return chunk > 0 && need < max_seq ? (int)need : max_seq;
 }
 
@@ -652,7 +651,10 @@ int launch_grouped_attention(const GroupedArgs<T>& a, float* ws, cudaStream_t st
     if (a.g.seq_len > 1) {
         if (a.cache_rows < a.max_seq && (a.chunk < 1 || a.chunk + a.g.seq_len > a.cache_rows))
             return fail(TLLM_ERR_SHAPE, "grouped attention: %d tokens with %d cache rows", a.g.seq_len, a.cache_rows);
-        const int st = launch_pdl("grouped_prep", grouped_prep_kernel<T>, dim3(a.g.rows()), dim3(kPrepThreads), 0, stream, a);
+        const int hpw = !rotates8(a) || a.dim > 128 ? 1 : a.dim > 64 ? 2 : 4, piece = 32 * Vec16<T>::n;
+        const int warps = (a.heads + a.kv_heads + hpw - 1) / hpw + (a.kv_heads * a.vdim + piece - 1) / piece;
+        const unsigned ctas = ((unsigned)a.g.rows() * warps + kPrepThreads / 32 - 1) / (kPrepThreads / 32);
+        const int st = launch_pdl("grouped_prep", grouped_prep_kernel<T>, dim3(ctas), dim3(kPrepThreads), 0, stream, a, warps, hpw);
         if (st) return st;
         if (prompt_fits(a)) return prompt_path(a, stream);
     }

@@ -181,6 +181,9 @@ int grouped_cache_rows(int max_seq, int chunk, int rows);
 bool grouped_supported(int heads, int kv_heads, int dim, int vdim);
 size_t grouped_workspace_floats(int heads, int vdim);
 // norms, rotations, cache append and attention of a step; ws: grouped_workspace_floats
+// the attention of prompts on tcgen05 (grouped_prompt.cu); keys and values are in the cache
+bool grouped_prompt_tcgen05_supported(const GroupedArgs<bf16>& a);
+int launch_grouped_prompt_tcgen05(const GroupedArgs<bf16>& a, cudaStream_t stream);
 template <typename T>
 int launch_grouped_attention(const GroupedArgs<T>& a, float* ws, cudaStream_t stream);
 

@@ -75,12 +75,42 @@ def test_grouped_attention(case, dt):
         close(torch.cat(got, dim=1), want, 3e-5 if dt == "float32" else 2e-2, f"cuts {cuts[:4]}")
 
 
+@pytest.mark.parametrize("d,e", [(64, 64), (64, 128), (128, 64), (128, 128)])
+@pytest.mark.parametrize("chunk,ring", [(0, 0), (100, 0), (128, 512), (300, 768), (1, 0)])
+def test_grouped_attention_over_long_prompts(chunk, ring, d, e):
+    """Head sizes and lengths of the tensor-memory kernel: portions of 128 tokens and more from
+    positions inside a tile, chunks of every alignment, a ring of cache rows, a sharp softmax whose
+    maximum keeps growing."""
+    H, G, n = 4, 2, 700
+    rng = np.random.default_rng(chunk + d)
+    x = rounded(rng.standard_normal((1, n, H * d + G * (d + e))), "bfloat16")
+    x[0, :, H * d:(H + G) * d] *= np.linspace(0.2, 3.0, n)[:, None]           # scores grow along the sequence
+    x = rounded(x, "bfloat16")
+    scale, rows = 4.0 * d ** -0.5, ring or n
+    want = attend(x[0], None, None, 1e-5, 300.0, 32, scale, chunk, H, G, d, e)[None]
+    for cuts in ([700], [128, 130, 442], [5, 300, 200, 195], [130, 1, 1, 568]):
+        if ring and max(cuts) > ring - chunk:
+            continue
+        kc = torch.full((1, rows, G * d), float("nan"), device="cuda", dtype=torch.bfloat16)
+        vc = torch.full((1, rows, G * e), float("nan"), device="cuda", dtype=torch.bfloat16)
+        got, pos = [], 0
+        for c in cuts:
+            o = torch.full((1, c, H * e), float("nan"), device="cuda", dtype=torch.bfloat16)
+            ops.grouped_attention(dev(x[:, pos:pos + c], torch.bfloat16), None, None, 1e-5, rope_table(n, 300.0, 32), 32, kc, vc, o, H, G, d, e, chunk,
+                                  rows, n, scale, 1, c, pos)
+            got.append(o)
+            pos += c
+        close(torch.cat(got, dim=1), want, 2e-2, f"cuts {cuts}")
+    tl.check_device_errors()
+
+
 @pytest.mark.parametrize("dt", list(DT))
 @pytest.mark.parametrize("chunk", [0, 200])
-def test_grouped_attention_finds_one_key_just_inside_and_never_outside(dt, chunk):
+@pytest.mark.parametrize("d", [16, 64])
+def test_grouped_attention_finds_one_key_just_inside_and_never_outside(dt, chunk, d):
     """One key matches the query of every position; its value is the output exactly where the mask
     shows it: from its own position to the end of its chunk."""
-    H, G, d, e, n = 2, 1, 16, 8, 470
+    H, G, e, n = 2, 1, {16: 8, 64: 64}[d], 470
     for at in (0, 63, 64, 199, 200, 399):
         x = np.zeros((1, n, H * d + G * (d + e)))
         x[..., d - 1:H * d:d] = 1.0
