@@ -173,7 +173,7 @@ int matrix_op(int delta, const void* qkv, const float* decay, const float* a, co
     float* ws = nullptr;
     return with_records((matrix_scan_workspace(sizeof(T) == 2, m.delta, g.rows(), heads, kv_heads, dim, vdim) + 3) / 4, &ws, s, [&] {
         m.ws = ws;
-        return launch_matrix_scan<T>(m, s);
+        return launch_matrix_scan<T>(m, static_cast<const GatedNormArgs<T>*>(nullptr), s);
     });
 }
 

@@ -15,6 +15,7 @@
 // as the BF16 numbers they are; their norms, decays and step sizes stay FP32 factors outside the
 // products; the FP32 operands (state, U, P, the inverse) enter as the sum of two BF16 numbers.
 #include "launch.cuh"
+#include "matrix_step.cuh"
 #include "mixers.cuh"
 #include "mma_sync.cuh"
 #include "tcgen05.cuh"
@@ -23,129 +24,10 @@ namespace tllm {
 
 namespace {
 
-constexpr float kUnitEps = 1e-6f;     // under the root of the unit vectors
-
-__device__ __forceinline__ float log_decay(float a, float dt_bias, float neg_a) { return neg_a * softplus_f(a + dt_bias); }
-
-// ---------------------------------------------------------------------------
-// Token by token
-// ---------------------------------------------------------------------------
-constexpr int kSeqThreads = 256, kSeqStates = 16, kSeqTokens = 8;   // entries of a column per lane; tokens staged together
-
-// A column of S is spread over `lpc` lanes in pieces of four entries; a CTA serves blockDim / lpc
-// columns of one head.
-template <typename T, bool DELTA>
-__global__ void __launch_bounds__(kSeqThreads)
-matrix_seq_kernel(const MatrixScanArgs<T> a, int lpc)
-{
-    extern __shared__ __align__(16) float smem[];
-    constexpr int NP = kSeqStates / 4;
-    const int cols = blockDim.x / lpc, D = a.dim, D4 = D >> 2;
-    float* ks = smem;                                   // [tokens][D]
-    float* qs = ks + kSeqTokens * D;
-    float* vs = qs + kSeqTokens * D;                    // [tokens][cols]
-    float* gs = vs + kSeqTokens * cols;                 // decay, step size
-    float* bs = gs + kSeqTokens;
-    pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
-    const int cl = tid / lpc, l = tid - cl * lpc, c0 = blockIdx.x * cols, c = c0 + cl, h = blockIdx.y, b = blockIdx.z;
-    const int kh = h / (a.heads / a.kv_heads);
-    const bool live = c < a.vdim;
-    pdl_wait();
-    const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
-    float4* st = reinterpret_cast<float4*>(a.state + (size_t)(a.g.first_slot + b) * a.slot_stride + ((size_t)h * a.vdim + (live ? c : 0)) * D);
-    float4 S[NP];
-#pragma unroll
-    for (int u = 0; u < NP; u++) {
-        const int p = l + u * lpc;
-        S[u] = (live && !fresh && p < D4) ? st[p] : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    const int n = a.g.seq_len;
-    const size_t row0 = (size_t)b * n;
-    for (int t0 = 0; t0 < n; t0 += kSeqTokens) {
-        const int nt = min(kSeqTokens, n - t0);
-        __syncthreads();
-        // a warp per vector: keys, queries, values of the staged tokens
-        for (int i = warp; i < 3 * nt; i += warps) {
-            const int t = i / 3, what = i - 3 * t;
-            const size_t row = row0 + t0 + t;
-            if (what == 2) {
-                const T* v = a.v + row * a.ld + (size_t)h * a.vdim + c0;
-                for (int j = lane; j < cols; j += 32) vs[t * cols + j] = c0 + j < a.vdim ? to_f<T>(v[j]) : 0.f;
-                if (lane == 0) {
-                    if (DELTA) {
-                        const float lg = log_decay(a.a[row * a.ld_ab + h], a.dt_bias[h], a.neg_a[h]);
-                        gs[t] = decay_exp(lg, expf(lg));
-                        bs[t] = sigmoid_f(a.b[row * a.ld_ab + h]);
-                    } else {
-                        gs[t] = a.decay[h];
-                    }
-                }
-                continue;
-            }
-            const T* x = (what ? a.q : a.k) + row * a.ld + (size_t)kh * D;
-            float* dst = (what ? qs : ks) + t * D;
-            float f = 1.f;
-            if (DELTA) {
-                float ss = 0.f;
-                for (int j = lane; j < D; j += 32) {
-                    const float v = to_f<T>(x[j]);
-                    ss += v * v;
-                }
-                f = 1.f / sqrtf(warp_sum(ss) + kUnitEps);
-                if (what) f *= a.q_scale;
-            }
-            for (int j = lane; j < D; j += 32) dst[j] = to_f<T>(x[j]) * f;
-        }
-        __syncthreads();
-        for (int t = 0; t < nt; t++) {
-            const float g = gs[t];
-            const float4 *kp = reinterpret_cast<const float4*>(ks + t * D), *qp = reinterpret_cast<const float4*>(qs + t * D);
-            float4 k[NP];
-#pragma unroll
-            for (int u = 0; u < NP; u++) k[u] = l + u * lpc < D4 ? kp[l + u * lpc] : make_float4(0.f, 0.f, 0.f, 0.f);
-            float add = vs[t * cols + cl];
-            if (DELTA) {
-                float p = 0.f;
-#pragma unroll
-                for (int u = 0; u < NP; u++) {
-                    S[u].x *= g;
-                    S[u].y *= g;
-                    S[u].z *= g;
-                    S[u].w *= g;
-                    p = fmaf(S[u].x, k[u].x, fmaf(S[u].y, k[u].y, fmaf(S[u].z, k[u].z, fmaf(S[u].w, k[u].w, p))));
-                }
-                for (int o = lpc >> 1; o > 0; o >>= 1) p += __shfl_xor_sync(0xffffffffu, p, o);
-                add = bs[t] * (add - p);
-            }
-            float o = 0.f;
-#pragma unroll
-            for (int u = 0; u < NP; u++) {
-                const float d = DELTA ? 1.f : g;
-                S[u].x = fmaf(k[u].x, add, d * S[u].x);
-                S[u].y = fmaf(k[u].y, add, d * S[u].y);
-                S[u].z = fmaf(k[u].z, add, d * S[u].z);
-                S[u].w = fmaf(k[u].w, add, d * S[u].w);
-                if (l + u * lpc < D4) {
-                    const float4 q = qp[l + u * lpc];
-                    o = fmaf(S[u].x, q.x, fmaf(S[u].y, q.y, fmaf(S[u].z, q.z, fmaf(S[u].w, q.w, o))));
-                }
-            }
-            for (int s = lpc >> 1; s > 0; s >>= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
-            if (live && l == 0) a.o[(row0 + t0 + t) * ((size_t)a.heads * a.vdim) + (size_t)h * a.vdim + c] = o;
-        }
-    }
-    if (live) {
-#pragma unroll
-        for (int u = 0; u < NP; u++)
-            if (l + u * lpc < D4) st[l + u * lpc] = S[u];
-    }
-}
-
 // ---------------------------------------------------------------------------
 // Chunks
 // ---------------------------------------------------------------------------
-constexpr int kC = 64, kChunkThreads = 128, kScanThreads = 256;
+constexpr int kC = 64, kChunkThreads = 256;
 constexpr int kLdC = kC + 8;                       // row stride of a [64][64] tile in shared memory
 constexpr int kLdA = kC + 4;                       // of an FP32 one
 
@@ -168,7 +50,9 @@ __device__ __forceinline__ void bulk_copy(void* dst, const void* src, uint32_t b
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
                  ::"r"(sm32(dst)), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
-__device__ __forceinline__ void carriers_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+template <int THREADS>
+__device__ __forceinline__ void carriers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
+constexpr int kThreadsPerCol = 16;                 // scan: carriers and outputs, 4 warps per group of 16 columns each
 __host__ __device__ inline size_t chunk_mats(bool delta) { return delta ? 4 : 2; }
 inline int chunks_of(int n) { return (n + kC - 1) / kC; }
 
@@ -196,13 +80,13 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
     pdl_wait();
     {
         const int pieces = D / 8, per = ld / 8;
-        for (int i = tid; i < kC * per; i += kChunkThreads) {
-            const int r = i / per, c = i - r * per;
-            const bool v = r < n && c < pieces;
-            const size_t o = (row0 + (v ? r : 0)) * a.ld + (size_t)kh * D + (v ? c * 8 : 0);
-            cp16(ks + r * ld + c * 8, a.k + o, v);
-            cp16(qs + r * ld + c * 8, a.q + o, v);
-        }
+        for (int r = warp; r < kC; r += kChunkThreads / 32)
+            for (int c = lane; c < per; c += 32) {
+                const bool v = r < n && c < pieces;
+                const size_t o = (row0 + (v ? r : 0)) * a.ld + (size_t)kh * D + (v ? c * 8 : 0);
+                cp16(ks + r * ld + c * 8, a.k + o, v);
+                cp16(qs + r * ld + c * 8, a.q + o, v);
+            }
         cp_commit();
     }
     if (DELTA && warp == 0) {
@@ -225,12 +109,14 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
     {
         const int slices = (a.vdim + ws.nv - 1) / ws.nv, per = ws.nv / 8, ldv = ws.nv + 8;
         bf16* v = ws.v + unit * slices * kC * ldv;
-        for (int i = tid; i < kC * slices * per; i += kChunkThreads) {
-            const int r = i / (slices * per), c = i - r * slices * per, s = c / per;
-            const uint4 x = (r < n && c * 8 < a.vdim) ? *(reinterpret_cast<const uint4*>(a.v + (row0 + r) * a.ld + (size_t)h * a.vdim) + c)
-                                                      : make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(v + (s * kC + r) * ldv + (c - s * per) * 8) = x;
-        }
+        const int shift = per == 2 ? 1 : 2;
+        for (int r = warp; r < kC; r += kChunkThreads / 32)
+            for (int c = lane; c < slices * per; c += 32) {
+                const uint4 x = (r < n && c * 8 < a.vdim) ? *(reinterpret_cast<const uint4*>(a.v + (row0 + r) * a.ld + (size_t)h * a.vdim) + c)
+                                                          : make_uint4(0, 0, 0, 0);
+                const int s = c >> shift;
+                *reinterpret_cast<uint4*>(v + (s * kC + r) * ldv + (c - s * per) * 8) = x;
+            }
     }
     cp_wait<0>();
     __syncthreads();
@@ -308,9 +194,9 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
                 *reinterpret_cast<uint32_t*>(mats + kC * kLdC + i * kLdC + c) = lo;
             }
     };
-    write_p(warp * 16);
+    if (warp >= 4) write_p((warp - 4) * 16);
     if (!DELTA) return;
-    {
+    if (warp < 4) {
         float s[8][4];
         gram(ks, warp * 16, s);
 #pragma unroll
@@ -342,41 +228,34 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
         }
     }
     __syncthreads();
-    // then block (j + d, j) = -inv_ii sum_k A_ik inv_kj, one distance after the other: 16 threads per
-    // block, 4 x 4 entries each
-    const int j = tid >> 4, tr = (tid >> 2 & 3) * 4, tc = (tid & 3) * 4;
-    auto tile_product = [&](const float* x, int ldx, const float* y, int ldy, int n, float (&v)[4][4]) {
-#pragma unroll
-        for (int r = 0; r < 4; r++)
-#pragma unroll
-            for (int c = 0; c < 4; c++) v[r][c] = 0.f;
-#pragma unroll 4
+    // then block (j + d, j) = -inv_ii sum_k A_ik inv_kj, one distance after the other: 64 threads per
+    // block, 2 x 2 entries each
+    const int j = tid >> 6, tr = (tid >> 3 & 7) * 2, tc = (tid & 7) * 2;
+    auto tile_product = [&](const float* x, int ldx, const float* y, int ldy, int n, float2 (&v)[2]) {
+        v[0] = v[1] = make_float2(0.f, 0.f);
+#pragma unroll 8
         for (int k = 0; k < n; k++) {
-            const float4 q = *reinterpret_cast<const float4*>(y + k * ldy + tc);
-#pragma unroll
-            for (int r = 0; r < 4; r++) {
-                const float p = x[(tr + r) * ldx + k];
-                v[r][0] = fmaf(p, q.x, v[r][0]);
-                v[r][1] = fmaf(p, q.y, v[r][1]);
-                v[r][2] = fmaf(p, q.z, v[r][2]);
-                v[r][3] = fmaf(p, q.w, v[r][3]);
-            }
+            const float2 q = *reinterpret_cast<const float2*>(y + k * ldy + tc);
+            const float p0 = x[tr * ldx + k], p1 = x[(tr + 1) * ldx + k];
+            v[0].x = fmaf(p0, q.x, v[0].x);
+            v[0].y = fmaf(p0, q.y, v[0].y);
+            v[1].x = fmaf(p1, q.x, v[1].x);
+            v[1].y = fmaf(p1, q.y, v[1].y);
         }
     };
     for (int d = 1; d < nb; d++) {
-        float v[4][4];
+        float2 v[2];
         const int i0 = (j + d) * kB;
         if (j + d < nb) {
             tile_product(A + i0 * kLdA + j * kB, kLdA, inv + j * kB * kLdA + j * kB, kLdA, d * kB, v);
-#pragma unroll
-            for (int r = 0; r < 4; r++) *reinterpret_cast<float4*>(tmp + j * kB * kB + (tr + r) * kB + tc) = make_float4(v[r][0], v[r][1], v[r][2], v[r][3]);
+            *reinterpret_cast<float2*>(tmp + j * kB * kB + tr * kB + tc) = v[0];
+            *reinterpret_cast<float2*>(tmp + j * kB * kB + (tr + 1) * kB + tc) = v[1];
         }
         __syncthreads();
         if (j + d < nb) {
             tile_product(inv + i0 * kLdA + i0, kLdA, tmp + j * kB * kB, kB, kB, v);
-#pragma unroll
-            for (int r = 0; r < 4; r++)
-                *reinterpret_cast<float4*>(inv + (i0 + tr + r) * kLdA + j * kB + tc) = make_float4(-v[r][0], -v[r][1], -v[r][2], -v[r][3]);
+            *reinterpret_cast<float2*>(inv + (i0 + tr) * kLdA + j * kB + tc) = make_float2(-v[0].x, -v[0].y);
+            *reinterpret_cast<float2*>(inv + (i0 + tr + 1) * kLdA + j * kB + tc) = make_float2(-v[1].x, -v[1].y);
         }
         __syncthreads();
     }
@@ -391,20 +270,21 @@ chunk_prepare_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws)
     }
 }
 
-// A segment of the chunks and NV columns of the state per CTA.  Four warps carry the state (U, then
-// the state behind the chunk; MT tiles of 16 rows each), four others compute the outputs beside
-// them.  `stages` chunks are in flight.
+// A segment of the chunks and NV columns of the state per CTA.  Half of the warps carry the state
+// (U, then the state behind the chunk), the others compute the outputs beside them; in each half
+// four row tiles (of tokens; of the state MT each) times groups of 16 columns.  `stages` chunks are
+// in flight.
 //
 // Linear attention is cut into segments that run at the same time: RECORD runs all but the last
 // from a zero state and keeps their final states, the second launch starts each segment from the
 // carried state and the records before it.  (The record of the last segment holds a copy of the
 // carried state, which that segment overwrites while others may not have started.)
 template <bool DELTA, int NV, int MT, bool RECORD>
-__global__ void __launch_bounds__(kScanThreads)
+__global__ void __launch_bounds__(kThreadsPerCol * NV)
 chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_seg, int nseg, int stages)
 {
     extern __shared__ __align__(16) uint8_t smem_raw[];
-    constexpr int ldv = NV + 8, NT = NV / 8, MATS = DELTA ? 4 : 2;
+    constexpr int kGroups = NV / 16, kThreads = kThreadsPerCol * NV, ldv = NV + 8, NT = 2, MATS = DELTA ? 4 : 2;
     const int D = a.dim, D16 = (D + 15) & ~15, ld = D16 + 8, ksteps = D16 / 16;
     const int tile = 2 * kC * ld + MATS * kC * kLdC + kC * ldv;               // bf16 of a stage, then 4 * 64 floats
     const size_t stage_bytes = (size_t)tile * 2 + 4 * kC * sizeof(float);
@@ -415,8 +295,11 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
     __shared__ __align__(8) uint64_t full[2];
     __shared__ int abort_flag;
     pdl_launch_dependents();
-    const int tid = threadIdx.x, warp = (tid >> 5) & 3, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
-    const bool carrier = tid < 128;                                            // carries the state
+    const int tid = threadIdx.x, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
+    const bool carrier = tid < kThreads / 2;                                   // carries the state
+    // the triangular products grow with the row: the other way round in the two halves, which share schedulers
+    const int warp = carrier ? tid >> 5 & 3 : 3 - (tid >> 5 & 3);
+    const int n0 = (tid >> 7) % kGroups * NT * 8;                              // first column of the warp
     const int slices = (a.vdim + NV - 1) / NV, seg = blockIdx.x / slices;
     const int v0 = (blockIdx.x - seg * slices) * NV, h = blockIdx.y, b = blockIdx.z, kh = h / (a.heads / a.kv_heads);
     const int nv = min(NV, a.vdim - v0), c0 = seg * per_seg, c1 = min(nchunk, c0 + per_seg);
@@ -447,7 +330,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
         bulk_copy(p + 2 * kC * ld + MATS * kC * kLdC, ws.v + (unit * slices + v0 / NV) * kC * ldv, v, bar);
         bulk_copy(p + tile, ws.vecs + unit * 4 * kC, vec, bar);
     };
-    const bool requester = tid == 128;
+    const bool requester = tid == kThreads / 2;
     if (requester) request(c0, 0);
 
     float S[MT][NT][4];
@@ -458,7 +341,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
             for (int j = 0; j < NT; j++)
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
-                    const int r = (warp + 4 * i) * 16 + gq + (e >> 1) * 8, c = j * 8 + 2 * tq + (e & 1);
+                    const int r = (warp + 4 * i) * 16 + gq + (e >> 1) * 8, c = n0 + j * 8 + 2 * tq + (e & 1);
                     const bool in = r < D && c < nv;
                     f(S[i][j][e], in, in ? (size_t)c * D + r : 0);   // a place that may be read either way
                 }
@@ -474,7 +357,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
                 for (int half = 0; half < 2; half++) {
                     uint32_t hi, lo;
                     split2(S[i][j][2 * half], S[i][j][2 * half + 1], hi, lo);
-                    const int o = (r + half * 8) * ldv + j * 8 + 2 * tq;
+                    const int o = (r + half * 8) * ldv + n0 + j * 8 + 2 * tq;
                     *reinterpret_cast<uint32_t*>(sh + o) = hi;
                     *reinterpret_cast<uint32_t*>(sh + D16 * ldv + o) = lo;
                 }
@@ -512,13 +395,10 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
     };
     // x += (16 rows of the matrix m, its columns 16 k ..) times rows 16 k .. of u
     auto times = [&](float (&x)[NT][4], const uint32_t (&f)[4], const bf16* u, int k) {
-#pragma unroll
-        for (int j = 0; j < NT; j += 2) {
-            uint32_t fb[4];
-            ldsm4t(fb, u + (k * 16 + lda) * ldv + j * 8 + ldb);
-            mma16816(x[j], f, fb[0], fb[1]);
-            mma16816(x[j + 1], f, fb[2], fb[3]);
-        }
+        uint32_t fb[4];
+        ldsm4t(fb, u + (k * 16 + lda) * ldv + n0 + ldb);
+        mma16816(x[0], f, fb[0], fb[1]);
+        mma16816(x[1], f, fb[2], fb[3]);
     };
 
     bool ok = true;
@@ -561,7 +441,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
                 for (int j = 0; j < NT; j++)
 #pragma unroll
                     for (int half = 0; half < 2; half++) {
-                        const int i = i0 + half * 8, o = i * ldv + j * 8 + 2 * tq;
+                        const int i = i0 + half * 8, o = i * ldv + n0 + j * 8 + 2 * tq;
                         const float f = dec[half] * rk[i], be = beta[i];
                         const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vt + o));
                         uint32_t hi, lo;
@@ -569,7 +449,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
                         *reinterpret_cast<uint32_t*>(rs + o) = hi;
                         *reinterpret_cast<uint32_t*>(rs + kC * ldv + o) = lo;
                     }
-                carriers_sync();
+                carriers_sync<kThreads / 2>();
                 float mid[NT][4];
                 zero(acc);
                 zero(low);
@@ -589,7 +469,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
             for (int j = 0; j < NT; j++)
 #pragma unroll
                 for (int half = 0; half < 2; half++) {
-                    const int o = (i0 + half * 8) * ldv + j * 8 + 2 * tq;
+                    const int o = (i0 + half * 8) * ldv + n0 + j * 8 + 2 * tq;
                     float2 u;
                     uint32_t hi, lo;
                     if (DELTA) {
@@ -604,7 +484,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
                     *reinterpret_cast<uint32_t*>(ups + o) = hi;
                     *reinterpret_cast<uint32_t*>(ups + kC * ldv + o) = lo;
                 }
-            if (!DELTA) carriers_sync();
+            if (!DELTA) carriers_sync<kThreads / 2>();
         } else if (!RECORD) {
 #pragma unroll 4
             for (int k = 0; k < ksteps; k++) {              // Q S0
@@ -655,7 +535,7 @@ chunk_scan_kernel(const MatrixScanArgs<bf16> a, ChunkWs ws, int nchunk, int per_
                 float* op = a.o + (row0 + (size_t)c * kC + i) * ((size_t)a.heads * a.vdim) + (size_t)h * a.vdim + v0;
 #pragma unroll
                 for (int j = 0; j < NT; j++) {
-                    const int cc = j * 8 + 2 * tq;
+                    const int cc = n0 + j * 8 + 2 * tq;
                     if (cc < nv) *reinterpret_cast<float2*>(op + cc) = make_float2(acc[j][2 * half], acc[j][2 * half + 1]);
                 }
             }
@@ -713,13 +593,14 @@ int chunk_scan(const MatrixScanArgs<bf16>& a, const ChunkWs& ws, int nchunk, cud
     if (nseg > 1) {
         const auto kernel = chunk_scan_kernel<DELTA, NV, MT, !DELTA>;
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        const int st = launch_pdl("chunk_record", kernel, dim3(slices * (nseg - 1), a.heads, a.g.n_seq), dim3(kScanThreads), smem, stream, a, ws, nchunk,
+        const int st = launch_pdl("chunk_record", kernel, dim3(slices * (nseg - 1), a.heads, a.g.n_seq), dim3(kThreadsPerCol * NV), smem, stream, a, ws, nchunk,
                                   per, nseg, stages);
         if (st) return st;
     }
     const auto kernel = chunk_scan_kernel<DELTA, NV, MT, false>;
     cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return launch_pdl("chunk_scan", kernel, dim3(slices * nseg, a.heads, a.g.n_seq), dim3(kScanThreads), smem, stream, a, ws, nchunk, per, nseg, stages);
+    return launch_pdl("chunk_scan", kernel, dim3(slices * nseg, a.heads, a.g.n_seq), dim3(kThreadsPerCol * NV), smem, stream, a, ws, nchunk, per, nseg,
+                      stages);
 }
 
 template <bool DELTA, int NV>
@@ -775,74 +656,39 @@ int chunk_path(const MatrixScanArgs<bf16>& a, cudaStream_t stream)
 int chunk_any(const MatrixScanArgs<bf16>& a, cudaStream_t stream) { return a.delta ? chunk_path<true>(a, stream) : chunk_path<false>(a, stream); }
 int chunk_any(const MatrixScanArgs<float>&, cudaStream_t) { return TLLM_ERR_SHAPE; }
 
+template <typename T, bool DELTA, bool NORM>
+__global__ void __launch_bounds__(NORM ? kSeqMaxThreads : kSeqThreads)
+matrix_seq_kernel(const MatrixScanArgs<T> a, const GatedNormArgs<T> norm, int lpc)
+{
+    extern __shared__ __align__(16) float smem[];
+    pdl_launch_dependents();
+    pdl_wait();
+    matrix_seq<T, DELTA, NORM>(a, norm, lpc, smem, blockIdx.x, blockIdx.y, blockIdx.z);
+}
+
 template <typename T, bool DELTA>
-int sequential(const MatrixScanArgs<T>& a, cudaStream_t stream)
+int sequential(const MatrixScanArgs<T>& a, const GatedNormArgs<T>* norm, cudaStream_t stream)
 {
-    int lpc = 1;
-    while (lpc * kSeqStates < a.dim) lpc *= 2;
-    int threads = kSeqThreads;
-    while (threads > 32 && threads / 2 / lpc >= a.vdim) threads /= 2;
-    const int cols = threads / lpc;
-    const size_t smem = (size_t)kSeqTokens * (2 * a.dim + cols + 2) * sizeof(float);
-    return launch_pdl("matrix_seq", matrix_seq_kernel<T, DELTA>, dim3((a.vdim + cols - 1) / cols, a.heads, a.g.n_seq), dim3(threads), smem, stream, a,
-                      lpc);
+    const SeqPlan p = seq_plan(a.dim, a.vdim);
+    const dim3 grid(p.blocks, a.heads, a.g.n_seq);
+    // one new token, a norm per head: a CTA takes the whole head and its norm
+    if (norm && a.g.seq_len == 1 && norm->groups == a.heads && p.lpc * a.vdim <= kSeqMaxThreads) {
+        const int threads = (p.lpc * a.vdim + 31) / 32 * 32;
+        return launch_pdl("matrix_seq", matrix_seq_kernel<T, DELTA, true>, dim3(1, a.heads, a.g.n_seq), dim3(threads),
+                          seq_smem(a.dim, threads / p.lpc), stream, a, *norm, p.lpc);
+    }
+    const int st = launch_pdl("matrix_seq", matrix_seq_kernel<T, DELTA, false>, grid, dim3(p.threads), p.smem, stream, a, GatedNormArgs<T>(), p.lpc);
+    return st || !norm ? st : launch_gated_norm<T>(*norm, stream);
 }
 
-// ---------------------------------------------------------------------------
-// Gated norm
-// ---------------------------------------------------------------------------
-constexpr int kGnThreads = 256, kGnWarps = kGnThreads / 32;
-
-__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void put4(bf16* p, float4 v)
-{
-    const __nv_bfloat162 x = __floats2bfloat162_rn(v.x, v.y), y = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
-}
-__device__ __forceinline__ float4 get4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 get4(const bf16* p)
-{
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
-                       __uint_as_float(v.y & 0xffff0000u));
-}
-
-// CTA per row; a warp per group, or the whole CTA when the row is one group
 template <typename T>
 __global__ void __launch_bounds__(kGnThreads)
 gated_norm_kernel(const GatedNormArgs<T> a)
 {
     __shared__ float sh[kGnWarps];
     pdl_launch_dependents();
-    const int row = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const bool whole = a.groups == 1;
-    const int step = whole ? kGnThreads : 32, i0 = whole ? tid : lane, n4 = a.n >> 2;
     pdl_wait();
-    for (int g = whole ? 0 : warp; g < a.groups; g += whole ? 1 : kGnWarps) {
-        const float* o = a.o + ((size_t)row * a.groups + g) * a.n;
-        const T* gate = a.gate + (size_t)row * a.ld_gate + (size_t)g * a.n;
-        T* out = a.out + (size_t)row * a.ld_out + (size_t)g * a.n;
-        float ss = 0.f;
-        for (int i = i0; i < n4; i += step) {
-            const float4 v = get4(o + 4 * i);
-            ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
-        }
-        ss = warp_sum(ss);
-        if (whole) {
-            if (lane == 0) sh[warp] = ss;
-            __syncthreads();
-            ss = 0.f;
-#pragma unroll
-            for (int i = 0; i < kGnWarps; i++) ss += sh[i];
-        }
-        const float r = a.out_scale / sqrtf(ss / (float)a.n_true + a.eps);
-        for (int i = i0; i < n4; i += step) {
-            const float4 v = get4(o + 4 * i), w = get4(a.w + 4 * i), z = get4(gate + 4 * i);
-            float t[4] = {z.x, z.y, z.z, z.w};
-            apply_act_n<4>(a.act, t);
-            put4(out + 4 * i, make_float4(v.x * r * w.x * t[0], v.y * r * w.y * t[1], v.z * r * w.z * t[2], v.w * r * w.w * t[3]));
-        }
-    }
+    gated_norm_row<T>(a, blockIdx.x, sh);
 }
 
 }  // namespace
@@ -859,14 +705,16 @@ size_t matrix_scan_workspace(bool bf16_path, bool delta, int rows, int heads, in
 }
 
 template <typename T>
-int launch_matrix_scan(const MatrixScanArgs<T>& a, cudaStream_t stream)
+int launch_matrix_scan(const MatrixScanArgs<T>& a, const GatedNormArgs<T>* norm, cudaStream_t stream)
 {
     if (a.g.rows() == 0) return TLLM_OK;
-    if (a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.dim < 8 || a.dim % 8 || a.dim > 512 || a.vdim < 8 || a.vdim % 8 || a.ld % 8 ||
-        (a.delta ? !a.a || !a.b || !a.neg_a || !a.dt_bias : !a.decay))
-        return fail(TLLM_ERR_SHAPE, "matrix_scan: heads=%d/%d dim=%d (8..512) vdim=%d ld=%d", a.heads, a.kv_heads, a.dim, a.vdim, a.ld);
-    if (sizeof(T) == 2 && chunked(a.g.seq_len, a.dim)) return chunk_any(a, stream);
-    return a.delta ? sequential<T, true>(a, stream) : sequential<T, false>(a, stream);
+    const int st = check_matrix_scan(a);
+    if (st) return st;
+    if (sizeof(T) == 2 && chunked(a.g.seq_len, a.dim)) {
+        const int c = chunk_any(a, stream);
+        return c || !norm ? c : launch_gated_norm<T>(*norm, stream);
+    }
+    return a.delta ? sequential<T, true>(a, norm, stream) : sequential<T, false>(a, norm, stream);
 }
 
 template <typename T>
@@ -878,7 +726,7 @@ int launch_gated_norm(const GatedNormArgs<T>& a, cudaStream_t stream)
 }
 
 #define TLLM_INSTANTIATE(T)                                                    \
-    template int launch_matrix_scan<T>(const MatrixScanArgs<T>&, cudaStream_t); \
+    template int launch_matrix_scan<T>(const MatrixScanArgs<T>&, const GatedNormArgs<T>*, cudaStream_t); \
     template int launch_gated_norm<T>(const GatedNormArgs<T>&, cudaStream_t);
 TLLM_INSTANTIATE(bf16)
 TLLM_INSTANTIATE(float)

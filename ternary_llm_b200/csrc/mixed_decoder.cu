@@ -162,6 +162,9 @@ private:
         return launch_pack<T>(src, p, dst, ld, nullptr);
     }
     int part_state(const HeadPart& p, PartState<T>* s);
+    GroupedArgs<T> grouped_args(const MixLayer<T>& L, const HeadPart& p, const PartState<T>& S, const StepGeo& g) const;
+    MatrixScanArgs<T> matrix_args(const MixLayer<T>& L, const HeadPart& p, const PartState<T>& S, const StepGeo& g) const;
+    GatedNormArgs<T> out_norm_args(const MixLayer<T>& L, const HeadPart& p, int n_rows) const;
     int heads_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, bool conv_done, cudaStream_t s);
     LinearArgs<T> in_product(const MixLayer<T>& L, int n_rows) const;
     LinearArgs<T> head_product(int n, float* out) const;
@@ -908,104 +911,126 @@ LinearArgs<T> MixedDecoder<T>::in_product(const MixLayer<T>& L, int n_rows) cons
     return l;
 }
 
+template <typename T>
+GroupedArgs<T> MixedDecoder<T>::grouped_args(const MixLayer<T>& L, const HeadPart& p, const PartState<T>& S, const StepGeo& g) const
+{
+    GroupedArgs<T> a;
+    a.proj = proj;
+    a.ld = L.in_ld;
+    a.q_off = p.q;
+    a.k_off = p.k;
+    a.v_off = p.v;
+    a.heads = p.heads;
+    a.kv_heads = p.kv_heads;
+    a.dim = p.dim;
+    a.vdim = p.vdim;
+    a.dim_true = p.dim_true;
+    a.q_norm = p.q_norm;
+    a.k_norm = p.k_norm;
+    a.eps = eps;
+    a.rope = p.rope;
+    a.rot_dims = p.rot_dims;
+    a.kc = S.k;
+    a.vc = S.v;
+    a.k_slot = S.k_slot;
+    a.v_slot = S.v_slot;
+    a.cache_rows = S.cache_rows;
+    a.max_seq = max_seq;
+    a.chunk = p.chunk;
+    a.scale = p.scale;
+    a.out_scale = p.out_scale;
+    a.out = mixed + p.out;
+    a.ld_out = L.out.ld;
+    a.g = g;
+    return a;
+}
+
+template <typename T>
+MatrixScanArgs<T> MixedDecoder<T>::matrix_args(const MixLayer<T>& L, const HeadPart& p, const PartState<T>& S, const StepGeo& g) const
+{
+    MatrixScanArgs<T> a;
+    a.delta = p.type == TLLM_MIXER_DELTA_RULE;
+    const T* x = proj + p.q;
+    a.ld = L.in_ld;
+    if (a.delta) {                             // behind the convolution
+        x = conv_out;
+        a.ld = p.conv_channels();
+        a.a = f32buf + p.a;
+        a.b = f32buf + p.b;
+        a.ld_ab = L.n_f32;
+        a.neg_a = p.neg_a;
+        a.dt_bias = p.dt_bias;
+        a.q_scale = 1.f / std::sqrt((float)p.dim_true);
+    } else {
+        a.decay = p.decay;
+    }
+    a.q = x;
+    a.k = x + (p.k - p.q);
+    a.v = x + (p.v - p.q);
+    a.heads = p.heads;
+    a.kv_heads = p.kv_heads;
+    a.dim = p.dim;
+    a.vdim = p.vdim;
+    a.state = S.rec;
+    a.slot_stride = S.rec_slot;
+    a.o = heads_o;
+    a.ws = scan_ws;
+    a.g = g;
+    return a;
+}
+
+template <typename T>
+GatedNormArgs<T> MixedDecoder<T>::out_norm_args(const MixLayer<T>& L, const HeadPart& p, int n_rows) const
+{
+    const bool per_head = p.type == TLLM_MIXER_DELTA_RULE;
+    GatedNormArgs<T> n;
+    n.o = heads_o;
+    n.w = p.norm;
+    n.gate = proj + p.gate;
+    n.ld_gate = L.in_ld;
+    n.act = p.gate_act;
+    n.eps = eps;
+    n.out_scale = p.out_scale;
+    n.out = mixed + p.out;
+    n.ld_out = L.out.ld;
+    n.rows = n_rows;
+    n.groups = per_head ? p.heads : 1;
+    n.n = per_head ? p.vdim : p.heads * p.vdim;
+    n.n_true = per_head ? p.vdim_true : p.heads * p.vdim_true;
+    return n;
+}
+
 // Mixers of heads: proj (and f32buf) -> mixed.  conv_done: conv_out is there already.
 template <typename T>
 int MixedDecoder<T>::heads_inner(const MixLayer<T>& L, const RunState<T>& R, const StepGeo& g, bool conv_done, cudaStream_t s)
 {
     int st;
+    if (g.seq_len == 1 && L.parts.size() == 2 && L.parts[0].type == TLLM_MIXER_ATTENTION && L.parts[1].type == TLLM_MIXER_LINEAR_ATTENTION)
+        return launch_heads_step<T>(grouped_args(L, L.parts[0], R.part[0], g), matrix_args(L, L.parts[1], R.part[1], g),
+                                    out_norm_args(L, L.parts[1], g.rows()), ws, s);
     for (size_t i = 0; i < L.parts.size(); i++) {
         const HeadPart& p = L.parts[i];
         const PartState<T>& S = R.part[i];
         if (p.type == TLLM_MIXER_ATTENTION) {
-            GroupedArgs<T> a;
-            a.proj = proj;
-            a.ld = L.in_ld;
-            a.q_off = p.q;
-            a.k_off = p.k;
-            a.v_off = p.v;
-            a.heads = p.heads;
-            a.kv_heads = p.kv_heads;
-            a.dim = p.dim;
-            a.vdim = p.vdim;
-            a.dim_true = p.dim_true;
-            a.q_norm = p.q_norm;
-            a.k_norm = p.k_norm;
-            a.eps = eps;
-            a.rope = p.rope;
-            a.rot_dims = p.rot_dims;
-            a.kc = S.k;
-            a.vc = S.v;
-            a.k_slot = S.k_slot;
-            a.v_slot = S.v_slot;
-            a.cache_rows = S.cache_rows;
-            a.max_seq = max_seq;
-            a.chunk = p.chunk;
-            a.scale = p.scale;
-            a.out_scale = p.out_scale;
-            a.out = mixed + p.out;
-            a.ld_out = L.out.ld;
-            a.g = g;
-            TRY(launch_grouped_attention<T>(a, ws, s));
+            TRY(launch_grouped_attention<T>(grouped_args(L, p, S, g), ws, s));
             continue;
         }
-        MatrixScanArgs<T> a;
-        a.delta = p.type == TLLM_MIXER_DELTA_RULE;
-        const T* x = proj + p.q;
-        a.ld = L.in_ld;
-        if (a.delta) {
-            if (!conv_done) {
-                ConvArgs<T> c;
-                c.x = proj + p.q;
-                c.ldx = L.in_ld;
-                c.w = p.conv;
-                c.state = S.conv;
-                c.slot_stride = S.conv_slot;
-                c.y = conv_out;
-                c.channels = p.conv_channels();
-                c.taps = p.taps;
-                c.act = p.in_act;
-                c.g = g;
-                TRY(launch_causal_conv<T>(c, s));
-            }
-            x = conv_out;
-            a.ld = p.conv_channels();
-            a.a = f32buf + p.a;
-            a.b = f32buf + p.b;
-            a.ld_ab = L.n_f32;
-            a.neg_a = p.neg_a;
-            a.dt_bias = p.dt_bias;
-            a.q_scale = 1.f / std::sqrt((float)p.dim_true);
-        } else {
-            a.decay = p.decay;
+        if (p.type == TLLM_MIXER_DELTA_RULE && !conv_done) {
+            ConvArgs<T> c;
+            c.x = proj + p.q;
+            c.ldx = L.in_ld;
+            c.w = p.conv;
+            c.state = S.conv;
+            c.slot_stride = S.conv_slot;
+            c.y = conv_out;
+            c.channels = p.conv_channels();
+            c.taps = p.taps;
+            c.act = p.in_act;
+            c.g = g;
+            TRY(launch_causal_conv<T>(c, s));
         }
-        a.q = x;
-        a.k = x + (p.k - p.q);
-        a.v = x + (p.v - p.q);
-        a.heads = p.heads;
-        a.kv_heads = p.kv_heads;
-        a.dim = p.dim;
-        a.vdim = p.vdim;
-        a.state = S.rec;
-        a.slot_stride = S.rec_slot;
-        a.o = heads_o;
-        a.ws = scan_ws;
-        a.g = g;
-        TRY(launch_matrix_scan<T>(a, s));
-        GatedNormArgs<T> n;
-        n.o = heads_o;
-        n.w = p.norm;
-        n.gate = proj + p.gate;
-        n.ld_gate = L.in_ld;
-        n.act = p.gate_act;
-        n.eps = eps;
-        n.out_scale = p.out_scale;
-        n.out = mixed + p.out;
-        n.ld_out = L.out.ld;
-        n.rows = g.rows();
-        n.groups = a.delta ? p.heads : 1;
-        n.n = a.delta ? p.vdim : p.heads * p.vdim;
-        n.n_true = a.delta ? p.vdim_true : p.heads * p.vdim_true;
-        TRY(launch_gated_norm<T>(n, s));
+        const GatedNormArgs<T> n = out_norm_args(L, p, g.rows());
+        TRY(launch_matrix_scan<T>(matrix_args(L, p, S, g), &n, s));
     }
     return TLLM_OK;
 }

@@ -212,7 +212,10 @@ struct MatrixScanArgs {
 // bytes for a step of `rows` tokens in all
 size_t matrix_scan_workspace(bool bf16_path, bool delta, int rows, int heads, int kv_heads, int dim, int vdim);
 template <typename T>
-int launch_matrix_scan(const MatrixScanArgs<T>& a, cudaStream_t stream);
+struct GatedNormArgs;
+// norm: null, or the norm that turns o into the mixer's output (o itself is scratch then)
+template <typename T>
+int launch_matrix_scan(const MatrixScanArgs<T>& a, const GatedNormArgs<T>* norm, cudaStream_t stream);
 
 // out = out_scale * (o / rms(o) * w) * act(gate), the norm over groups of n entries (n_true of
 // them count), `groups` per row
@@ -229,6 +232,11 @@ struct GatedNormArgs {
 };
 template <typename T>
 int launch_gated_norm(const GatedNormArgs<T>& a, cudaStream_t stream);
+
+// One new token per sequence of attention and linear attention side by side, in two launches:
+// ranges of positions beside the state's step, then the merge beside the norm.
+template <typename T>
+int launch_heads_step(const GroupedArgs<T>& att, const MatrixScanArgs<T>& scan, const GatedNormArgs<T>& norm, float* ws, cudaStream_t stream);
 
 // ---- mixture of experts ----------------------------------------------------------------------
 // Router logits [rows, ld_z]; the `top` largest are chosen (the lower index on a tie) and weighed
