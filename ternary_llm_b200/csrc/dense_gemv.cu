@@ -264,11 +264,15 @@ dense_gemv_kernel(const LinearArgs<T> a, const GemvNorm f, const GemvTail<T> t, 
                 request();
                 slot = slot == kGroups - 1 ? 0 : slot + 1;
             }
+            if (ROUTE == kRouteSum) {                            // the lanes' parts meet at the end
+                res[0][0] = part == 0 ? wgt[0] * acc[0] : fmaf(wgt[part], acc[0], res[0][0]);
+                if (part + 1 < parts) continue;
+                acc[0] = res[0][0];
+            }
 #pragma unroll
             for (int m = 0; m < MB; m++) {
                 for (int o = lanes_per_row >> 1; o > 0; o >>= 1) acc[m] += __shfl_xor_sync(0xffffffffu, acc[m], o);
-                if (ROUTE == kRouteSum) res[0][m] = part == 0 ? wgt[0] * acc[m] : fmaf(wgt[part], acc[m], res[0][m]);
-                else if (part == 0) res[0][m] = acc[m];
+                if (part == 0 || ROUTE == kRouteSum) res[0][m] = acc[m];
                 else res[1][m] = acc[m];
             }
         }

@@ -147,18 +147,20 @@ __device__ __forceinline__ void grouped_span(const GroupedArgs<T>& a, float* __r
     const size_t krow = (size_t)a.kv_heads * D, vrow = (size_t)a.kv_heads * E;
     const int stored = ONE ? pos : pos + 1;                           // positions before it are in the cache
     auto load = [&](int k0) {
-        const int nk = D / V, nv = E / V;
-        for (int i = tid; i < TK * nk; i += kSpanThreads) {
-            const int r = i / nk, c = i - r * nk, p = k0 + r;
-            const bool v = p < p1 && p < stored;
+        // a row per warp and turn, its key pieces and then its value pieces
+        const int nk = D / V, nv = E / V, base = k0 % a.cache_rows;
+        for (int r = warp; r < TK; r += kSpanWarps) {
+            const int p = k0 + r;
             if (ONE && p == pos) continue;                            // written below
-            copy16(kt + r * ldk + c * V, v ? kc + (size_t)(p % a.cache_rows) * krow + c * V : kc, v);
-        }
-        for (int i = tid; i < TK * nv; i += kSpanThreads) {
-            const int r = i / nv, c = i - r * nv, p = k0 + r;
             const bool v = p < p1 && p < stored;
-            if (ONE && p == pos) continue;
-            copy16(vt + r * E + c * V, v ? vc + (size_t)(p % a.cache_rows) * vrow + c * V : vc, v);
+            int ring = base + r;
+            if (v && ring >= a.cache_rows) ring -= a.cache_rows;
+            const T *ksrc = v ? kc + (size_t)ring * krow : kc, *vsrc = v ? vc + (size_t)ring * vrow : vc;
+            T *kdst = kt + r * ldk, *vdst = vt + r * E;
+            for (int c = lane; c < nk + nv; c += 32) {
+                if (c < nk) copy16(kdst + c * V, v ? ksrc + c * V : kc, v);
+                else copy16(vdst + (c - nk) * V, v ? vsrc + (c - nk) * V : vc, v);
+            }
         }
         cp_commit();
         if (ONE && pos >= k0 && pos < k0 + TK && pos < p1) {          // the new token's key and value, here and into the cache

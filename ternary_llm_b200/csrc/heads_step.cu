@@ -12,7 +12,7 @@ static_assert(kSpanThreads == kSeqThreads && kSpanThreads == kGnThreads, "one bl
 
 template <typename T, int TK>
 __global__ void __launch_bounds__(kSpanThreads)
-heads_step_kernel(const GroupedArgs<T> a, const MatrixScanArgs<T> m, float* __restrict__ ws, int hb, int blocks, int nsplit, int lpc, int col_blocks)
+heads_step_kernel(const GroupedArgs<T> a, const MatrixScanArgs<T> m, float* __restrict__ ws, int hb, int blocks, int nsplit, int log_lpc, int col_blocks)
 {
     extern __shared__ __align__(16) uint8_t smem[];
     pdl_launch_dependents();
@@ -21,7 +21,7 @@ heads_step_kernel(const GroupedArgs<T> a, const MatrixScanArgs<T> m, float* __re
     int i = blockIdx.x;
     if (i < seq_ctas) {
         const int bx = i % col_blocks, h = i / col_blocks % m.heads, b = i / (col_blocks * m.heads);
-        matrix_seq<T, false, false>(m, GatedNormArgs<T>(), lpc, reinterpret_cast<float*>(smem), bx, h, b);
+        matrix_one<T, false, false>(m, GatedNormArgs<T>(), log_lpc, nullptr, bx, h, b);
         return;
     }
     i -= seq_ctas;
@@ -50,11 +50,11 @@ template <typename T, int TK>
 int step_tk(const GroupedArgs<T>& a, const MatrixScanArgs<T>& m, const GatedNormArgs<T>& norm, float* ws, const SpanPlan& p, cudaStream_t stream)
 {
     const SeqPlan q = seq_plan(m.dim, m.vdim);
-    const size_t smem = p.smem > q.smem ? p.smem : q.smem;
+    const size_t smem = p.smem;
     const int rows = a.g.n_seq, ctas = q.blocks * m.heads * rows + rows * a.kv_heads * p.blocks * p.nsplit;
     const auto kernel = heads_step_kernel<T, TK>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    const int st = launch_pdl("heads_step", kernel, dim3(ctas), dim3(kSpanThreads), smem, stream, a, m, ws, p.hb, p.blocks, p.nsplit, q.lpc, q.blocks);
+    const int st = launch_pdl("heads_step", kernel, dim3(ctas), dim3(kSpanThreads), smem, stream, a, m, ws, p.hb, p.blocks, p.nsplit, q.log_lpc, q.blocks);
     if (st) return st;
     return launch_pdl("heads_finish", heads_finish_kernel<T, TK>, dim3(norm.rows + (p.nsplit > 1 ? rows * a.heads : 0)), dim3(kGnThreads), 0, stream, a,
                       norm, ws, p.nsplit);

@@ -36,9 +36,10 @@ inline void prefer_max_shared(const void* kernel)
 }
 
 
+// cluster_x: CTAs along x that form a cluster
 template <typename... KArgs, typename... Args>
-int launch_pdl(const char* what, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
-               Args... args)
+int launch_pdl_cluster(const char* what, void (*kernel)(KArgs...), int cluster_x, dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                       Args... args)
 {
     prefer_max_shared(reinterpret_cast<const void*>(kernel));
     cudaLaunchConfig_t cfg = {};
@@ -46,17 +47,27 @@ int launch_pdl(const char* what, void (*kernel)(KArgs...), dim3 grid, dim3 block
     cfg.blockDim = block;
     cfg.dynamicSmemBytes = smem;
     cfg.stream = stream;
-    cudaLaunchAttribute at[1];
+    cudaLaunchAttribute at[2];
     at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     at[0].val.programmaticStreamSerializationAllowed = 1;
+    at[1].id = cudaLaunchAttributeClusterDimension;
+    at[1].val.clusterDim.x = cluster_x;
+    at[1].val.clusterDim.y = at[1].val.clusterDim.z = 1;
     cfg.attrs = at;
-    cfg.numAttrs = 1;
+    cfg.numAttrs = cluster_x > 1 ? 2 : 1;
     const cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
     if (e != cudaSuccess) {
         cudaGetLastError();
         return fail(TLLM_ERR_LAUNCH, "%s launch: %s", what, cudaGetErrorString(e));
     }
     return TLLM_OK;
+}
+
+template <typename... KArgs, typename... Args>
+int launch_pdl(const char* what, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+               Args... args)
+{
+    return launch_pdl_cluster(what, kernel, 1, grid, block, smem, stream, args...);
 }
 
 }  // namespace tllm

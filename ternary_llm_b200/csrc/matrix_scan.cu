@@ -656,14 +656,24 @@ int chunk_path(const MatrixScanArgs<bf16>& a, cudaStream_t stream)
 int chunk_any(const MatrixScanArgs<bf16>& a, cudaStream_t stream) { return a.delta ? chunk_path<true>(a, stream) : chunk_path<false>(a, stream); }
 int chunk_any(const MatrixScanArgs<float>&, cudaStream_t) { return TLLM_ERR_SHAPE; }
 
-template <typename T, bool DELTA, bool NORM>
-__global__ void __launch_bounds__(NORM ? kSeqMaxThreads : kSeqThreads)
-matrix_seq_kernel(const MatrixScanArgs<T> a, const GatedNormArgs<T> norm, int lpc)
+template <typename T, bool DELTA>
+__global__ void __launch_bounds__(kSeqThreads)
+matrix_seq_kernel(const MatrixScanArgs<T> a, int lpc)
 {
     extern __shared__ __align__(16) float smem[];
     pdl_launch_dependents();
     pdl_wait();
-    matrix_seq<T, DELTA, NORM>(a, norm, lpc, smem, blockIdx.x, blockIdx.y, blockIdx.z);
+    matrix_seq<T, DELTA>(a, lpc, smem, blockIdx.x, blockIdx.y, blockIdx.z);
+}
+
+template <typename T, bool DELTA, bool NORM>
+__global__ void __launch_bounds__(kSeqThreads)
+matrix_one_kernel(const MatrixScanArgs<T> a, const GatedNormArgs<T> norm, int log_lpc)
+{
+    __shared__ float sh[kSeqThreads / 32 + kSeqMaxCluster];
+    pdl_launch_dependents();
+    pdl_wait();
+    matrix_one<T, DELTA, NORM>(a, norm, log_lpc, sh, blockIdx.x, blockIdx.y, blockIdx.z);
 }
 
 template <typename T, bool DELTA>
@@ -671,13 +681,12 @@ int sequential(const MatrixScanArgs<T>& a, const GatedNormArgs<T>* norm, cudaStr
 {
     const SeqPlan p = seq_plan(a.dim, a.vdim);
     const dim3 grid(p.blocks, a.heads, a.g.n_seq);
-    // one new token, a norm per head: a CTA takes the whole head and its norm
-    if (norm && a.g.seq_len == 1 && norm->groups == a.heads && p.lpc * a.vdim <= kSeqMaxThreads) {
-        const int threads = (p.lpc * a.vdim + 31) / 32 * 32;
-        return launch_pdl("matrix_seq", matrix_seq_kernel<T, DELTA, true>, dim3(1, a.heads, a.g.n_seq), dim3(threads),
-                          seq_smem(a.dim, threads / p.lpc), stream, a, *norm, p.lpc);
-    }
-    const int st = launch_pdl("matrix_seq", matrix_seq_kernel<T, DELTA, false>, grid, dim3(p.threads), p.smem, stream, a, GatedNormArgs<T>(), p.lpc);
+    // one new token, a norm per head: the CTAs of a head share its sum of squares
+    if (norm && a.g.seq_len == 1 && norm->groups == a.heads && p.blocks <= kSeqMaxCluster)
+        return launch_pdl_cluster("matrix_one", matrix_one_kernel<T, DELTA, true>, p.blocks, grid, dim3(p.threads), 0, stream, a, *norm, p.log_lpc);
+    const int st = a.g.seq_len == 1
+                       ? launch_pdl("matrix_one", matrix_one_kernel<T, DELTA, false>, grid, dim3(p.threads), 0, stream, a, GatedNormArgs<T>(), p.log_lpc)
+                       : launch_pdl("matrix_seq", matrix_seq_kernel<T, DELTA>, grid, dim3(p.threads), p.smem, stream, a, p.lpc);
     return st || !norm ? st : launch_gated_norm<T>(*norm, stream);
 }
 

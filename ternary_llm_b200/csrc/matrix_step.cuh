@@ -1,6 +1,8 @@
 // Device code of the matrix recurrences that several kernels share: the token-by-token form and the
 // gated norm of an output row.
 #pragma once
+#include <cooperative_groups.h>
+
 #include "launch.cuh"
 #include "mixers.cuh"
 
@@ -12,18 +14,30 @@ constexpr float kUnitEps = 1e-6f;     // under the root of the unit vectors
 
 __device__ __forceinline__ float log_decay(float a, float dt_bias, float neg_a) { return neg_a * softplus_f(a + dt_bias); }
 
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(bf16* p, float4 v)
+{
+    const __nv_bfloat162 x = __floats2bfloat162_rn(v.x, v.y), y = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
+}
+__device__ __forceinline__ float4 get4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 get4(const bf16* p)
+{
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
+                       __uint_as_float(v.y & 0xffff0000u));
+}
+
 // ---------------------------------------------------------------------------
 // Token by token
 // ---------------------------------------------------------------------------
-constexpr int kSeqThreads = 256, kSeqMaxThreads = 1024, kSeqStates = 16, kSeqTokens = 8;   // entries of a column per lane; tokens staged together
+constexpr int kSeqThreads = 256, kSeqMaxCluster = 8, kSeqStates = 16, kSeqTokens = 8;   // entries of a column per lane; tokens staged together
 
 // A column of S is spread over `lpc` lanes in pieces of four entries; a CTA serves blockDim / lpc
 // columns of one head.
-//
-// NORM (a single new token, one CTA per head): the head's output goes through its norm and gate
-// here.  (bx, h, b): column block, head, sequence.
-template <typename T, bool DELTA, bool NORM>
-__device__ __forceinline__ void matrix_seq(const MatrixScanArgs<T>& a, const GatedNormArgs<T>& norm, int lpc, float* smem, int bx, int h, int b)
+// (bx, h, b): column block, head, sequence.
+template <typename T, bool DELTA>
+__device__ __forceinline__ void matrix_seq(const MatrixScanArgs<T>& a, int lpc, float* smem, int bx, int h, int b)
 {
     constexpr int NP = kSeqStates / 4;
     const int cols = blockDim.x / lpc, D = a.dim, D4 = D >> 2;
@@ -43,13 +57,7 @@ __device__ __forceinline__ void matrix_seq(const MatrixScanArgs<T>& a, const Gat
         const int p = l + u * lpc;
         S[u] = p < D4 ? st[p] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    // requested together with the state, needed behind it
     const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
-    float gate = 0.f, weight = 0.f;
-    if (NORM && live && l == 0) {
-        gate = to_f<T>(norm.gate[(size_t)b * norm.ld_gate + (size_t)h * a.vdim + c]);
-        weight = norm.w[c];
-    }
     if (fresh || !live) {
 #pragma unroll
         for (int u = 0; u < NP; u++) S[u] = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -99,7 +107,6 @@ __device__ __forceinline__ void matrix_seq(const MatrixScanArgs<T>& a, const Gat
 #pragma unroll
             for (int u = 0; u < NP; u++) k[u] = l + u * lpc < D4 ? kp[l + u * lpc] : make_float4(0.f, 0.f, 0.f, 0.f);
             float add = vs[t * cols + cl];
-            if (NORM) __syncthreads();                      // vs is used again
             if (DELTA) {
                 float p = 0.f;
 #pragma unroll
@@ -127,18 +134,7 @@ __device__ __forceinline__ void matrix_seq(const MatrixScanArgs<T>& a, const Gat
                 }
             }
             for (int s = lpc >> 1; s > 0; s >>= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
-            if (NORM) {
-                // sum of squares over the columns, each counted once
-                float ss = warp_sum(l == 0 && live ? o * o : 0.f);
-                if (lane == 0) vs[warp] = ss;               // the value has been read by now: see the barrier
-                __syncthreads();
-                ss = 0.f;
-                for (int i = 0; i < warps; i++) ss += vs[i];
-                if (live && l == 0) {
-                    const float f = norm.out_scale / sqrtf(ss / (float)norm.n_true + norm.eps);
-                    norm.out[(size_t)b * norm.ld_out + (size_t)h * a.vdim + c] = from_f<T>(o * f * weight * apply_act(norm.act, gate));
-                }
-            } else if (live && l == 0) a.o[(row0 + t0 + t) * ((size_t)a.heads * a.vdim) + (size_t)h * a.vdim + c] = o;
+            if (live && l == 0) a.o[(row0 + t0 + t) * ((size_t)a.heads * a.vdim) + (size_t)h * a.vdim + c] = o;
         }
     }
     if (live) {
@@ -148,16 +144,129 @@ __device__ __forceinline__ void matrix_seq(const MatrixScanArgs<T>& a, const Gat
     }
 }
 
+// A single new token per sequence, the same layout of a column over lanes: everything a thread needs
+// is requested at once, and the lanes of a column find the vectors' lengths among themselves.
+// NORM (the CTAs of a head form a cluster): the head's output goes through its norm and gate here;
+// sh: 16 words of shared memory.
+template <typename T, bool DELTA, bool NORM>
+__device__ __forceinline__ void matrix_one(const MatrixScanArgs<T>& a, const GatedNormArgs<T>& norm, int log_lpc, float* sh, int bx, int h, int b)
+{
+    constexpr int NP = kSeqStates / 4;
+    const int tid = threadIdx.x, lane = tid & 31, D = a.dim, D4 = D >> 2, lpc = 1 << log_lpc;
+    if (NORM && gridDim.x > 1) cooperative_groups::this_cluster().barrier_arrive();
+    const int l = tid & (lpc - 1), c = bx * (blockDim.x >> log_lpc) + (tid >> log_lpc);
+    const bool live = c < a.vdim;
+    const int col = live ? c : 0, kh = a.kv_heads == a.heads ? h : h / (a.heads / a.kv_heads);
+    float4* st = reinterpret_cast<float4*>(a.state + (size_t)(a.g.first_slot + b) * a.slot_stride + ((size_t)h * a.vdim + col) * D);
+    const T *kp = a.k + (size_t)b * a.ld + (size_t)kh * D, *qp = a.q + (size_t)b * a.ld + (size_t)kh * D;
+    float4 S[NP], k[NP], q[NP];
+#pragma unroll
+    for (int u = 0; u < NP; u++) {
+        const int p = l + (u << log_lpc);
+        const bool in = p < D4;
+        S[u] = in ? st[p] : make_float4(0.f, 0.f, 0.f, 0.f);
+        k[u] = in ? get4(kp + 4 * p) : make_float4(0.f, 0.f, 0.f, 0.f);
+        q[u] = in ? get4(qp + 4 * p) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    float add = to_f<T>(a.v[(size_t)b * a.ld + (size_t)h * a.vdim + col]);
+    const size_t ab = (size_t)b * a.ld_ab + h;
+    float g, beta = 0.f, gate = 0.f, weight = 0.f;
+    if (DELTA) {
+        beta = a.b[ab];
+        g = log_decay(a.a[ab], a.dt_bias[h], a.neg_a[h]);
+    } else {
+        g = a.decay[h];
+    }
+    if (NORM) {
+        gate = to_f<T>(norm.gate[(size_t)b * norm.ld_gate + (size_t)h * a.vdim + col]);
+        weight = norm.w[col];
+    }
+    const bool fresh = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) == 0;
+    if (fresh) {
+#pragma unroll
+        for (int u = 0; u < NP; u++) S[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    float fq = 1.f;
+    if (DELTA) {
+        beta = sigmoid_f(beta);
+        g = decay_exp(g, expf(g));
+        float kk = 0.f, qq = 0.f, p = 0.f;
+#pragma unroll
+        for (int u = 0; u < NP; u++) {
+            kk += (k[u].x * k[u].x + k[u].y * k[u].y) + (k[u].z * k[u].z + k[u].w * k[u].w);
+            qq += (q[u].x * q[u].x + q[u].y * q[u].y) + (q[u].z * q[u].z + q[u].w * q[u].w);
+        }
+        for (int o = lpc >> 1; o > 0; o >>= 1) {
+            kk += __shfl_xor_sync(0xffffffffu, kk, o);
+            qq += __shfl_xor_sync(0xffffffffu, qq, o);
+        }
+        const float fk = 1.f / sqrtf(kk + kUnitEps);
+        fq = a.q_scale / sqrtf(qq + kUnitEps);
+#pragma unroll
+        for (int u = 0; u < NP; u++) {
+            k[u].x *= fk;
+            k[u].y *= fk;
+            k[u].z *= fk;
+            k[u].w *= fk;
+            S[u].x *= g;
+            S[u].y *= g;
+            S[u].z *= g;
+            S[u].w *= g;
+            p = fmaf(S[u].x, k[u].x, fmaf(S[u].y, k[u].y, fmaf(S[u].z, k[u].z, fmaf(S[u].w, k[u].w, p))));
+        }
+        for (int o = lpc >> 1; o > 0; o >>= 1) p += __shfl_xor_sync(0xffffffffu, p, o);
+        add = beta * (add - p);
+    }
+    float o = 0.f;
+#pragma unroll
+    for (int u = 0; u < NP; u++) {
+        const float d = DELTA ? 1.f : g;
+        S[u].x = fmaf(k[u].x, add, d * S[u].x);
+        S[u].y = fmaf(k[u].y, add, d * S[u].y);
+        S[u].z = fmaf(k[u].z, add, d * S[u].z);
+        S[u].w = fmaf(k[u].w, add, d * S[u].w);
+        o = fmaf(S[u].x, q[u].x, fmaf(S[u].y, q[u].y, fmaf(S[u].z, q[u].z, fmaf(S[u].w, q[u].w, o))));
+        if (live && l + (u << log_lpc) < D4) st[l + (u << log_lpc)] = S[u];
+    }
+    for (int s = lpc >> 1; s > 0; s >>= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
+    o *= fq;
+    if (!NORM) {
+        if (live && l == 0) a.o[((size_t)b * a.heads + h) * a.vdim + c] = o;
+        return;
+    }
+    float ss = warp_sum(l == 0 && live ? o * o : 0.f);           // each column counts once
+    const int warps = blockDim.x >> 5;
+    if (lane == 0) sh[tid >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int i = 0; i < warps; i++) ss += sh[i];
+    if (gridDim.x > 1) {
+        cooperative_groups::cluster_group cluster = cooperative_groups::this_cluster();
+        cluster.barrier_wait();                                  // the others are running, their shared memory is there
+        if (tid < (int)gridDim.x) cluster.map_shared_rank(sh, tid)[8 + bx] = ss;
+        cluster.sync();
+        ss = 0.f;
+        for (int i = 0; i < (int)gridDim.x; i++) ss += sh[8 + i];
+    }
+    if (live && l == 0)
+        norm.out[(size_t)b * norm.ld_out + (size_t)h * a.vdim + c] =
+            from_f<T>(o * (norm.out_scale / sqrtf(ss / (float)norm.n_true + norm.eps)) * weight * apply_act(norm.act, gate));
+}
+
 struct SeqPlan {
-    int lpc, threads, blocks;
+    int lpc, log_lpc, threads, blocks;
     size_t smem;
 };
-inline size_t seq_smem(int dim, int cols) { return ((size_t)kSeqTokens * (2 * dim + cols + 2) + 32) * sizeof(float); }
+inline size_t seq_smem(int dim, int cols) { return (size_t)kSeqTokens * (2 * dim + cols + 2) * sizeof(float); }
 inline SeqPlan seq_plan(int dim, int vdim)
 {
     SeqPlan p;
     p.lpc = 1;
-    while (p.lpc * kSeqStates < dim) p.lpc *= 2;
+    p.log_lpc = 0;
+    while (p.lpc * kSeqStates < dim) {
+        p.lpc *= 2;
+        p.log_lpc++;
+    }
     p.threads = kSeqThreads;
     const int cols = p.threads / p.lpc;
     p.blocks = (vdim + cols - 1) / cols;
@@ -178,20 +287,6 @@ int check_matrix_scan(const MatrixScanArgs<T>& a)
 // Gated norm
 // ---------------------------------------------------------------------------
 constexpr int kGnThreads = 256, kGnWarps = kGnThreads / 32;
-
-__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void put4(bf16* p, float4 v)
-{
-    const __nv_bfloat162 x = __floats2bfloat162_rn(v.x, v.y), y = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
-}
-__device__ __forceinline__ float4 get4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 get4(const bf16* p)
-{
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
-                       __uint_as_float(v.y & 0xffff0000u));
-}
 
 // One row by a CTA; sh: kGnWarps words; a warp per group, or the whole CTA when the row is one group
 template <typename T>
