@@ -302,22 +302,33 @@ __device__ __forceinline__ void grouped_span(const GroupedArgs<T>& a, float* __r
 template <typename T, int TK>
 __device__ __forceinline__ void grouped_merge(const GroupedArgs<T>& a, const float* __restrict__ ws, int nsplit, int row, int h, float* wgt)
 {
-    const int t = row % a.g.seq_len;
+    constexpr int kAtOnce = 16;
+    const int t = row % a.g.seq_len, c0 = threadIdx.x;
+    const size_t ld = a.vdim + 2;
+    const float* rec = ws + ((size_t)row * a.heads + h) * nsplit * ld;
+    // the records are requested before it is known how many of them count
+    float v[kAtOnce], m = -FLT_MAX, l = 0.f;
+#pragma unroll
+    for (int s = 0; s < kAtOnce; s++) v[s] = (s < nsplit && c0 < a.vdim) ? rec[s * ld + c0] : 0.f;
+    if (threadIdx.x < nsplit) {
+        m = rec[threadIdx.x * ld + a.vdim];
+        l = rec[threadIdx.x * ld + a.vdim + 1];
+    }
     const int pos = (a.g.pos_dev ? *a.g.pos_dev : a.g.start_pos) + t;
     if (pos >= a.max_seq) return;
     const int span = pos + 1 - first_seen(pos, a.chunk), len = range_len(span, nsplit, TK), n = (span + len - 1) / len;
-    const float* rec = ws + ((size_t)row * a.heads + h) * nsplit * (a.vdim + 2);
     if (threadIdx.x < 32) {
-        const int s = threadIdx.x;
-        const float m = s < n ? rec[(size_t)s * (a.vdim + 2) + a.vdim] : -FLT_MAX, mx = warp_max(m);
-        const float e = s < n ? expf(m - mx) : 0.f, l = warp_sum(s < n ? e * rec[(size_t)s * (a.vdim + 2) + a.vdim + 1] : 0.f);
-        wgt[s] = e * a.out_scale / l;
+        const bool counts = threadIdx.x < n;
+        const float mx = warp_max(counts ? m : -FLT_MAX), e = counts ? expf(m - mx) : 0.f, sum = warp_sum(counts ? e * l : 0.f);
+        wgt[threadIdx.x] = e * a.out_scale / sum;
     }
     __syncthreads();
-    for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) {
+    for (int c = c0; c < a.vdim; c += blockDim.x) {
         float o = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < n; s++) o = fmaf(wgt[s], rec[(size_t)s * (a.vdim + 2) + c], o);
+#pragma unroll
+        for (int s = 0; s < kAtOnce; s++)
+            if (s < n) o = fmaf(wgt[s], c == c0 ? v[s] : rec[s * ld + c], o);
+        for (int s = kAtOnce; s < n; s++) o = fmaf(wgt[s], rec[s * ld + c], o);
         a.out[(size_t)row * a.ld_out + (size_t)h * a.vdim + c] = from_f<T>(o);
     }
 }
