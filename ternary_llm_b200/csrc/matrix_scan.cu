@@ -36,7 +36,8 @@ __host__ __device__ inline int inverse_floats(int ld) { return kC * (ld / 2 > kL
 
 // What the first launch leaves for the second, laid out as it lies in shared memory there, so that a
 // tile is one bulk copy.  Per (sequence, chunk, key head): keys, then queries, [64][ld], zero behind
-// the sequence; per (sequence, chunk, head): slices of `nv` value columns [64][nv + 8]; matrices [64][kLdC] as they lie in shared memory, BF16 high and low parts -- P, then with the delta
+// the sequence; per (sequence, chunk, head): slices of `nv` value columns [64][nv + 8]; matrices
+// [64][kLdC], BF16 high and low parts -- P, then with the delta
 // rule the inverse -- and four vectors of 64 floats (log of the running decay, step size, 1/|k|,
 // q_scale/|q|)
 struct ChunkWs {

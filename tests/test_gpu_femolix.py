@@ -22,11 +22,11 @@ LIMIT = {"float32": 1e-4, "bfloat16": 6e-2}
 
 CONFIGS = {
     "all": X.config([X.delta(mlp=X.dense(40)), X.parallel(mlp=X.moe(6, 2, 24)), X.parallel(size=16, mlp=X.dense(18)), X.delta(conv=2, mlp=X.moe(5, 3, 20))]),
-    "delta": X.config([X.delta(heads=2, kv_heads=1, dim=64, vdim=64, conv=4), X.delta(heads=3, kv_heads=3, dim=9, vdim=7, conv=1, mlp=X.dense(11)),
+    "delta": X.config([X.delta(heads=3, kv_heads=1, dim=64, vdim=80, conv=4), X.delta(heads=3, kv_heads=3, dim=9, vdim=7, conv=1, mlp=X.dense(11)),
                        X.delta(heads=4, kv_heads=4, dim=24, vdim=72, conv=5)], width=72, vocab=257, eps=1e-3, alpha=1.0),
     "parallel": X.config([X.parallel(heads=8, kv_heads=8, dim=24, vdim=24, size=50, rot=24, r_heads=2, r_dim=40, r_vdim=72),
                           X.parallel(heads=5, kv_heads=1, dim=10, vdim=9, size=1, rot=2, r_heads=1, r_dim=7, r_vdim=33, decay=[0.999]),
-                          X.parallel(heads=4, kv_heads=2, size=200, rot=4, left=1.0, right=1.0, r_heads=6, r_dim=16, r_vdim=8)], width=50, alpha=2.5),
+                          X.parallel(heads=4, kv_heads=2, size=130, rot=4, left=1.0, right=1.0, r_heads=6, r_dim=16, r_vdim=8)], width=50, alpha=2.5),
     "experts": X.config([X.delta(mlp=X.moe(3, 3, 9)), X.delta(mlp=X.moe(12, 1, 16)), X.parallel(mlp=X.moe(9, 4, 33))], width=30, cap=3.0),
     "narrow": X.config([X.delta(heads=1, kv_heads=1, dim=4, vdim=5, conv=4, mlp=X.dense(6)), X.parallel(heads=2, kv_heads=1, dim=4, vdim=3, rot=2, r_heads=1)],
                        width=9, vocab=17, alpha=0.8),

@@ -105,20 +105,20 @@ def test_grouped_attention_over_long_prompts(chunk, ring, d, e):
 
 
 @pytest.mark.parametrize("dt", list(DT))
-@pytest.mark.parametrize("chunk", [0, 200])
+@pytest.mark.parametrize("chunk", [0, 190])
 @pytest.mark.parametrize("d", [16, 64])
 def test_grouped_attention_finds_one_key_just_inside_and_never_outside(dt, chunk, d):
     """One key matches the query of every position; its value is the output exactly where the mask
     shows it: from its own position to the end of its chunk."""
     H, G, e, n = 2, 1, {16: 8, 64: 64}[d], 470
-    for at in (0, 63, 64, 199, 200, 399):
+    for at in (0, 63, 64, 189, 190, 379):
         x = np.zeros((1, n, H * d + G * (d + e)))
         x[..., d - 1:H * d:d] = 1.0
         x[:, :, H * d] = 1.0                                     # every other key: orthogonal to the queries
         x[:, at, H * d], x[:, at, H * d + d - 1] = 0.0, 1.0
         x[:, at, (H + G) * d:] = 5.0
         # decode: the last positions one by one, from just before the next chunk's edge
-        for cuts in ([n], [390] + [1] * 80, [190] + [1] * 25 + [255]):
+        for cuts in ([n], [370] + [1] * 100, [180] + [1] * 25 + [265]):
             kc, vc = (torch.zeros(1, n, w, device="cuda", dtype=DT[dt]) for w in (d, e))
             got, pos = [], 0
             for c in cuts:
