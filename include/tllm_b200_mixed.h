@@ -28,8 +28,8 @@ enum {
     TLLM_MIXER_SELECTIVE_SCAN = 2,   /* Mamba */
     TLLM_MIXER_GATED_RECURRENCE = 3, /* Griffin's RG-LRU block */
     TLLM_MIXER_ATTENTION = 4,        /* grouped-query softmax attention */
-    TLLM_MIXER_LINEAR_ATTENTION = 5, /* S <- decay S + k v^T, o = S^T q, a constant decay per head */
-    TLLM_MIXER_DELTA_RULE = 6        /* S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q */
+    TLLM_MIXER_LINEAR_ATTENTION = 5, /* a decaying sum of (key, value) pairs per head, read by the query */
+    TLLM_MIXER_DELTA_RULE = 6        /* a decaying memory per head in which a key's value is replaced, not added */
 };
 enum { TLLM_ACT_NONE = 0, TLLM_ACT_GELU_TANH = 1, TLLM_ACT_SILU = 2, TLLM_ACT_SIGMOID = 4 };
 

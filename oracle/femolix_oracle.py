@@ -52,7 +52,8 @@ def chunked_attention(q, k, v, scale, size):
 # ---- recurrences on a matrix per head ----------------------------------------------------
 def delta_rule(q, k, v, g, beta):
     """q, k [tokens, H, d], v [tokens, H, e], g, beta [tokens, H]:
-    S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q."""
+    the memory fades by g, what it holds under the key moves by the fraction beta towards the value,
+    and the query reads the result."""
     n, H, d = q.shape
     S = np.zeros((H, d, v.shape[2]), F)
     out = np.zeros_like(v, dtype=F)
@@ -66,7 +67,7 @@ def delta_rule(q, k, v, g, beta):
 
 
 def decayed_linear_attention(q, k, v, decay):
-    """S <- decay_h S + k v^T;  o = S^T q."""
+    """A memory per head that fades by its decay and adds each value under its key; the query reads."""
     n, H, d = q.shape
     S = np.zeros((H, d, v.shape[2]), F)
     out = np.zeros_like(v, dtype=F)
