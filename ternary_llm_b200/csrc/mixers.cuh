@@ -188,9 +188,10 @@ template <typename T>
 int launch_grouped_attention(const GroupedArgs<T>& a, float* ws, cudaStream_t stream);
 
 // ---- recurrences on a matrix per head ------------------------------------------------------
-// delta: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, with unit-length q (times
-//   q_scale) and k, g = exp(neg_a softplus(a + dt_bias)), beta = sigmoid(b);
-// else:  S <- decay S + k v^T; o = S^T q.
+// With S_t [vdim][dim] the state behind token t, o_t = S_t q_t and
+//   delta: S_t = g S_(t-1) + beta (v_t - g S_(t-1) k_t) k_t', with unit-length q (times q_scale) and
+//          k, g = exp(neg_a softplus(a + dt_bias)), beta = sigmoid(b);
+//   else:  S_t = decay S_(t-1) + v_t k_t'.
 // Head h reads query/key head h / (heads / kv_heads).  State [slot][heads][vdim][dim].
 template <typename T>
 struct MatrixScanArgs {

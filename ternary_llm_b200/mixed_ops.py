@@ -100,7 +100,7 @@ def grouped_attention(proj, q_norm, k_norm, eps: float, rope, rot_dims: int, kc,
 
 
 def linear_attention(qkv, decay, state, o, heads: int, dim: int, vdim: int, n_seq: int, seq_len: int, start_pos: int) -> None:
-    """S = decay S + k v^T, o = S^T q; qkv [rows, q | k | v], state [n_seq, heads, vdim, dim]."""
+    """S_t = decay S_(t-1) + v k', o = S_t q; qkv [rows, q | k | v], state [n_seq, heads, vdim, dim]."""
     rows = n_seq * seq_len
     _lib.check(_lib.lib().tllm_b200_matrix_scan(
         _kind(qkv), 0, _chk(qkv, qkv.dtype, "qkv", rows * heads * (2 * dim + vdim)), _chk(decay, _F, "decay", heads), None, None, None, None, 1.0,
@@ -110,7 +110,7 @@ def linear_attention(qkv, decay, state, o, heads: int, dim: int, vdim: int, n_se
 
 def delta_rule(qkv, a, b, neg_a, dt_bias, q_scale: float, state, o, heads: int, kv_heads: int, dim: int, vdim: int, n_seq: int, seq_len: int,
                start_pos: int) -> None:
-    """S = g S, u = beta (v - S^T k), S = S + k u^T, o = S^T q with unit-length q (times q_scale)
+    """S_t = g S_(t-1) + beta (v - g S_(t-1) k) k', o = S_t q with unit-length q (times q_scale)
     and k, g = exp(neg_a softplus(a + dt_bias)), beta = sigmoid(b)."""
     rows = n_seq * seq_len
     _lib.check(_lib.lib().tllm_b200_matrix_scan(
